@@ -1,0 +1,291 @@
+// Dense linears on many activation rows (prompts and long portions).
+//
+// bf16: tensor cores.  The weight rows are the 128-row operand of tcgen05.mma and TN tokens its N dimension, so a thread
+// of the epilogue owns one weight row (one segment, one bias) and a warp stores 32 consecutive outputs of a token.
+// Persistent CTAs, one per SM, walk the tiles with the token tiles innermost: the CTAs in flight share a few weight row
+// tiles, which are read from HBM once.  Roles (192 threads): warp 0 TMA producer of both operands (128-byte swizzle, 64
+// columns per stage), warp 1 MMA issuer (one lane), warps 2-5 epilogue.  Two accumulators in TMEM: a tile's epilogue
+// runs under the next tile's MMAs.  Every mbarrier wait is bounded (see greta_cuda_linear_gemm_status).
+//
+// fp32: plain 64 x 64 tiles of 32-bit FMAs, for models that run in 32-bit.
+#include <algorithm>
+
+#include "dense_device.cuh"
+#include "tc_device.cuh"
+
+using namespace greta;
+
+namespace greta {
+int check_linear(const char *what, const greta_linear *l, Segments *sg);
+}
+
+namespace {
+
+template <int TN>
+struct DCfg {
+  static constexpr int A_BYTES = TILE_N * BK * 2, B_BYTES = TN * BK * 2, STAGE = A_BYTES + B_BYTES;
+  static constexpr int ST = TN == 256 ? 4 : TN == 128 ? 6 : 8;
+  static constexpr int COLS = 2 * TN < 32 ? 32 : 2 * TN;  // two accumulators; a power of two
+  static constexpr int THREADS = 192;
+  static constexpr size_t SMEM = (size_t)ST * STAGE + 1024 + 256;
+  static_assert(COLS <= 512 && SMEM <= 232448, "tile configuration");
+};
+
+template <int TN>
+__global__ void __launch_bounds__(DCfg<TN>::THREADS, 1)
+linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ Segments sg, uint32_t M,
+                 uint32_t N, uint32_t K) {
+  using C = DCfg<TN>;
+  constexpr int ST = C::ST;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t *smem = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint64_t *bars = reinterpret_cast<uint64_t *>(smem + (size_t)ST * C::STAGE);
+  uint64_t *full = bars, *empty = bars + ST, *acc_full = bars + 2 * ST, *acc_empty = acc_full + 2;
+  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(acc_empty + 2);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint32_t KT = (K + BK - 1) / BK, tok_tiles = (M + TN - 1) / TN, tiles = tok_tiles * ((N + TILE_N - 1) / TILE_N);
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < ST; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
+    }
+    for (int b = 0; b < 2; ++b) {
+      mbar_init(&acc_full[b], 1);
+      mbar_init(&acc_empty[b], 4);
+    }
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_w) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_x) : "memory");
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, C::COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  pdl_launch_dependents();
+  pdl_wait();
+
+  if (warp == 0) {
+    if (lane == 0) {
+      uint32_t issued = 0, s = 0, ph = 1;
+      bool ok = true;
+      for (uint32_t t = blockIdx.x; t < tiles && ok; t += gridDim.x) {
+        const int n0 = (int)(t / tok_tiles) * TILE_N, m0 = (int)(t % tok_tiles) * TN;
+        for (uint32_t kt = 0; kt < KT; ++kt) {
+          ok = mbar_wait(&empty[s], ph, abort_flag, 100 + s);
+          if (!ok) break;
+          uint8_t *st = smem + (size_t)s * C::STAGE;
+          mbar_arrive_expect_tx(&full[s], C::STAGE);
+          tma_load_2d(st, &tmap_w, (int)(kt * BK), n0, &full[s]);
+          tma_load_2d(st + C::A_BYTES, &tmap_x, (int)(kt * BK), m0, &full[s]);
+          ++issued;
+          if (++s == ST) {
+            s = 0;
+            ph ^= 1;
+          }
+        }
+      }
+      if (*abort_flag) {  // a bounded chance for the copies in flight to land before the CTA exits
+        for (uint32_t j = issued > (uint32_t)ST ? issued - ST : 0; j < issued; ++j) {
+          const long long t0 = clock64();
+          while (!mbar_try_wait(&full[j % ST], (j / ST) & 1) && clock64() - t0 < 20000000ll) {
+          }
+        }
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc = instr_desc_bf16(TILE_N, TN);
+      const uint32_t lo0 = smem_desc_lo(smem_u32(smem));
+      uint32_t s = 0, ph = 0, it = 0;
+      bool ok = true;
+      for (uint32_t t = blockIdx.x; t < tiles && ok; t += gridDim.x, ++it) {
+        const uint32_t b = it & 1;
+        ok = mbar_wait(&acc_empty[b], ((it >> 1) & 1) ^ 1, abort_flag, 300 + b);
+        if (!ok) break;
+        tc_fence_after();
+        for (uint32_t kt = 0; kt < KT; ++kt) {
+          ok = mbar_wait(&full[s], ph, abort_flag, 200 + s);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t w_lo = lo0 + s * (C::STAGE >> 4), x_lo = w_lo + (C::A_BYTES >> 4);
+#pragma unroll
+          for (int k16 = 0; k16 < BK / 16; ++k16)
+            umma_f16(tmem_base + b * TN, w_lo + k16 * 2, x_lo + k16 * 2, SMEM_DESC_HI_SW128, idesc, (kt | k16) ? 1u : 0u);
+          umma_commit(&empty[s]);
+          if (++s == ST) {
+            s = 0;
+            ph ^= 1;
+          }
+        }
+        if (ok) umma_commit(&acc_full[b]);
+      }
+    }
+  } else {
+    const int quad = warp & 3;
+    uint32_t it = 0;
+    for (uint32_t t = blockIdx.x; t < tiles; t += gridDim.x, ++it) {
+      const uint32_t b = it & 1, m0 = (t % tok_tiles) * TN, row = (t / tok_tiles) * TILE_N + quad * 32 + lane;
+      if (!mbar_wait(&acc_full[b], (it >> 1) & 1, abort_flag, 400 + b)) break;
+      tc_fence_after();
+      greta_out_segment g{};
+      uint32_t r = 0;
+      float bias = 0.f;
+      if (row < N) {
+        g = sg.s[segment_of(sg, row)];
+        r = row - g.row0;
+        if (g.bias) bias = __ldg(g.bias + r);
+      }
+#pragma unroll 1
+      for (int c = 0; c < TN; c += 32) {
+        uint32_t v[32];
+        __syncwarp();
+        if (m0 + c < M) {
+          tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + b * TN + c, v);
+          tmem_ld_wait();
+        }
+        if (c + 32 >= TN) {  // accumulator read: the issuer may overwrite it
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&acc_empty[b]);
+        }
+        if (row < N && m0 + c < M) {
+          const uint32_t cnt = min(32u, M - m0 - c);
+          const size_t base = (size_t)(m0 + c) * g.ld + g.col0 + r;
+          if (g.accumulate) {
+            float *o = static_cast<float *>(g.out) + base;
+            float old[32];
+#pragma unroll
+            for (int j = 0; j < 32; ++j) old[j] = j < cnt ? o[(size_t)j * g.ld] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (j < cnt) o[(size_t)j * g.ld] = old[j] + apply_act(g.act, __uint_as_float(v[j]) + bias);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(g.act, __uint_as_float(v[j]) + bias), g.pair_offset);
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, C::COLS);
+  }
+}
+
+// C tile 64 rows of x x 64 rows of W, 256 threads, 4 x 4 outputs each, 16 columns per step.
+__global__ void __launch_bounds__(256) linear_f32_kernel(const float *__restrict__ W, uint32_t N, uint32_t ldw, const float *__restrict__ x, uint32_t ldx,
+                                                         uint32_t M, const __grid_constant__ Segments sg) {
+  __shared__ float ws[16][68], xs[16][68];
+  pdl_launch_dependents();
+  pdl_wait();
+  const uint32_t n0 = blockIdx.x * 64, m0 = blockIdx.y * 64;
+  const uint32_t lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;  // loads: row, column group
+  const uint32_t tn = (threadIdx.x & 15) * 4, tm = (threadIdx.x >> 4) * 4;
+  const float *wp = W + (size_t)min(n0 + lr, N - 1) * ldw + lc, *xp = x + (size_t)min(m0 + lr, M - 1) * ldx + lc;
+  float acc[4][4] = {};
+  for (uint32_t k = 0; k < ldw; k += 16) {
+    const float4 a = *reinterpret_cast<const float4 *>(wp + k), b = *reinterpret_cast<const float4 *>(xp + k);
+    __syncthreads();
+    ws[lc][lr] = a.x, ws[lc + 1][lr] = a.y, ws[lc + 2][lr] = a.z, ws[lc + 3][lr] = a.w;
+    xs[lc][lr] = b.x, xs[lc + 1][lr] = b.y, xs[lc + 2][lr] = b.z, xs[lc + 3][lr] = b.w;
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < 16; ++kk) {
+      const float4 p = *reinterpret_cast<const float4 *>(&ws[kk][tn]), q = *reinterpret_cast<const float4 *>(&xs[kk][tm]);
+      const float pn[4] = {p.x, p.y, p.z, p.w}, qm[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(qm[i], pn[j], acc[i][j]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const uint32_t row = n0 + tn + j;
+    if (row >= N) continue;
+    const greta_out_segment &g = sg.s[segment_of(sg, row)];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (m0 + tm + i < M) store_segment(g, row, m0 + tm + i, acc[i][j]);
+  }
+}
+
+int make_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, uint32_t ld, uint32_t box_rows) {
+  EncodeTiledFn enc = encode_tiled();
+  if (!enc) {
+    set_error("linear_gemm: cuTensorMapEncodeTiled is not available from this driver");
+    return GRETA_ERR_NOT_IMPLEMENTED;
+  }
+  const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(cuuint64_t)ld * 2};
+  const cuuint32_t box[2] = {BK, box_rows}, estr[2] = {1, 1};
+  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) {
+    set_error("linear_gemm: cuTensorMapEncodeTiled failed with code %d", (int)r);
+    return GRETA_ERR_INVALID_ARGS;
+  }
+  return GRETA_OK;
+}
+
+template <int TN>
+int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, const void *x, uint32_t ldx, uint32_t M) {
+  using C = DCfg<TN>;
+  static bool attr_set[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !attr_set[dev]) {
+    GRETA_CUDA_TRY(cudaFuncSetAttribute(linear_tc_kernel<TN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+    attr_set[dev] = true;
+  }
+  CUtensorMap mw, mx;
+  if (int rc = make_map(&mw, l->w, l->K, l->N, l->ldw, TILE_N)) return rc;  // columns past K read as zero in both operands
+  if (int rc = make_map(&mx, x, l->K, M, ldx, TN)) return rc;
+  const uint32_t tiles = ((l->N + TILE_N - 1) / TILE_N) * ((M + TN - 1) / TN);
+  GRETA_CUDA_TRY(launch_pdl(linear_tc_kernel<TN>, dim3(std::min(tiles, (uint32_t)sm_count())), dim3(C::THREADS), C::SMEM, s, mw, mx, sg, M, l->N, l->K));
+  return launched("linear_tc_kernel");
+}
+
+}  // namespace
+
+extern "C" {
+
+int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *l, const void *x, uint32_t ldx, uint32_t M) {
+  if (M == 0) return GRETA_OK;
+  Segments sg{};
+  if (int rc = check_linear("linear_gemm", l, &sg)) return rc;
+  GRETA_REQUIRE(x && aligned16(x), "linear_gemm: null or misaligned activations");
+  cudaStream_t s = (cudaStream_t)stream;
+  if (l->fmt == GRETA_FMT_F32) {
+    GRETA_REQUIRE(ldx >= l->ldw && ldx % 4 == 0, "linear_gemm: fp32 activations need rows of ldw=%u columns (ldx=%u)", l->ldw, ldx);
+    GRETA_CUDA_TRY(launch_pdl(linear_f32_kernel, dim3((l->N + 63) / 64, (M + 63) / 64), dim3(256), 0, s, static_cast<const float *>(l->w), l->N, l->ldw,
+                              static_cast<const float *>(x), ldx, M, sg));
+    return launched("linear_f32_kernel");
+  }
+  GRETA_REQUIRE(ldx >= l->K && ldx % 8 == 0, "linear_gemm: ldx=%u K=%u", ldx, l->K);
+  // the widest token tile that still gives most SMs a tile
+  const uint32_t row_tiles = (l->N + TILE_N - 1) / TILE_N;
+  auto enough = [&](uint32_t tn) { return row_tiles * ((M + tn - 1) / tn) >= 120 && M > tn / 2; };
+  if (enough(256)) return launch_dense<256>(s, l, sg, x, ldx, M);
+  if (enough(128)) return launch_dense<128>(s, l, sg, x, ldx, M);
+  if (enough(64)) return launch_dense<64>(s, l, sg, x, ldx, M);
+  return launch_dense<32>(s, l, sg, x, ldx, M);
+}
+
+int greta_cuda_linear_gemm_status(int *code) {
+  GRETA_REQUIRE(code, "linear_gemm_status: null out pointer");
+  GRETA_CUDA_TRY(cudaMemcpyFromSymbol(code, g_gemm_error, sizeof(int)));
+  return GRETA_OK;
+}
+
+}  // extern "C"

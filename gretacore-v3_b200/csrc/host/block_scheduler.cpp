@@ -91,6 +91,7 @@ bool BlockScheduler::init(const ModelConfig &config, std::string *err) {
   config_ = config;
   const ModelConfig &c = config_;
   if (c.tp_size == 0 || c.tp_rank >= c.tp_size) return fail(err, "init: bad tensor-parallel rank");
+  if (c.arch == ModelArch::HYBRID) return init_hybrid(err);
   if (c.dim % 256 || c.hidden_dim % (32 * c.tp_size) || c.num_heads % c.tp_size || c.num_heads_kv % c.tp_size ||
       c.num_heads % c.num_heads_kv || c.vocab_size % c.tp_size)
     return fail(err, "init: model shape is not divisible by the quant block / tensor-parallel degree");
@@ -116,6 +117,10 @@ bool BlockScheduler::allocate_weights(std::string *err) {
   const int fmt = fmt_of(c.weight_type);
   blocks_ = std::vector<BlockBuffers>(c.num_layers);
   weight_bytes_ = 0;
+  if (c.arch == ModelArch::HYBRID) {  // sized and filled layer by layer when the weights are loaded
+    hybrid_ = std::vector<HybridLayerBuffers>(c.num_layers);
+    return true;
+  }
   for (auto &b : blocks_) {
     for (int t = 0; t <= (int)LayerTensor::W3_UP; ++t) {
       Shape s = shard_of(c, (LayerTensor)t);
@@ -159,6 +164,7 @@ bool BlockScheduler::allocate_activations(size_t batch_size, size_t max_seq_len,
   max_seq_ = max_seq_len;
   batch_ = (uint32_t)batch_size;
   cur_seq_ = 0;
+  if (c.arch == ModelArch::HYBRID) return allocate_hybrid_activations(err);
   const size_t S = std::max(max_seq_len, batch_size), D = c.dim, B = batch_size;
   const size_t ql = (size_t)heads_l_ * c.head_dim, kvl = (size_t)kv_heads_l_ * c.head_dim;
   auto dev = [&](Buffer &b, size_t bytes, GretaDataType t = GretaDataType::FP32) { return b.allocate(bytes, BufferUsage::DeviceOnly, t, err); };
@@ -207,6 +213,7 @@ static bool upload_blocks(GretaDataType type, const uint8_t *host, uint32_t rows
 }
 
 bool BlockScheduler::set_layer_tensor(size_t layer, LayerTensor which, const void *host, size_t bytes, std::string *err) {
+  if (config_.arch == ModelArch::HYBRID) return fail(err, "set_layer_tensor: a hybrid model is loaded as a whole (load_weights)");
   if (layer >= blocks_.size()) return fail(err, "set_layer_tensor: layer out of range (allocate_weights first)");
   BlockBuffers &b = blocks_[layer];
   if (which == LayerTensor::ATTN_NORM || which == LayerTensor::FFN_NORM) {
@@ -282,6 +289,7 @@ bool BlockScheduler::set_global_tensor_kquant(GlobalTensor which, int ggml_type,
 
 bool BlockScheduler::set_global_tensor(GlobalTensor which, const void *host, size_t bytes, std::string *err) {
   const ModelConfig &c = config_;
+  if (c.arch == ModelArch::HYBRID) return fail(err, "set_global_tensor: a hybrid model is loaded as a whole (load_weights)");
   if (which == GlobalTensor::TOK_EMBD) {
     if (bytes != token_embd_.size()) return fail(err, "set_global_tensor: embedding size mismatch");
     return token_embd_.copy_to_device(host, bytes, err);
@@ -303,6 +311,7 @@ bool BlockScheduler::set_global_tensor(GlobalTensor which, const void *host, siz
 
 bool BlockScheduler::load_synthetic_weights(uint64_t seed, std::string *err) {
   if (blocks_.empty()) return fail(err, "load_synthetic_weights: allocate_weights first");
+  if (config_.arch == ModelArch::HYBRID) return load_hybrid_synthetic(seed, err);
   const ModelConfig &c = config_;
   const size_t bb = block_bytes(c.weight_type);
   Buffer staging;
@@ -575,6 +584,7 @@ bool BlockScheduler::execute_layer(size_t layer_idx, size_t seq_start, size_t se
   const ModelConfig &c = config_;
   ActivationBuffers &a = activations_;
   if (layer_idx >= blocks_.size()) return fail(err, "execute_layer: layer out of range");
+  if (c.arch == ModelArch::HYBRID) return hybrid_layer(layer_idx, greta_rows{(uint32_t)seq_len, cur_seq_, (uint32_t)seq_start, nullptr}, err);
   BlockBuffers &b = blocks_[layer_idx];
   cudaStream_t s = H(stream_);
   const int fmt = fmt_of(c.weight_type);
@@ -620,6 +630,14 @@ bool BlockScheduler::forward(const int32_t *tokens, size_t seq_start, size_t seq
   const ModelConfig &c = config_;
   ActivationBuffers &a = activations_;
   cudaStream_t s = H(stream_);
+  if (c.arch == ModelArch::HYBRID) {
+    auto last = [&](size_t first, size_t n) {
+      return first + n < seq_len || hybrid_logits(static_cast<const float *>(a.x.data()) + (n - 1) * c.dim, 1, static_cast<float *>(logits_.data()), err);
+    };
+    if (!hybrid_run(tokens, seq_start, seq_len, last, err)) return false;
+    GRETA_TRY(greta_cuda_stream_synchronize(s), "forward");
+    return true;
+  }
   GRETA_TRY(greta_cuda_memcpy_h2d(a.tokens.data(), tokens, seq_len * 4, s), "token upload");
   GRETA_TRY(greta_cuda_embedding(s, static_cast<const int32_t *>(a.tokens.data()), token_embd_.data(), 1, static_cast<float *>(a.x.data()),
                                  (uint32_t)seq_len, c.dim, c.vocab_size),
@@ -636,6 +654,43 @@ bool BlockScheduler::forward(const int32_t *tokens, size_t seq_start, size_t seq
   }
   if (!lm_head(static_cast<const float *>(a.x.data()) + (seq_len - 1) * c.dim, err)) return false;
   GRETA_TRY(greta_cuda_stream_synchronize(s), "forward");
+  return true;
+}
+
+bool BlockScheduler::forward_logits(const int32_t *tokens, size_t seq_start, size_t seq_len, const uint32_t *rows, size_t n_rows, float *out,
+                                    std::string *err) {
+  for (size_t i = 0; i < n_rows; ++i)
+    if (rows[i] >= seq_len || (i && rows[i] <= rows[i - 1])) return fail(err, "forward_logits: rows must ascend inside the portion");
+  const ModelConfig &c = config_;
+  const float *x = static_cast<const float *>(activations_.x.data());
+  if (c.arch != ModelArch::HYBRID) {
+    if (!forward(tokens, seq_start, seq_len, err)) return false;
+    for (size_t i = 0; i < n_rows; ++i) {
+      if (c.tp_size > 1) GRETA_TRY(greta_cuda_memset(logits_.data(), 0, logits_.size(), H(stream_)), "logits clear");
+      if (!lm_head(x + (size_t)rows[i] * c.dim, err)) return false;
+      GRETA_TRY(greta_cuda_stream_synchronize(H(stream_)), "forward_logits");
+      if (!logits_.copy_to_host_offset(out + i * c.vocab_size, 0, (size_t)c.vocab_size * 4, err)) return false;
+    }
+    return true;
+  }
+  if (blocks_.empty() || !x) return fail(err, "forward_logits: allocate weights and activations first");
+  if (seq_len == 0 || seq_start + seq_len > max_seq_) return fail(err, "forward_logits: sequence exceeds max_seq_len");
+  size_t done = 0;
+  auto wanted = [&](size_t first, size_t n) {  // the wanted rows of this portion, at most 64 at a time
+    while (done < n_rows && rows[done] < first + n) {
+      uint32_t list[64], k = 0;
+      for (; k < 64 && done + k < n_rows && rows[done + k] < first + n; ++k) list[k] = rows[done + k] - (uint32_t)first;
+      float *xr = static_cast<float *>(hact_.x_rows.data()), *z = static_cast<float *>(hact_.logits_rows.data());
+      GRETA_TRY(greta_cuda_gather_rows(H(stream_), x, c.dim, list, k, xr), "gather_rows");
+      if (!hybrid_logits(xr, k, z, err)) return false;
+      GRETA_TRY(greta_cuda_stream_synchronize(H(stream_)), "forward_logits");
+      if (!hact_.logits_rows.copy_to_host_offset(out + done * c.vocab_size, 0, (size_t)k * c.vocab_size * 4, err)) return false;
+      done += k;
+    }
+    return true;
+  };
+  if (!hybrid_run(tokens, seq_start, seq_len, wanted, err)) return false;
+  GRETA_TRY(greta_cuda_stream_synchronize(H(stream_)), "forward_logits");
   return true;
 }
 
@@ -730,15 +785,25 @@ bool BlockScheduler::begin_decode_batch(const int32_t *first_tokens, const uint3
     // gives identical results and is kept as an option: measured slower so far (the per-phase
     // activation staging and grid barriers cost more than the launches they replace).
     const char *env = std::getenv("GRETA_PERSISTENT_STEP");
-    persistent_step_ = c.tp_size == 1 && batch_ == 1 && env && env[0] == '1';
+    const bool hybrid = c.arch == ModelArch::HYBRID;
+    persistent_step_ = !hybrid && c.tp_size == 1 && batch_ == 1 && env && env[0] == '1';
     if (persistent_step_ && !build_decode_plan(err)) return false;
     greta_decode_desc desc;
-    fill_decode_desc(desc, c, a, token_embd_, max_seq_);
+    if (!hybrid) fill_decode_desc(desc, c, a, token_embd_, max_seq_);
     graph_ = gcore::rt::GretaContext::instance().create_graph();
     graph_->capture_start(stream_);  // void, as in the reference: a capture that failed shows at instantiate()
     bool ok;
     const float *x_last = static_cast<const float *>(a.x.data());
-    if (batch_ > 1) {
+    if (hybrid) {
+      const greta_rows rows{batch_, 0, 0, static_cast<const uint32_t *>(a.d_pos.data())};
+      ok = hybrid_embed(static_cast<const int32_t *>(a.d_next.data()), rows, err);
+      for (size_t l = 0; ok && l < hybrid_.size(); ++l) ok = hybrid_layer(l, rows, err);
+      ok = ok && hybrid_logits(x_last, batch_, static_cast<float *>(logits_.data()), err);
+      uint32_t *dp = static_cast<uint32_t *>(a.d_pos.data());
+      ok = ok && greta_cuda_argmax_advance_batch(s, static_cast<const float *>(logits_.data()), c.vocab_size, batch_,
+                                                 static_cast<int32_t *>(a.d_next.data()), dp, static_cast<int32_t *>(a.out_tokens.data()), dp + batch_,
+                                                 (uint32_t)max_seq_) == GRETA_OK;
+    } else if (batch_ > 1) {
       ok = greta_cuda_embedding(s, static_cast<const int32_t *>(a.d_next.data()), token_embd_.data(), 1, static_cast<float *>(a.x.data()), batch_,
                                 c.dim, c.vocab_size) == GRETA_OK;
       if (ok && c.tp_size > 1) ok = greta_cuda_memset(logits_.data(), 0, logits_.size(), s) == GRETA_OK;
@@ -756,9 +821,9 @@ bool BlockScheduler::begin_decode_batch(const int32_t *first_tokens, const uint3
       if (ok && c.tp_size > 1) ok = greta_cuda_memset(logits_.data(), 0, logits_.size(), s) == GRETA_OK;
       ok = ok && decode_layers(err, peer_.tp > 1, &x_last);
     }
-    if (batch_ == 1) ok = ok && lm_head(x_last, err);
+    if (batch_ == 1 && !hybrid) ok = ok && lm_head(x_last, err);
     uint32_t *dp = static_cast<uint32_t *>(a.d_pos.data());
-    if (batch_ == 1) ok = ok && greta_cuda_argmax_advance(s, static_cast<const float *>(logits_.data()), c.vocab_size, static_cast<int32_t *>(a.d_next.data()), dp,
+    if (batch_ == 1 && !hybrid) ok = ok && greta_cuda_argmax_advance(s, static_cast<const float *>(logits_.data()), c.vocab_size, static_cast<int32_t *>(a.d_next.data()), dp,
                                          static_cast<int32_t *>(a.out_tokens.data()), dp + 1, (uint32_t)max_seq_) == GRETA_OK;
     graph_->capture_end(stream_);
     if (!ok || graph_->instantiate() != gcore::rt::GretaResult::SUCCESS) {

@@ -399,12 +399,23 @@ std::unique_ptr<WeightLoader> create_weight_loader(const std::string &path, std:
     if (!l->open(path, err)) return nullptr;
     return l;
   }
-  fail(err, "create_weight_loader: only .gguf files are read on this path");
+  struct stat st;
+  if (stat(path.c_str(), &st) == 0 && S_ISDIR(st.st_mode)) {
+    auto l = std::make_unique<SafetensorsLoader>();
+    if (!l->open(path, err)) return nullptr;
+    return l;
+  }
+  fail(err, "create_weight_loader: " + path + " is neither a .gguf file nor a model folder");
   return nullptr;
 }
 
 // ------------------------------------------------------------------ BlockScheduler::load_weights
 bool BlockScheduler::load_weights(WeightLoader &loader, std::string *err) {
+  if (config_.arch == ModelArch::HYBRID) {
+    auto *st = dynamic_cast<SafetensorsLoader *>(&loader);
+    if (!st) return fail(err, "load_weights: a hybrid model is read from a model folder (SafetensorsLoader)");
+    return load_hybrid_file(*st, err);
+  }
   auto *gguf = dynamic_cast<GGUFLoader *>(&loader);
   if (!gguf) return fail(err, "load_weights: this path reads GGUF files (GGUFLoader)");
   if (blocks_.empty()) return fail(err, "load_weights: allocate_weights first");

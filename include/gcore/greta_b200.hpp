@@ -352,6 +352,27 @@ public:
 
 namespace gcore::inference {
 
+// Layer kinds of the hybrid designs (unquantised weights, one pre-norm per layer, mixer and feed-forward side by side:
+// x += mixer(LN(x)) + ff(LN(x))).  A design is a list of layers; every size and constant is a field here.
+enum class MixerKind { WINDOW_ATTENTION, GENERAL_DELTA };
+struct MixerSpec {
+  MixerKind kind = MixerKind::WINDOW_ATTENTION;
+  uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0;  // general delta: heads and dim only
+  uint32_t taps = 0;                                    // short causal convolution on q, k, v; 0 = none
+  uint32_t window = 0, keep_first = 0;                  // window 0 = every earlier position
+  float scale = 1.0f, softcap = 0.0f;                   // softcap 0 = none
+  bool temp = false, distance_bias = false, sink = false;  // per-head vectors that the layer has
+  uint32_t rank = 0;                                    // general delta: width of the low-rank decay path
+  // Projected columns in front of the feed-forward's: attention q|k|v; delta r|k|v|gate|a (the low-rank path follows).
+  uint32_t proj_cols() const { return kind == MixerKind::GENERAL_DELTA ? 5 * heads * dim : (heads + kv_heads) * dim + kv_heads * vdim; }
+  uint32_t out_cols() const { return kind == MixerKind::GENERAL_DELTA ? heads * dim : heads * vdim; }
+};
+struct LayerSpec {
+  MixerSpec mixer;
+  uint32_t ff = 0;  // width of the gelu feed-forward; 0 = none
+};
+enum class ModelArch { LLAMA, HYBRID };
+
 struct ModelConfig {
   uint32_t dim = 4096;
   uint32_t num_heads = 32;
@@ -369,6 +390,12 @@ struct ModelConfig {
   gcore::rt::GretaDataType lm_head_type = gcore::rt::GretaDataType::FP16;
   // Tensor parallelism (Megatron style): this process holds shard tp_rank of tp_size.
   uint32_t tp_rank = 0, tp_size = 1;
+  // Which layers the scheduler runs.  HYBRID: `layers` describes them, dim is the width, rms_eps the epsilon of every norm,
+  // max_seq_len the number of learned positions, weight_type BF16 or FP32 (FP32: everything in 32-bit).
+  ModelArch arch = ModelArch::LLAMA;
+  std::string architecture;        // name in the model registry
+  std::vector<LayerSpec> layers;
+  uint32_t prefill_chunk = 2048;   // HYBRID: most positions of a prompt that run at once (longer prompts run in portions)
 
   static ModelConfig llama2_7b() { return ModelConfig{}; }
   static ModelConfig llama2_13b() {
@@ -446,6 +473,35 @@ private:
   std::unique_ptr<Impl> impl_;
 };
 
+// A model folder: config.json, whose "architecture" picks the entry of the model registry that reads it, and
+// model.safetensors (BF16, F16, F32 and I32 tensors; 8-byte little-endian header length, JSON header, data).
+class SafetensorsLoader : public WeightLoader {
+public:
+  SafetensorsLoader();
+  ~SafetensorsLoader() override;
+  bool open(const std::string &path, std::string *err) override;
+  std::vector<TensorInfo> list_tensors() const override;
+  bool load_tensor(const std::string &name, gcore::rt::cuda::Buffer &buffer, std::string *err) override;
+  bool load_tensor_fp16(const std::string &name, gcore::rt::cuda::Buffer &buffer, std::string *err) override;
+  bool load_tensor_int8(const std::string &name, gcore::rt::cuda::Buffer &buffer, gcore::rt::cuda::Buffer &scales, std::string *err) override;
+  bool load_tensor_int4(const std::string &name, gcore::rt::cuda::Buffer &buffer, gcore::rt::cuda::Buffer &scales,
+                        gcore::rt::cuda::Buffer &head_scales, std::string *err) override;
+  ModelConfig get_config() const override;
+  const TensorInfo *find(const std::string &name) const;
+  bool read_floats(const std::string &name, std::vector<float> *out, std::string *err) const;  // any float type, on the host
+
+private:
+  struct Impl;
+  std::unique_ptr<Impl> impl_;
+};
+
+// Model registry: architecture name -> reader of its config.json.  shape_of gives a tensor's shape, or null when the file
+// has no such tensor (or no file is at hand).
+using ShapeOf = std::function<const std::vector<size_t> *(const std::string &name)>;
+std::vector<std::string> registered_architectures();
+bool config_from_json(const std::string &json_text, const ShapeOf &shape_of, ModelConfig *out, std::string *err);
+
+// A folder (SafetensorsLoader) or a .gguf file (GGUFLoader).
 std::unique_ptr<WeightLoader> create_weight_loader(const std::string &path, std::string *err);
 
 struct BlockBuffers {
@@ -458,6 +514,18 @@ struct ActivationBuffers {
   gcore::rt::cuda::Buffer x, q, k, v, attn_out, mlp_gate, mlp_up, mlp_out, norm_out;
   gcore::rt::cuda::Buffer kv_cache_k, kv_cache_v;   // fp16 [L][Hkv_local][max_seq][Dh]
   gcore::rt::cuda::Buffer tokens, d_pos, d_next, attn_scratch, gemm_ws, out_tokens;
+};
+
+// One layer of a hybrid design: everything that reads the norm's output packed in one weight (w_in), both sublayers' output
+// projections side by side in another (w_out: [mixer | feed-forward] columns), and the sequences' caches or states.
+struct HybridLayerBuffers {
+  gcore::rt::cuda::Buffer norm_w, norm_b, w_in, w_out;
+  uint32_t in_rows = 0, in_ld = 0, out_cols = 0, out_ld = 0, ff_col = 0;  // ff_col: first feed-forward column of w_out
+  gcore::rt::cuda::Buffer temp, r1, r2, sink, conv;                       // attention, fp32
+  gcore::rt::cuda::Buffer w2, w2_packed, w0, a_bias, out_norm;            // general delta; w2 fp32, w2_packed for portions
+  uint32_t w2_ld = 0;
+  gcore::rt::cuda::Buffer k_cache, v_cache, history, state;               // [slots][...]
+  uint32_t ring = 0;
 };
 
 // Hook for the exchange step of tensor parallelism: in-place sum of `count`
@@ -489,6 +557,8 @@ public:
   bool execute_layer(size_t layer_idx, size_t seq_start, size_t seq_len, const int32_t *tokens, std::string *err);
   // Runs seq_len tokens starting at seq_start; logits of the last position are left in get_logits().
   bool forward(const int32_t *tokens, size_t seq_start, size_t seq_len, std::string *err);
+  // The same, with the logits of the listed rows (0 .. seq_len - 1, ascending) copied to host memory: out [n_rows][vocab].
+  bool forward_logits(const int32_t *tokens, size_t seq_start, size_t seq_len, const uint32_t *rows, size_t n_rows, float *out, std::string *err);
   int32_t sample_greedy_gpu(size_t logits_offset_bytes, std::string *err);
 
   // Decode fast path: one token per call, everything on the device.  The step (embedding of the
@@ -530,6 +600,20 @@ private:
   void invalidate_graph();
   bool build_decode_plan(std::string *err);
   bool lm_head(const float *x_row, std::string *err);
+  // Hybrid designs (hybrid_layers.cpp)
+  class TensorSource;
+  struct FileSource;
+  struct SynthSource;
+  bool init_hybrid(std::string *err);
+  bool allocate_hybrid_activations(std::string *err);
+  bool load_hybrid(TensorSource &src, std::string *err);
+  bool load_hybrid_file(SafetensorsLoader &loader, std::string *err);
+  bool load_hybrid_synthetic(uint64_t seed, std::string *err);
+  bool hybrid_embed(const int32_t *d_tokens, const greta_rows &rows, std::string *err);
+  bool hybrid_layer(size_t layer, const greta_rows &rows, std::string *err);
+  bool hybrid_logits(const float *x, uint32_t n, float *logits, std::string *err);
+  // Runs seq_len tokens in portions; after each, `after(first row, rows)` sees its hidden rows in activations_.x.
+  bool hybrid_run(const int32_t *tokens, size_t seq_start, size_t seq_len, const std::function<bool(size_t, size_t)> &after, std::string *err);
   ModelConfig config_;
   std::vector<BlockBuffers> blocks_;
   ActivationBuffers activations_;
@@ -546,6 +630,13 @@ private:
   AllReduceFn all_reduce_;
   greta_peer_exchange peer_{};            // tp == 0: not installed
   gcore::rt::cuda::Buffer x_alt_;         // second copy of the residual stream for the fused exchange
+  std::vector<HybridLayerBuffers> hybrid_;
+  struct HybridActivations {
+    gcore::rt::cuda::Buffer h, proj, cat, cat16, q, low, low16, decay, o, x_rows, logits_rows;
+    uint32_t h_ld = 0, proj_ld = 0, cat_ld = 0, low_ld = 0, low16_ld = 0, decay_ld = 0;
+  } hact_;
+  gcore::rt::cuda::Buffer pos_embd_, final_norm_b_;
+  uint32_t head_ld_ = 0;
   uint64_t weight_bytes_ = 0;
   // local (per-rank) shapes
   uint32_t heads_l_ = 0, kv_heads_l_ = 0, hidden_l_ = 0, vocab_l_ = 0;

@@ -53,7 +53,9 @@ enum {
 /* Weight formats.  Values continue gcore::rt::GretaDataType (greta_runtime.hpp:24-33,
  * FP32=0 .. FP8_E5M2=7) so that the C++ layer can pass data_type() straight through. */
 enum {
+  GRETA_FMT_F32 = 0,  /* plain floats: dense linears only */
   GRETA_FMT_F16 = 1,
+  GRETA_FMT_BF16 = 2, /* plain bf16: dense linears only */
   GRETA_FMT_REF_INT8 = 3, /* reference storage: int8 w[N][K], fp32 scale per 32 along the flat index */
   GRETA_FMT_REF_INT4 = 4, /* reference storage: uint8 w[N][K/2], elem 2j low nibble, two's complement, fp32 scales */
   GRETA_FMT_Q4_0 = 8,
@@ -418,6 +420,119 @@ GRETA_API int greta_cuda_argmax_advance(greta_stream_t stream, const float *logi
 GRETA_API int greta_cuda_argmax_advance_batch(greta_stream_t stream, const float *logits, uint32_t n, uint32_t batch,
                                               int32_t *d_next, uint32_t *d_pos, int32_t *d_out_tokens, uint32_t *d_count,
                                               uint32_t out_capacity);
+
+/* ------------------------------------------------------------------ dense linears (bf16 / fp32 weights)
+ * Operators of the hybrid decoder designs (parallel attention / recurrent mixers over unquantised weights).  The reference
+ * has no such models; its dense route is GretaCompute::gemm on FP16 buffers (src/compute/src/greta_compute_hip.cpp:148-374).
+ *
+ * A linear multiplies activation rows x[m] with a packed weight W[N x ldw] (N rows, K used columns, the rest of every row
+ * zero).  Several projections that read the same input are packed below one another; each is an output SEGMENT of the
+ * weight rows with its own bias, activation, destination and storage type, applied in the kernel's epilogue:
+ *   out[m * ld + col0 + (n - row0)]  =  act(W[n] . x[m] + bias[n - row0])     (accumulate: added to what is there, fp32)
+ * ldw is a multiple of 64 elements; W is 16-byte aligned. */
+enum { GRETA_ACT_NONE = 0, GRETA_ACT_GELU_ERF = 1, GRETA_ACT_SIGMOID = 2, GRETA_ACT_TANH = 3, GRETA_ACT_DELTA_DECAY = 4 /* exp(-exp(-1/2) sigmoid(z)) */ };
+/* Storage of an output: fp32, bf16, or a bf16 pair (hi at the element's place, lo = bf16(z - hi) pair_offset elements on). */
+enum { GRETA_OUT_F32 = 0, GRETA_OUT_BF16 = 2, GRETA_OUT_BF16_PAIR = 10 };
+#define GRETA_MAX_SEGMENTS 8
+typedef struct greta_out_segment {
+  uint32_t row0, rows;
+  int act, out_fmt, accumulate;
+  const float *bias; /* [rows] or NULL */
+  void *out;
+  uint32_t ld, col0, pair_offset;
+} greta_out_segment;
+typedef struct greta_linear {
+  int fmt;           /* GRETA_FMT_BF16 or GRETA_FMT_F32 */
+  const void *w;
+  uint32_t N, K, ldw;
+  uint32_t n_segments;
+  greta_out_segment seg[GRETA_MAX_SEGMENTS];
+} greta_linear;
+/* Few rows (1 <= M <= 8): weights streamed once for all rows, activations in fp32 whatever the weights' format.  With
+ * ln_w / ln_b the input rows are layer-normalised on the way in (K = width of the norm). x [M][ldx]. */
+GRETA_API int greta_cuda_linear_gemv(greta_stream_t stream, const greta_linear *lin, const float *x, uint32_t ldx, const float *ln_w,
+                                     const float *ln_b, float eps, uint32_t M);
+/* Many rows.  BF16: tensor cores (tcgen05), x is bf16 [M][ldx], ldx a multiple of 8 and its columns K .. ldw-1 zero where
+ * ldx >= ldw.  F32: true 32-bit products on the CUDA cores, x is fp32 [M][ldx], ldx >= ldw, zero-padded. */
+GRETA_API int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *lin, const void *x, uint32_t ldx, uint32_t M);
+/* Same contract as greta_cuda_gemm_status, for the kernels of greta_cuda_linear_gemm. */
+GRETA_API int greta_cuda_linear_gemm_status(int *code);
+/* y = (x - mean) / sqrt(var + eps) * w + b per row of D values; out fp32 or bf16 (GRETA_OUT_*), row stride ld_out. */
+GRETA_API int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w, const float *b, float eps, void *out, int out_fmt,
+                                    uint32_t M, uint32_t D, uint32_t ld_out);
+/* out[m] = table[tokens[m]] + pos_table[p], p = d_pos[m] or pos0 + m; tables in fmt BF16 or F32; ids or positions outside
+ * their table contribute zeros. */
+GRETA_API int greta_cuda_embedding_positions(greta_stream_t stream, const int32_t *tokens, const void *table, const void *pos_table, int fmt,
+                                             float *out, uint32_t M, uint32_t D, uint32_t vocab, uint32_t max_positions, const uint32_t *d_pos,
+                                             uint32_t pos0);
+/* out[i] = x[rows[i]], rows of D floats (n <= 64, row numbers on the host). */
+GRETA_API int greta_cuda_gather_rows(greta_stream_t stream, const float *x, uint32_t D, const uint32_t *rows, uint32_t n, float *out);
+
+/* Which sequence and position every activation row belongs to.  d_pos != NULL: row m is the next token of sequence
+ * slot0 + m, at position d_pos[m] (batched decode).  d_pos == NULL: rows are consecutive positions pos0 + m of sequence
+ * slot0 (a prompt or a portion of one). */
+typedef struct greta_rows {
+  uint32_t M, slot0, pos0;
+  const uint32_t *d_pos;
+} greta_rows;
+
+/* ------------------------------------------------------------------ windowed attention with kept first tokens
+ * q, k, v come as one fp32 row per token: proj[m] = [q: H*dim | k: G*dim | v: G*vdim], C values, row stride ld_proj.
+ *  1. depthwise causal convolution over time, conv [C][taps] (NULL: none); the projected rows in front of the current ones
+ *     come from `history` [slots][taps][C], position p in row p % taps;
+ *  2. q and k divided by their root mean square per head;
+ *  3. s = (q.k) scale temp_h;  s = softcap tanh(s / softcap);  s -= r1_h ln(1 + r2_h (i - j));
+ *  4. softmax over the keys j <= i with i - j < window or j < keep_first, exp(sink_h) added to the denominator.
+ * Optional parts: softcap <= 0 (none), temp / r1+r2 / sink NULL (none), window 0 (every earlier key).
+ * Caches: [slots][G][keep_first + ring][dim8] and [..][vdim8] (dim8, vdim8: rounded up to 8), F16 or F32; position p lies in
+ * row p for p < keep_first, else keep_first + (p - keep_first) % ring.  ring must be at least window - 1 + the rows of the
+ * largest portion (or the whole length). */
+typedef struct greta_window_attn {
+  uint32_t heads, kv_heads, dim, vdim, taps, window, keep_first, ring;
+  float scale, softcap, eps;
+  const float *temp, *r1, *r2, *sink; /* [heads] */
+  const float *conv, *proj;
+  uint32_t ld_proj;
+  int cache_fmt; /* GRETA_FMT_F16 or GRETA_FMT_F32; F32 also selects the accurate math functions */
+  void *k_cache, *v_cache;
+  float *history;
+} greta_window_attn;
+/* Portions: steps 1 and 2 for all rows; q -> q_out fp32 [M][H][dim8], k and v -> cache; then the history's new rows. */
+GRETA_API int greta_cuda_window_attn_prepare(greta_stream_t stream, const greta_window_attn *a, const greta_rows *rows, float *q_out);
+/* Steps 3 and 4, one CTA cluster per row and group of query heads.  q: output of _prepare, or NULL for one new token per sequence
+ * (rows->d_pos set): the kernel then runs steps 1 and 2 itself and writes the cache and history rows.
+ * out[m * ld_out + h * vdim + c], GRETA_OUT_F32 or GRETA_OUT_BF16.  max_len bounds the position of any row plus one. */
+GRETA_API int greta_cuda_window_attn(greta_stream_t stream, const greta_window_attn *a, const greta_rows *rows, const float *q, void *out,
+                                     int out_fmt, uint32_t ld_out, uint32_t max_len);
+/* The same for a portion on the tensor cores (F16 cache): tiles of query positions x tiles of keys. */
+GRETA_API int greta_cuda_window_attn_prefill(greta_stream_t stream, const greta_window_attn *a, const greta_rows *rows, const float *q,
+                                             void *out, int out_fmt, uint32_t ld_out);
+
+/* ------------------------------------------------------------------ generalised delta rule
+ * Per head, key dimension = value dimension = dim, state S [dim x dim] in fp32, zero in front of position 0:
+ *   u = k / sqrt(k.k + 1e-6);  S <- diag(w) S - (a * u)(u^T S) + k v^T;  o = S^T r
+ * with w = exp(-exp(-1/2) sigmoid(W2 t + w0)), t = low-rank activations; then per head o / rms(o), times norm and gate.
+ * r, k, v, a, gate: fp32 [M][heads*dim] at column offsets of rows of stride ld.
+ * State: [slots][heads][dim columns][dim32 rows] (dim32: rounded up to 32), value columns outermost. */
+typedef struct greta_delta_rule {
+  uint32_t heads, dim, rank, ld;
+  float eps;
+  const float *r, *k, *v, *a, *gate;
+  const float *decay;             /* [M][heads*dim], row stride ld_decay: portions */
+  uint32_t ld_decay;
+  const float *t;                 /* [M][rank], row stride ld_t: one token per sequence */
+  uint32_t ld_t;
+  const float *w2, *w0;           /* [heads*dim][rank], [heads*dim] */
+  const float *norm;              /* [heads*dim] */
+  float *state;
+} greta_delta_rule;
+GRETA_API size_t greta_cuda_delta_state_bytes(uint32_t heads, uint32_t dim); /* of one sequence */
+/* One new token per sequence (rows->d_pos set), everything from w2 to the gated output in one kernel. */
+GRETA_API int greta_cuda_delta_step(greta_stream_t stream, const greta_delta_rule *d, const greta_rows *rows, void *out, int out_fmt, uint32_t ld_out);
+/* A portion: the recurrence over its rows, o -> o_buf fp32 [M][heads*dim]; then norm and gate. */
+GRETA_API int greta_cuda_delta_scan(greta_stream_t stream, const greta_delta_rule *d, const greta_rows *rows, float *o_buf);
+GRETA_API int greta_cuda_delta_output(greta_stream_t stream, const greta_delta_rule *d, const float *o_buf, uint32_t M, void *out, int out_fmt,
+                                      uint32_t ld_out);
 
 /* ------------------------------------------------------------------ tensor-parallel exchange
  * The reference is single-GPU (hipSetDevice(0), greta_runtime_hip.cpp:153); these are new.
