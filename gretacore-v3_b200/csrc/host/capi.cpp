@@ -1,4 +1,5 @@
 // C handles onto the C++ host layer (see greta_host.h).
+#include <algorithm>
 #include <cstring>
 #include <memory>
 #include <string>
@@ -120,6 +121,57 @@ int greta_model_create_batch(const greta_model_config *c, uint32_t batch, greta_
   *out = m.release();
   return 0;
 }
+namespace {
+// Registry and file formats share one path: `loader` may be null (synthetic weights follow).
+int open_model(ModelConfig k, WeightLoader *loader, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk, greta_model_t *out) {
+  std::string err;
+  auto m = std::make_unique<Model>();
+  if (k.arch == ModelArch::HYBRID) {
+    if (fmt != GRETA_FMT_BF16 && fmt != GRETA_FMT_F32) return done(false, "model_open: a hybrid design runs in BF16 or F32");
+    k.weight_type = k.lm_head_type = fmt == GRETA_FMT_F32 ? GretaDataType::FP32 : GretaDataType::BF16;
+    if (prefill_chunk) k.prefill_chunk = prefill_chunk;
+  }
+  m->cfg = k;
+  const bool ok = m->sched.init(k, &err) && m->sched.allocate_weights(&err) && (!loader || m->sched.load_weights(*loader, &err)) &&
+                  m->sched.allocate_activations(batch, max_seq ? max_seq : k.max_seq_len, &err) && m->gen.init(k, &m->sched, &err);
+  if (!ok) return done(false, err);
+  *out = m.release();
+  return 0;
+}
+}  // namespace
+int greta_model_open(const char *path, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk, greta_model_t *out) {
+  std::string err;
+  if (!path || !out) return done(false, "model_open: null argument");
+  std::unique_ptr<WeightLoader> ld = create_weight_loader(path, &err);
+  if (!ld) return done(false, err);
+  return open_model(ld->get_config(), ld.get(), fmt, batch, max_seq, prefill_chunk, out);
+}
+int greta_model_create_from_json(const char *json, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk, greta_model_t *out) {
+  std::string err;
+  ModelConfig k;
+  if (!json || !out) return done(false, "model_create_from_json: null argument");
+  if (!config_from_json(json, nullptr, &k, &err)) return done(false, err);
+  return open_model(k, nullptr, fmt, batch, max_seq, prefill_chunk, out);
+}
+int greta_model_info(greta_model_t m, uint32_t *out5) {
+  const ModelConfig &c = M(m)->cfg;
+  out5[0] = c.dim; out5[1] = c.vocab_size; out5[2] = c.num_layers; out5[3] = (uint32_t)M(m)->sched.max_seq_len();
+  out5[4] = c.arch == ModelArch::HYBRID;
+  return 0;
+}
+const char *greta_host_architectures(void) {
+  static const std::string names = [] {
+    std::string s;
+    for (const std::string &n : registered_architectures()) s += (s.empty() ? "" : "\n") + n;
+    return s;
+  }();
+  return names.c_str();
+}
+int greta_host_check_config(const char *json) {
+  std::string err;
+  ModelConfig k;
+  return done(json && config_from_json(json, nullptr, &k, &err), err);
+}
 int greta_model_destroy(greta_model_t m) {
   delete static_cast<Model *>(m);
   return 0;
@@ -139,6 +191,22 @@ int greta_model_set_global_tensor(greta_model_t m, int which, const void *host, 
 int greta_model_forward(greta_model_t m, const int32_t *tokens, uint32_t seq_start, uint32_t seq_len) {
   std::string err;
   return done(M(m)->sched.forward(tokens, seq_start, seq_len, &err), err);
+}
+int greta_model_forward_logits(greta_model_t m, const int32_t *tokens, uint32_t seq_start, uint32_t seq_len, const uint32_t *rows, uint32_t n_rows,
+                               float *out) {
+  std::string err;
+  return done(M(m)->sched.forward_logits(tokens, seq_start, seq_len, rows, n_rows, out, &err), err);
+}
+int greta_model_forward_timed(greta_model_t m, const int32_t *tokens, uint32_t n, uint32_t reps, float *ms) {
+  std::string err;
+  auto &ctx = gcore::rt::GretaContext::instance();
+  std::unique_ptr<gcore::rt::GretaEvent> e0(ctx.create_event()), e1(ctx.create_event());
+  e0->record(M(m)->sched.stream());
+  for (uint32_t i = 0; i < reps; ++i)
+    if (!M(m)->sched.forward(tokens, 0, n, &err)) return done(false, err);
+  e1->record(M(m)->sched.stream());
+  *ms = e1->elapsed_time_since(e0.get()) / (float)std::max(1u, reps);
+  return 0;
 }
 int greta_model_get_logits(greta_model_t m, float *out, uint32_t n) {
   std::string err;
@@ -189,14 +257,14 @@ int greta_model_begin_decode_batch(greta_model_t m, const int32_t *first_tokens,
   std::string err;
   return done(M(m)->sched.begin_decode_batch(first_tokens, positions, &err), err);
 }
-int greta_model_generate_batch(greta_model_t m, const int32_t *prompts, uint32_t n_prompt, uint32_t n_new, int32_t *out) {
+int greta_model_generate_prompts(greta_model_t m, const int32_t *prompts, const uint32_t *n_prompt, uint32_t n_new, int32_t *out) {
   std::string err;
   SamplingParams sp;
   sp.greedy = true;
   sp.max_tokens = (int32_t)n_new;
   const size_t B = M(m)->sched.batch_size();
   std::vector<std::vector<int32_t>> in(B);
-  for (size_t b = 0; b < B; ++b) in[b].assign(prompts + b * n_prompt, prompts + (b + 1) * n_prompt);
+  for (size_t b = 0; b < B; prompts += n_prompt[b++]) in[b].assign(prompts, prompts + n_prompt[b]);
   std::vector<std::vector<int32_t>> ids = M(m)->gen.generate_batch(in, sp, &err);
   if (ids.size() != B) return done(false, err.empty() ? "batched generation failed" : err);
   for (size_t b = 0; b < B; ++b) {
@@ -204,6 +272,10 @@ int greta_model_generate_batch(greta_model_t m, const int32_t *prompts, uint32_t
     std::memcpy(out + b * n_new, ids[b].data(), (size_t)n_new * 4);
   }
   return 0;
+}
+int greta_model_generate_batch(greta_model_t m, const int32_t *prompts, uint32_t n_prompt, uint32_t n_new, int32_t *out) {
+  const std::vector<uint32_t> n(M(m)->sched.batch_size(), n_prompt);
+  return greta_model_generate_prompts(m, prompts, n.data(), n_new, out);
 }
 int greta_model_begin_decode(greta_model_t m, int32_t first_token, uint32_t pos) {
   std::string err;

@@ -15,6 +15,7 @@ _ROOT = os.path.dirname(_HERE)
 INCLUDE_DIR = os.path.join(_ROOT, "include")
 
 FMT_F16, FMT_REF_INT8, FMT_REF_INT4, FMT_Q4_0, FMT_Q8_0 = 1, 3, 4, 8, 9
+FMT_F32, FMT_BF16 = 0, 2                      # dense linears and hybrid designs
 PAYLOAD_BYTES = {FMT_Q4_0: 16, FMT_Q8_0: 32}
 GGUF_BLOCK_BYTES = {FMT_Q4_0: 18, FMT_Q8_0: 34}
 
@@ -70,6 +71,36 @@ def _load(libname, header):
         fn.restype, fn.argtypes = restype, argtypes
     _libs[libname] = lib
     return lib
+
+
+# Structures of the dense linears and the mixers (include/greta_cuda.h).
+ACT_NONE, ACT_GELU_ERF, ACT_SIGMOID, ACT_TANH, ACT_DELTA_DECAY = range(5)
+OUT_F32, OUT_BF16, OUT_BF16_PAIR = 0, 2, 10
+_U, _F, _P = C.c_uint32, C.c_float, C.c_void_p
+
+
+class OutSegment(C.Structure):
+    _fields_ = [("row0", _U), ("rows", _U), ("act", C.c_int), ("out_fmt", C.c_int), ("accumulate", C.c_int), ("bias", _P), ("out", _P), ("ld", _U),
+                ("col0", _U), ("pair_offset", _U)]
+
+
+class Linear(C.Structure):
+    _fields_ = [("fmt", C.c_int), ("w", _P), ("N", _U), ("K", _U), ("ldw", _U), ("n_segments", _U), ("seg", OutSegment * 8)]
+
+
+class Rows(C.Structure):
+    _fields_ = [("M", _U), ("slot0", _U), ("pos0", _U), ("d_pos", _P)]
+
+
+class WindowAttn(C.Structure):
+    _fields_ = [(n, _U) for n in ("heads", "kv_heads", "dim", "vdim", "taps", "window", "keep_first", "ring")] + \
+               [(n, _F) for n in ("scale", "softcap", "eps")] + [(n, _P) for n in ("temp", "r1", "r2", "sink", "conv", "proj")] + \
+               [("ld_proj", _U), ("cache_fmt", C.c_int), ("k_cache", _P), ("v_cache", _P), ("history", _P)]
+
+
+class DeltaRule(C.Structure):
+    _fields_ = [(n, _U) for n in ("heads", "dim", "rank", "ld")] + [("eps", _F)] + [(n, _P) for n in ("r", "k", "v", "a", "gate", "decay")] + \
+               [("ld_decay", _U), ("t", _P), ("ld_t", _U), ("w2", _P), ("w0", _P), ("norm", _P), ("state", _P)]
 
 
 def cuda():

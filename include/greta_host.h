@@ -59,6 +59,19 @@ GRETA_API int greta_model_create(const greta_model_config *cfg, greta_model_t *o
 /* The same with allocate_activations(batch, max_seq_len): `batch` sequences (1..32) that decode in step, each with its own
  * KV cache and position.  New with this build: the reference's scheduler holds one sequence. */
 GRETA_API int greta_model_create_batch(const greta_model_config *cfg, uint32_t batch, greta_model_t *out);
+/* Model folders (config.json + model.safetensors, read through the model registry) and GGUF files: create, load the weights
+ * and allocate `batch` sequences.  fmt: GRETA_FMT_BF16, or GRETA_FMT_F32 to run an unquantised design in true 32-bit (ignored
+ * for GGUF files).  max_seq 0: the model's own limit; prefill_chunk 0: the default portion size. */
+GRETA_API int greta_model_open(const char *path, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk, greta_model_t *out);
+/* The same from the text of a config.json, without weights: follow with greta_model_load_synthetic. */
+GRETA_API int greta_model_create_from_json(const char *config_json, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk,
+                                           greta_model_t *out);
+/* out5 = {width, vocabulary, layers, positions of a sequence, 1 for a hybrid design}. */
+GRETA_API int greta_model_info(greta_model_t m, uint32_t *out5);
+/* Names in the model registry, separated by newlines. */
+GRETA_API const char *greta_host_architectures(void);
+/* config.json text -> checked, without a device (shape-dependent parts take their defaults). */
+GRETA_API int greta_host_check_config(const char *config_json);
 GRETA_API int greta_model_destroy(greta_model_t m);
 GRETA_API int greta_model_load_synthetic(greta_model_t m, uint64_t seed);                 /* load_synthetic_weights */
 /* BlockScheduler::load_weights from a GGUF file whose projections are stored as Q4_0 / Q8_0: blocks go to the device as
@@ -68,6 +81,11 @@ GRETA_API int greta_model_load_gguf(greta_model_t m, const char *path);
 GRETA_API int greta_model_set_layer_tensor(greta_model_t m, uint32_t layer, int which, const void *host, size_t bytes);
 GRETA_API int greta_model_set_global_tensor(greta_model_t m, int which, const void *host, size_t bytes);
 GRETA_API int greta_model_forward(greta_model_t m, const int32_t *tokens, uint32_t seq_start, uint32_t seq_len);  /* forward */
+/* BlockScheduler::forward_logits: forward with the logits of the listed rows (ascending) -> out [n_rows][vocab]. */
+GRETA_API int greta_model_forward_logits(greta_model_t m, const int32_t *tokens, uint32_t seq_start, uint32_t seq_len, const uint32_t *rows,
+                                         uint32_t n_rows, float *out);
+/* forward() of a prompt of n tokens from position 0, `reps` times between two events; *ms = device time of one. */
+GRETA_API int greta_model_forward_timed(greta_model_t m, const int32_t *tokens, uint32_t n, uint32_t reps, float *ms);
 GRETA_API int greta_model_get_logits(greta_model_t m, float *out, uint32_t n);           /* get_logits() -> host */
 GRETA_API int greta_model_get_hidden(greta_model_t m, float *out, uint32_t row, uint32_t n); /* get_hidden_state() row -> host */
 GRETA_API int greta_model_sample_greedy(greta_model_t m, int32_t *id);                   /* sample_greedy_gpu */
@@ -85,6 +103,8 @@ GRETA_API int greta_model_begin_decode(greta_model_t m, int32_t first_token, uin
 GRETA_API int greta_model_set_sequence(greta_model_t m, uint32_t seq);
 GRETA_API int greta_model_begin_decode_batch(greta_model_t m, const int32_t *first_tokens, const uint32_t *positions);
 GRETA_API int greta_model_generate_batch(greta_model_t m, const int32_t *prompts, uint32_t n_prompt, uint32_t n_new, int32_t *out);
+/* generate_batch with prompts of their own lengths: prompt b is the next n_prompt[b] ids of `prompts`. */
+GRETA_API int greta_model_generate_prompts(greta_model_t m, const int32_t *prompts, const uint32_t *n_prompt, uint32_t n_new, int32_t *out);
 GRETA_API int greta_model_decode_step(greta_model_t m);                                   /* decode_step (asynchronous) */
 GRETA_API int greta_model_read_generated(greta_model_t m, int32_t *out, uint32_t n);      /* read_generated (synchronises); out is [batch][n] */
 /* `steps` decode_step() calls bracketed by events on the model's stream; *ms = device time. */
