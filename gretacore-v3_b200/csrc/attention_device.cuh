@@ -200,6 +200,7 @@ template <int DPL, int NW>
 __device__ __forceinline__ void attn_partial_staged(const AttnParams &p, const uint32_t k0, const uint32_t k1, const uint32_t head,
                                                     const uint32_t qi, uint8_t *stage, float &fm, float &fl, float &fo) {
   constexpr int Dh = DPL * 8, ROW = Dh * 2, TK = ATT_TILE_KEYS, NT = ATT_TILES_IN_FLIGHT, TILE_BYTES = TK * ROW * 2;
+  constexpr uint32_t PIECES = ROW / 16;  // 16-byte pieces of a K row, and as many of a V row
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int sub = lane & 7, grp = lane >> 3;
   const uint32_t kvh = head / (p.H / p.Hkv);
@@ -210,8 +211,8 @@ __device__ __forceinline__ void attn_partial_staged(const AttnParams &p, const u
     if (t < n_tiles) {
       const uint32_t key0 = k0 + t * TK, nk = min((uint32_t)TK, k1 - key0);
       uint8_t *slot = stage + (t % NT) * TILE_BYTES;
-      for (uint32_t piece = tid; piece < nk * 32; piece += NW * 32) {  // 16 K pieces and 16 V pieces of 16 bytes per key
-        const uint32_t row = piece >> 5, c = piece & 31, is_v = c >> 4, cc = c & 15;
+      for (uint32_t piece = tid; piece < nk * 2 * PIECES; piece += NW * 32) {
+        const uint32_t row = piece / (2 * PIECES), c = piece % (2 * PIECES), is_v = c / PIECES, cc = c % PIECES;
         const uint8_t *src = (is_v ? vg : kg) + (size_t)(key0 + row) * ROW + cc * 16;
         const uint32_t dst = (uint32_t)__cvta_generic_to_shared(slot + is_v * (TK * ROW) + row * ROW + cc * 16);
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");

@@ -488,7 +488,7 @@ def test_fused_exchange_wait_runs_out_and_recovers(g, tuning):
 
 
 # ----------------------------------------------------------------------------- attention
-@pytest.mark.parametrize("H,Hkv,Dh,L,max_seq", [(4, 4, 128, 1, 8), (4, 4, 128, 63, 64), (8, 2, 64, 200, 256),
+@pytest.mark.parametrize("H,Hkv,Dh,L,max_seq", [(4, 4, 128, 1, 8), (4, 4, 128, 63, 64), (8, 2, 64, 200, 256), (4, 2, 64, 2060, 2064), (6, 3, 64, 1536, 1536),
                                                 (32, 32, 128, 2049, 2304), (64, 8, 128, 777, 1024)])
 @pytest.mark.parametrize("use_dpos", [False, True])
 @pytest.mark.parametrize("cluster", ["1", "0"])
