@@ -498,6 +498,235 @@ def gemv_batch_shapes(pkg, M=16, prepared=True):
 
 
 # ----------------------------------------------------------------------------- small single-kernel cases (for ncu)
+# ----------------------------------------------------------------------------- hybrid designs
+HYBRID_SIZES = {  # width, delta heads x 64, attention heads / kv heads x head size, ff; Llama's hidden size for the same weights
+    "2048": dict(width=2048, delta_heads=32, heads=32, kv=8, dim=64, ff=8192, llama_ff=5632, layers=8),
+    "4096": dict(width=4096, delta_heads=64, heads=32, kv=8, dim=128, ff=16384, llama_ff=11008, layers=4),
+}
+HYBRID_WINDOW, HYBRID_KEEP, HYBRID_VOCAB, HYBRID_CONTEXT = 1024, 64, 32000, 2048
+
+
+def hybrid_config(z, max_positions):
+    attn = {"type": "attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+            "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "conv": 4, "scale": z["dim"] ** -0.5, "softcap": 30.0,
+                      "mask": {"size": HYBRID_WINDOW, "keep_first": HYBRID_KEEP}}}
+    delta = {"type": "general_delta", "mlp": {"kind": "dense", "ff": z["ff"]}, "mixer": {"heads": z["delta_heads"], "dim": 64, "rank": 64}}
+    return {"architecture": "Bidonex", "width": z["width"], "vocab": HYBRID_VOCAB, "max_positions": max_positions, "norm": {"eps": 1e-6},
+            "layers": [delta if i % 2 == 0 else attn for i in range(z["layers"])]}
+
+
+def hybrid_models(pkg):
+    """Prefill and decode throughput of the hybrid design beside the Llama-shaped model of the same width, layers and weight
+    count (Q8_0).  Device times (events on the model's stream); a model's weights exceed L2, so nothing is served from it
+    between steps.  One JSON line per model and size."""
+    g = pkg.ffi
+    lib = g.cuda()
+    peak, peak_src = measured_peak_gbs()
+    for name, z in HYBRID_SIZES.items():
+        for design in ("hybrid bf16", "llama q8_0"):
+            res = {}
+            for batch in (1, 8, 16):
+                if design == "hybrid bf16":
+                    m = pkg.model.Model.from_config(hybrid_config(z, 2560), batch=batch)
+                else:
+                    m = pkg.model.Model(dict(dim=z["width"], num_heads=z["heads"], num_heads_kv=z["kv"], num_layers=z["layers"], vocab=HYBRID_VOCAB,
+                                             hidden_dim=z["llama_ff"], head_dim=z["dim"], max_seq=2560, rope_base=10000.0, rms_eps=1e-5),
+                                        weight_fmt=g.FMT_Q8_0, batch=batch)
+                m.load_synthetic(1)
+                toks = pkg.model.synth_tokens(1, HYBRID_CONTEXT, HYBRID_VOCAB)
+                sampler = ClockSampler(0)
+                sampler.start()
+                t0 = time.time()
+                if batch == 1:
+                    for T in (512, 2048):
+                        m.forward_timed(toks[:T], 3)
+                        res[f"prefill_{T}_tok_per_s"] = round(T / min(m.forward_timed(toks[:T], 5) for _ in range(3)) * 1e3)
+                for b in range(batch):
+                    if batch > 1:
+                        m.set_sequence(b)
+                    m.forward(toks, 0)
+                m.begin_decode(1 if batch == 1 else [1] * batch, HYBRID_CONTEXT)
+                m.decode_timed(16)
+                n0 = lib.greta_cuda_launch_count()
+                ms = m.decode_timed(128) / 128
+                res[f"decode_b{batch}_tok_per_s"] = round(batch / ms * 1e3)
+                res[f"decode_b{batch}_us_per_step"] = round(ms * 1e3, 1)
+                res[f"decode_b{batch}_weight_stream_frac_of_peak"] = round(m.weight_bytes() / ms / 1e6 / peak, 3)
+                res["launches_per_step"] = (lib.greta_cuda_launch_count() - n0) / 128
+                res["clocks"] = sampler.stop(t0, time.time())
+                wb = m.weight_bytes()
+                m.close()
+            print(json.dumps({"case": "hybrid_models", "size": name, "design": design, "layers": z["layers"], "weight_bytes": wb, **res,
+                              "window": HYBRID_WINDOW, "context": HYBRID_CONTEXT, "peak_source": f"of {peak_src}"}), flush=True)
+
+
+def hybrid_kernels(pkg, only=None):
+    """The hybrid design's kernels and the like kernels of the Llama-shaped model, one by one, with the roofline each is held
+    against: HBM bytes, tensor-core FLOPs (bf16), or - the delta-rule scan - fp32 FMA throughput.  Buffers rotate beyond L2."""
+    import ctypes as C
+    g = pkg.ffi
+    lib = g.cuda()
+    peak, _ = measured_peak_gbs()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tc = float(json.load(f)["bf16_tflops"])
+    except Exception:
+        tc = 1590.0
+    fma = 148 * 128 * 2 * 1.965e9 / 1e12                     # TFLOP/s of 32-bit FMAs at the maximum clock
+    stream = C.c_void_p()
+    g.check(lib.greta_cuda_stream_create(C.byref(stream)))
+    e0, e1 = C.c_void_p(), C.c_void_p()
+    lib.greta_cuda_event_create(C.byref(e0))
+    lib.greta_cuda_event_create(C.byref(e1))
+    rng = np.random.default_rng(0)
+
+    def buf(nbytes, kind="zero"):
+        b = g.DeviceBuffer(int(nbytes), zero=True)
+        if kind == "bf16":
+            block = (np.abs(rng.normal(0, 0.02, 1 << 20)).astype(np.float32).view(np.uint32) >> 16).astype(np.uint16)
+        elif kind == "f32":
+            block = rng.normal(0, 0.5, 1 << 20).astype(np.float32)
+        else:
+            return b
+        raw = block.view(np.uint8)
+        for at in range(0, int(nbytes), raw.size):
+            b.upload(raw[:min(raw.size, int(nbytes) - at)], at)
+        return b
+
+    def report(name, size, launches, copies, hbm=0.0, tensor=0.0, fp32=0.0):
+        """launches(i) enqueues copy i; hbm bytes, tensor and fp32 flops of one launch."""
+        if only and only not in name:
+            return
+        for i in range(copies):
+            launches(i)
+        g.check(lib.greta_cuda_stream_synchronize(stream))
+        graph, ex = C.c_void_p(), C.c_void_p()
+        reps = max(1, 24 // copies)
+        g.check(lib.greta_cuda_graph_capture_begin(stream))
+        for _ in range(reps):
+            for i in range(copies):
+                launches(i)
+        g.check(lib.greta_cuda_graph_capture_end(stream, C.byref(graph)))
+        g.check(lib.greta_cuda_graph_instantiate(graph, C.byref(ex)))
+        best = 1e30
+        for it in range(6):
+            lib.greta_cuda_event_record(e0, stream)
+            lib.greta_cuda_graph_launch(ex, stream)
+            lib.greta_cuda_event_record(e1, stream)
+            lib.greta_cuda_event_synchronize(e1)
+            ms = C.c_float()
+            lib.greta_cuda_event_elapsed_ms(e0, e1, C.byref(ms))
+            if it >= 3:
+                best = min(best, ms.value)
+        lib.greta_cuda_graph_exec_destroy(ex)
+        lib.greta_cuda_graph_destroy(graph)
+        us = best * 1e3 / (reps * copies)
+        roof = {"hbm": hbm / peak / 1e3, "tensor": tensor / tc / 1e6, "fp32": fp32 / fma / 1e6}
+        bound = max(roof, key=roof.get)
+        print(json.dumps({"case": "hybrid_kernels", "size": size, "kernel": name, "us": round(us, 2), "bound": bound,
+                          "roofline_us": round(roof[bound], 2), "frac": round(roof[bound] / us, 3)}), flush=True)
+
+    def dense(N, K, segs):
+        ld = (K + 63) // 64 * 64
+        w = buf(N * ld * 2, "bf16")
+        lin = g.Linear(g.FMT_BF16, w.ptr, N, K, ld, len(segs))
+        row = 0
+        for i, (n, act, fmt, out, ldo, acc) in enumerate(segs):
+            lin.seg[i] = g.OutSegment(row, n, act, fmt, acc, None, out.ptr, ldo, 0, 0)
+            row += n
+        return w, lin
+
+    for size, z in HYBRID_SIZES.items():
+        D, F, H, G, Dh = z["width"], z["ff"], z["heads"], z["kv"], z["dim"]
+        HD, LF, T = z["delta_heads"] * 64, z["llama_ff"], 2048
+        C_att = (H + 2 * G) * Dh
+        N_in, K_out = 5 * HD + 64 + F, HD + F
+        x, xb = buf(T * max(K_out, D) * 4, "f32"), buf(T * K_out * 2, "bf16")
+        proj, cat, o = buf(T * (5 * HD + C_att) * 4, "f32"), buf(T * K_out * 4), buf(T * max(HD, D) * 4)
+        ln = buf(D * 4, "f32")
+        copies = max(2, int(4e8 // (N_in * D * 2)))
+        ins = [dense(N_in, D, [(5 * HD + 64, 0, g.OUT_F32, proj, 5 * HD + 64, 0), (F, g.ACT_GELU_ERF, g.OUT_BF16, cat, F, 0)]) for _ in range(copies)]
+        ins32 = [g.Linear.from_buffer_copy(l) for _, l in ins]
+        for l in ins32:
+            l.seg[1].out_fmt = g.OUT_F32
+        outs = [dense(D, K_out, [(D, 0, g.OUT_F32, o, D, 1)]) for _ in range(copies)]
+        for M in (1, 8):
+            report(f"linear_gemv in M={M}", size, lambda i: g.check(lib.greta_cuda_linear_gemv(stream, C.byref(ins32[i]), x.ptr, D, ln.ptr, ln.ptr, 1e-6, M)),
+                   copies, hbm=N_in * D * 2)
+            report(f"linear_gemv out M={M}", size,
+                   lambda i: g.check(lib.greta_cuda_linear_gemv(stream, C.byref(outs[i][1]), x.ptr, K_out, None, None, 0.0, M)), copies, hbm=D * K_out * 2)
+        for M in (16, 128, 512, T):
+            report(f"linear_gemm in T={M}", size, lambda i: g.check(lib.greta_cuda_linear_gemm(stream, C.byref(ins[i][1]), xb.ptr, D, M)), copies,
+                   hbm=N_in * D * 2 + M * (D * 2 + (N_in - F) * 4 + F * 2), tensor=2.0 * M * N_in * D)
+            report(f"linear_gemm out T={M}", size, lambda i: g.check(lib.greta_cuda_linear_gemm(stream, C.byref(outs[i][1]), xb.ptr, K_out, M)), copies,
+                   hbm=D * K_out * 2 + M * (K_out * 2 + D * 8), tensor=2.0 * M * K_out * D)
+        del ins, ins32, outs
+        # Llama's: quantised GEMV (ffn front, residual), GEMM
+        q = [(buf(2 * LF * D), buf(2 * LF * D // 16)) for _ in range(copies * 2)]
+        y = buf(T * LF * 4)
+        report("llama ffn_front q8_0 M=1", size, lambda i: g.check(lib.greta_cuda_fused_ffn_front(
+            stream, g.FMT_Q8_0, x.ptr, ln.ptr, 1e-5, q[i][0].ptr, q[i][1].ptr, q[i][0].ptr + LF * D, q[i][1].ptr + LF * D // 16, y.ptr, D, LF)),
+            copies * 2, hbm=2 * LF * D * 34 / 32)
+        report("llama gemv_residual q8_0 M=1", size, lambda i: g.check(lib.greta_cuda_gemv_residual(
+            stream, g.FMT_Q8_0, x.ptr, q[i][0].ptr, q[i][1].ptr, o.ptr, o.ptr, D, LF)), copies * 2, hbm=LF * D * 34 / 32)
+        ws = buf(lib.greta_cuda_gemv_batch_workspace_bytes(32, max(D, LF)))
+        for M in (8, 16):
+            report(f"llama ffn_front q8_0 M={M}", size, lambda i: g.check(lib.greta_cuda_fused_ffn_front_batch(
+                stream, g.FMT_Q8_0, x.ptr, ln.ptr, 1e-5, q[i][0].ptr, q[i][1].ptr, q[i][0].ptr + LF * D, q[i][1].ptr + LF * D // 16, y.ptr, M, D, LF, ws.ptr)),
+                copies * 2, hbm=2 * LF * D * 34 / 32)
+        gws = buf(lib.greta_cuda_gemm_workspace_bytes(T, max(D, LF)))
+        for M in (128, 512, T):
+            report(f"llama gemm q8_0 T={M}", size, lambda i: g.check(lib.greta_cuda_gemm(stream, g.FMT_Q8_0, xb.ptr, 1, q[i][0].ptr, q[i][1].ptr, y.ptr, 0, M, LF, D,
+                                                                                      gws.ptr)), copies * 2, hbm=LF * D * 34 / 32 + M * (D * 2 + LF * 4), tensor=2.0 * M * LF * D)
+        del q
+        # attention
+        p = [buf(H * 4, "f32") for _ in range(4)]
+        conv = buf(C_att * 4 * 4, "f32")
+        rows_c = HYBRID_KEEP + HYBRID_WINDOW - 1 + T
+        n_copy = max(2, int(2e8 // (rows_c * G * Dh * 4)))
+        caches = [(buf(rows_c * G * Dh * 2), buf(rows_c * G * Dh * 2), buf(4 * C_att * 4)) for _ in range(n_copy)]
+        att = [g.WindowAttn(H, G, Dh, Dh, 4, HYBRID_WINDOW, HYBRID_KEEP, rows_c - HYBRID_KEEP, Dh ** -0.5, 30.0, 1e-6, *[v.ptr for v in p], conv.ptr, proj.ptr,
+                            C_att, g.FMT_F16, k.ptr, v.ptr, h.ptr) for k, v, h in caches]
+        dpos = g.DeviceBuffer.from_numpy(np.full(1, HYBRID_CONTEXT, np.uint32))
+        one, many = g.Rows(1, 0, 0, dpos.ptr), g.Rows(T, 0, 0, None)
+        keys = HYBRID_WINDOW + HYBRID_KEEP
+        report("window_rows decode", size, lambda i: g.check(lib.greta_cuda_window_attn(stream, C.byref(att[i]), C.byref(one), None, cat.ptr, 0, H * Dh, 2560)),
+               n_copy, hbm=keys * G * Dh * 4)
+        qb = buf(T * H * Dh * 4, "f32")
+        report("conv_norm + history T=2048", size, lambda i: g.check(lib.greta_cuda_window_attn_prepare(stream, C.byref(att[i]), C.byref(many), qb.ptr)), n_copy,
+               hbm=T * (C_att * 4 + H * Dh * 4 + G * Dh * 4))
+        pairs = sum(min(i + 1, HYBRID_WINDOW + min(HYBRID_KEEP, max(0, i + 1 - HYBRID_WINDOW))) for i in range(T))
+        report("window_mma T=2048", size, lambda i: g.check(lib.greta_cuda_window_attn_prefill(stream, C.byref(att[i]), C.byref(many), qb.ptr, cat.ptr,
+                                                                                             g.OUT_BF16, H * Dh)), n_copy, tensor=4.0 * pairs * H * Dh,
+               hbm=T * H * Dh * 6)
+        sc = buf(lib.greta_cuda_attn_decode_scratch_bytes(H, Dh))
+        kpos = g.DeviceBuffer.from_numpy(np.full(1, keys - 1, np.uint32))
+        report("llama attn_decode", size, lambda i: g.check(lib.greta_cuda_attn_decode(stream, qb.ptr, caches[i][0].ptr, caches[i][1].ptr, cat.ptr, kpos.ptr, 0, H, G,
+                                                                                    Dh, rows_c, Dh ** -0.5, sc.ptr, sc.nbytes)), n_copy, hbm=keys * G * Dh * 4)
+        report("llama attn_prefill T=2048", size, lambda i: g.check(lib.greta_cuda_attn_prefill(stream, qb.ptr, caches[i][0].ptr, caches[i][1].ptr, cat.ptr, T, 0, H,
+                                                                                               G, Dh, rows_c, Dh ** -0.5)), n_copy, tensor=4.0 * H * Dh * T * (T + 1) / 2,
+               hbm=T * H * Dh * 8)
+        # delta rule
+        HE = z["delta_heads"]
+        states = [buf(lib.greta_cuda_delta_state_bytes(HE, 64)) for _ in range(max(2, int(2e8 // (HE * 64 * 64 * 4))))]
+        w2, low = buf(HD * 64 * 4, "f32"), buf(T * 64 * 4, "f32")
+        ds = []
+        for st in states:
+            at = lambda i: proj.ptr + 4 * i * HD
+            ds.append(g.DeltaRule(HE, 64, 64, 5 * HD, 1e-6, at(0), at(1), at(2), at(3), at(4), qb.ptr if HD <= H * Dh else proj.ptr, HD, low.ptr, 64, w2.ptr,
+                                  w2.ptr, w2.ptr, st.ptr))
+        report("delta_step", size, lambda i: g.check(lib.greta_cuda_delta_step(stream, C.byref(ds[i]), C.byref(one), cat.ptr, 0, HD)), len(ds),
+               hbm=HE * 64 * 64 * 8 + HD * 64 * 4)
+        report("delta_scan T=2048", size, lambda i: g.check(lib.greta_cuda_delta_scan(stream, C.byref(ds[i]), C.byref(many), o.ptr)), 2, hbm=T * HD * 4 * 6,
+               fp32=2.0 * T * HE * 64 * 64 * 5)
+        report("delta_output T=2048", size, lambda i: g.check(lib.greta_cuda_delta_output(stream, C.byref(ds[i]), o.ptr, T, cat.ptr, g.OUT_BF16, HD)), 2,
+               hbm=T * HD * (4 + 4 + 2))
+        xs = [buf(T * D * 4, "f32") for _ in range(8)]
+        report("layer_norm T=2048", size, lambda i: g.check(lib.greta_cuda_layer_norm(stream, xs[i].ptr, ln.ptr, ln.ptr, 1e-6, cat.ptr, g.OUT_BF16, T, D, D)), 8,
+               hbm=T * D * 6)
+        del caches, att, states, ds, xs
+
+
 def run_case(pkg, name):
     """A few launches of one kernel on a small case whose data is larger than L2, for profiler captures
     (`ncu -k regex:<kernel> ... python bench.py --case <name>`).  Prints nothing but 'ok'."""
@@ -608,7 +837,8 @@ def main():
     ap.add_argument("--exchange", choices=["fused", "nccl"], default="fused",
                     help="tensor-parallel exchange of the decode step: fused into the GEMV kernels over peer memory, or NCCL all-reduce")
     ap.add_argument("--case", default=None, help="run a small single-kernel case (gemv_swiglu, gemv_plain, gemm_c2, gemm_small, attn_decode, decode_step, gemv_batch, attn_batch) and exit; "
-                         "gemv_shapes prints the GEMV bandwidth of every projection shape")
+                         "gemv_shapes prints the GEMV bandwidth of every projection shape; hybrid_models and hybrid_kernels (or "
+                         "hybrid_kernels:<part of a name>) measure the hybrid design beside the Llama-shaped model")
     args = ap.parse_args()
     pkg = load_pkg()
     ranks = pkg.rendezvous.Ranks()
@@ -622,6 +852,14 @@ def main():
     if args.case == "gemv_batch_shapes":
         pkg.ffi.require_device()
         gemv_batch_shapes(pkg, args.batch or 16)
+        return
+    if args.case == "hybrid_models":
+        pkg.ffi.require_device()
+        hybrid_models(pkg)
+        return
+    if args.case and args.case.startswith("hybrid_kernels"):
+        pkg.ffi.require_device()
+        hybrid_kernels(pkg, args.case.partition(":")[2] or None)
         return
     if args.case:
         run_case(pkg, args.case)
