@@ -3,8 +3,13 @@
 // The columns of S (one per value channel) do not mix: column j only needs the scalar c_j = k^T S_j of the old state,
 //   S_j <- w * S_j + k v_j - ak c_j,   ak = a * k / (k.k + 1e-6),   o_j = r^T S_j,
 // so eight lanes hold one column in registers (row i * 32 + lane8 * 4 + e in register 4 i + e) and a step is two dot
-// products over eight lanes and one update.  The scan computes o_t and the next token's c together from the new state:
-// one reduction per token.  Rows past dim are padding: every vector is zero there, so they stay zero.
+// products over eight lanes and one update.  Rows past dim are padding: every vector is zero there, so they stay zero.
+//
+// The scan looks one token ahead so that no step waits for a reduction it has just started: with S' the state before token t,
+//   k'^T S_j = (k' * w)^T S'_j + (k'.k) v_j - (k'.ak) c_j      (k' the next token's key)
+// and the first term needs only S', one step earlier than the state it belongs to.  Producer warps stage the tokens' vectors
+// (cp.async), derive ak, k' * w and the two scalars, and write the outputs back, one chunk ahead of and behind the warps that
+// hold the state.
 #include <algorithm>
 
 #include "dense_device.cuh"
@@ -116,145 +121,282 @@ __device__ __forceinline__ void cp4(void *dst, const void *src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// The recurrence over a portion: grid (heads, column groups).  A CTA keeps COLS columns of one head in registers (NC per
-// group of eight lanes) and walks the tokens in chunks of TC staged by cp.async, two chunks in shared memory.
-template <int RB>
+typedef unsigned long long f32x2;  // two floats for the packed 32-bit arithmetic
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+  return d;
+}
+__device__ __forceinline__ float sum_halves(f32x2 v) {
+  float a, b;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+  return a + b;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ ulonglong2 lds2(const float *p) { return *reinterpret_cast<const ulonglong2 *>(p); }
+
+// The recurrence over a portion: grid (heads, column groups).  A CTA keeps 32 columns of one head in the registers of its
+// first warps, NC columns per group of eight lanes, and walks the tokens in chunks of TC; three chunk buffers rotate.
+template <int RB, int NC>
 struct ScanCfg {
   static constexpr int DP = RB * 32, COLS = 32;
   static constexpr int TC = RB <= 4 ? 16 : 8;
-  static constexpr int ROW = 4 * DP + COLS;  // floats of a staged token: w, k, ak, r, v
-  static constexpr size_t SMEM = (size_t)(2 * TC * ROW + TC * COLS) * 4;
+  static constexpr int ROW = 5 * DP + COLS + 4;   // floats of a staged token: w, k, ak, r, k' * w, v, {k'.k, k'.ak}
+  static constexpr int BUF = (TC + 1) * ROW;      // one more token: its key is the last one's k'
+  static constexpr int CW = COLS / (4 * NC), PW = 4, THREADS = (CW + PW) * 32;
+  static constexpr size_t SMEM = (size_t)(3 * BUF + 2 * TC * COLS) * 4;
+  static_assert(SMEM <= 232448, "chunk buffers exceed shared memory");
 };
 template <int RB, int NC>
-__global__ void __launch_bounds__(ScanCfg<RB>::COLS / NC * 8) delta_scan_kernel(const __grid_constant__ DeltaArgs a, float *__restrict__ o_buf, int vec) {
-  using C = ScanCfg<RB>;
-  constexpr int DP = C::DP, TC = C::TC, ROW = C::ROW, COLS = C::COLS, THREADS = COLS / NC * 8, NW = THREADS / 32;
+__global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(const __grid_constant__ DeltaArgs a, float *__restrict__ o_buf, int vec) {
+  using C = ScanCfg<RB, NC>;
+  constexpr int DP = C::DP, TC = C::TC, ROW = C::ROW, COLS = C::COLS, BUF = C::BUF;
   extern __shared__ __align__(16) float sm[];
-  float *so = sm + 2 * TC * ROW;  // [TC][COLS]
+  float *so = sm + 3 * BUF;  // [2][TC][COLS]
   const greta_delta_rule &d = a.d;
   const uint32_t h = blockIdx.x, c0 = blockIdx.y * COLS, D = d.dim, T = a.rows.M;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7, grp = threadIdx.x >> 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
+  const bool producer = warp >= C::CW;
+  const int pw = warp - C::CW;
+  const uint32_t vcols = min((uint32_t)COLS, D - c0), chunks = (T + TC - 1) / TC;
   float *state = d.state + ((size_t)a.rows.slot0 * d.heads + h) * D * DP;
-  for (int i = threadIdx.x; i < 2 * TC * ROW; i += THREADS) sm[i] = 0.f;
+  for (int i = threadIdx.x; i < 3 * BUF; i += C::THREADS) sm[i] = 0.f;
   pdl_launch_dependents();
   pdl_wait();
   __syncthreads();
-  const uint32_t vcols = min((uint32_t)COLS, D - c0);
-  auto stage = [&](uint32_t t0, int buf) {
-    const uint32_t n = t0 < T ? min((uint32_t)TC, T - t0) : 0;
-    float *b = sm + buf * TC * ROW;
-    const uint32_t unit = vec ? 4 : 1, per = D / unit, vper = vec ? vcols / 4 : vcols, tok = 4 * per + vper;
-    for (uint32_t i = threadIdx.x; i < n * tok; i += THREADS) {
-      const uint32_t t = i / tok, j = i % tok, which = j < 4 * per ? j / per : 4, e = (which < 4 ? j % per : j - 4 * per) * unit;
-      const size_t m = t0 + t, at = m * d.ld + (size_t)h * D;
-      const float *src = which == 0 ? d.decay + m * d.ld_decay + (size_t)h * D + e
-                         : which == 1 ? d.k + at + e
-                         : which == 2 ? d.a + at + e
-                         : which == 3 ? d.r + at + e
-                                      : d.v + at + c0 + e;
-      float *dst = b + t * ROW + which * DP + e;
-      if (vec)
-        cp16(dst, src);
-      else
-        cp4(dst, src);
+
+  auto stage = [&](uint32_t c) {  // producer warps: the chunk's tokens and one more
+    if (c < chunks) {
+      const uint32_t t0 = c * TC, n = min((uint32_t)TC + 1, T - t0);
+      float *b = sm + (c % 3) * BUF;
+      const uint32_t unit = vec ? 4 : 1, per = D / unit, vper = vec ? vcols / 4 : vcols, tok = 4 * per + vper;
+      for (uint32_t t = pw; t < n; t += C::PW) {
+        const size_t m = t0 + t, at = m * d.ld + (size_t)h * D;
+        float *dst = b + t * ROW;
+        for (uint32_t j = lane; j < tok; j += 32) {
+          const uint32_t which = j < 4 * per ? j / per : 4, e = (j - which * per) * unit;
+          const float *src = which == 0 ? d.decay + m * d.ld_decay + (size_t)h * D
+                             : which == 1 ? d.k + at
+                             : which == 2 ? d.a + at
+                             : which == 3 ? d.r + at
+                                          : d.v + at + c0;
+          float *to = dst + (which < 4 ? which * DP : 5 * DP) + e;
+          if (vec)
+            cp16(to, src + e);
+          else
+            cp4(to, src + e);
+        }
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float4 s[NC][RB];
-  bool on[NC];
-#pragma unroll
-  for (int c = 0; c < NC; ++c) {
-    const uint32_t col = c0 + grp * NC + c;
-    on[c] = col < D;
-#pragma unroll
-    for (int i = 0; i < RB; ++i)
-      s[c][i] = on[c] && a.rows.pos0 ? *reinterpret_cast<const float4 *>(state + (size_t)col * DP + i * 32 + l8 * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  stage(0, 0);
-  for (uint32_t t0 = 0, buf = 0; t0 < T; t0 += TC, buf ^= 1) {
-    stage(t0 + TC, buf ^ 1);
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    float *b = sm + buf * TC * ROW;
-    const int n = (int)min((uint32_t)TC, T - t0);
-    for (int t = warp; t < n; t += NW) {  // ak = a k / (k.k + 1e-6)
+  auto prepare = [&](uint32_t c) {  // producer warps, once the chunk has landed: ak, k' * w, k'.k, k'.ak
+    if (c >= chunks) return;
+    const int n = (int)min((uint32_t)TC, T - c * TC);
+    float *b = sm + (c % 3) * BUF;
+    for (int t = pw; t < n; t += C::PW) {
       float *row = b + t * ROW;
-      float kk = 0.f;
-#pragma unroll
-      for (int i = 0; i < RB; ++i) kk = fmaf(row[DP + i * 32 + lane], row[DP + i * 32 + lane], kk);
-      const float inv2 = 1.f / (warp_sum(kk) + 1e-6f);
-#pragma unroll
-      for (int i = 0; i < RB; ++i) row[2 * DP + i * 32 + lane] *= row[DP + i * 32 + lane] * inv2;
-    }
-    __syncthreads();
-    float4 k[RB];
-    float nc[NC];
-#pragma unroll
-    for (int i = 0; i < RB; ++i) k[i] = lds4(b + DP + i * 32 + l8 * 4);
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      float x = 0.f;
-#pragma unroll
-      for (int i = 0; i < RB; ++i) x = dot4(k[i], s[c][i], x);
-      nc[c] = -sum8(x);
-    }
-    for (int t = 0; t < n; ++t) {
-      const float *row = b + t * ROW;
-      float v[NC], o[NC], x[NC];
-#pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        v[c] = row[4 * DP + grp * NC + c];
-        o[c] = x[c] = 0.f;
-      }
-      const float *next = t + 1 < n ? row + ROW : row;  // the last token's look-ahead is not used
+      float k[RB], kk = 0.f, next_k = 0.f, next_ak = 0.f;
 #pragma unroll
       for (int i = 0; i < RB; ++i) {
-        const int at = i * 32 + l8 * 4;
-        const float4 w = lds4(row + at), ak = lds4(row + 2 * DP + at), r = lds4(row + 3 * DP + at), kn = lds4(next + DP + at);
+        k[i] = row[DP + i * 32 + lane];
+        kk = fmaf(k[i], k[i], kk);
+      }
+      const float inv2 = 1.f / (warp_sum(kk) + 1e-6f);
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        const int e = i * 32 + lane;
+        const float k1 = row[ROW + DP + e], ak = row[2 * DP + e] * k[i] * inv2;
+        row[2 * DP + e] = ak;
+        row[4 * DP + e] = k1 * row[e];
+        next_k = fmaf(k1, k[i], next_k);
+        next_ak = fmaf(k1, ak, next_ak);
+      }
+      next_k = warp_sum(next_k);
+      next_ak = warp_sum(next_ak);
+      if (lane == 0) {
+        row[5 * DP + COLS] = next_k;
+        row[5 * DP + COLS + 1] = next_ak;
+      }
+    }
+  };
+  auto landed = [&]() {  // the chunk before the last one staged is complete for every producer
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    asm volatile("bar.sync 1, %0;" ::"n"(C::PW * 32) : "memory");
+  };
+  auto write_back = [&](uint32_t c) {
+    const uint32_t n = min((uint32_t)TC, T - c * TC);
+    const float *src = so + (c & 1) * TC * COLS;
+    for (uint32_t t = pw; t < n; t += C::PW)
+      if (lane < (int)vcols) o_buf[((size_t)(c * TC + t) * d.heads + h) * D + c0 + lane] = src[t * COLS + lane];
+  };
+
+  const int grp = threadIdx.x >> 3;  // state warps: columns c0 + grp * NC ..
+  f32x2 s[NC][2 * RB];
+  float nc[NC];
+  if (producer) {
+    stage(0);
+    stage(1);
+    landed();
+    prepare(0);
+  } else {
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const uint32_t col = c0 + grp * NC + c;
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        const bool on = col < D && a.rows.pos0;
+        const ulonglong2 v = on ? *reinterpret_cast<const ulonglong2 *>(state + (size_t)col * DP + i * 32 + l8 * 4) : make_ulonglong2(0ull, 0ull);
+        s[c][2 * i] = v.x;
+        s[c][2 * i + 1] = v.y;
+      }
+    }
+  }
+  __syncthreads();
+  if (!producer) {  // the first token's c
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      f32x2 x = 0ull;
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        const ulonglong2 k = lds2(sm + DP + i * 32 + l8 * 4);
+        x = fma2(k.x, s[c][2 * i], x);
+        x = fma2(k.y, s[c][2 * i + 1], x);
+      }
+      nc[c] = -sum8(sum_halves(x));
+    }
+  }
+  for (uint32_t ch = 0; ch < chunks; ++ch) {
+    if (producer) {
+      stage(ch + 2);
+      landed();
+      prepare(ch + 1);
+      if (ch) write_back(ch - 1);
+    } else {
+      const float *b = sm + (ch % 3) * BUF;
+      float *out = so + (ch & 1) * TC * COLS;
+      const int n = (int)min((uint32_t)TC, T - ch * TC);
+#pragma unroll 2
+      for (int t = 0; t < n; ++t) {
+        const float *row = b + t * ROW;
+        f32x2 x[NC], o[NC], v2[NC], nc2[NC];
+        float v[NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-          update4(s[c][i], w, k[i], ak, v[c], nc[c]);
-          o[c] = dot4(r, s[c][i], o[c]);
-          x[c] = dot4(kn, s[c][i], x[c]);
+          v[c] = row[5 * DP + grp * NC + c];
+          v2[c] = pack2(v[c], v[c]);
+          nc2[c] = pack2(nc[c], nc[c]);
+          x[c] = o[c] = 0ull;
         }
-        k[i] = kn;
-      }
 #pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        o[c] = sum8(o[c]);
-        nc[c] = -sum8(x[c]);
-        if (l8 == 0) so[t * COLS + grp * NC + c] = o[c];
+        for (int i = 0; i < RB; ++i) {
+          const ulonglong2 kw = lds2(row + 4 * DP + i * 32 + l8 * 4);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            x[c] = fma2(kw.x, s[c][2 * i], x[c]);
+            x[c] = fma2(kw.y, s[c][2 * i + 1], x[c]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < RB; ++i) {
+          const int at = i * 32 + l8 * 4;
+          const ulonglong2 w = lds2(row + at), k = lds2(row + DP + at), ak = lds2(row + 2 * DP + at), r = lds2(row + 3 * DP + at);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            s[c][2 * i] = fma2(w.x, s[c][2 * i], fma2(k.x, v2[c], mul2(ak.x, nc2[c])));
+            s[c][2 * i + 1] = fma2(w.y, s[c][2 * i + 1], fma2(k.y, v2[c], mul2(ak.y, nc2[c])));
+            o[c] = fma2(r.x, s[c][2 * i], o[c]);
+            o[c] = fma2(r.y, s[c][2 * i + 1], o[c]);
+          }
+        }
+        const float2 nx = *reinterpret_cast<const float2 *>(row + 5 * DP + COLS);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          const float ahead = sum8(sum_halves(x[c]));
+          nc[c] = -fmaf(nx.y, nc[c], fmaf(nx.x, v[c], ahead));
+          const float y = sum8(sum_halves(o[c]));
+          if (l8 == c) out[t * COLS + grp * NC + c] = y;
+        }
       }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < n * COLS; i += THREADS) {
-      const uint32_t t = i / COLS, c = i % COLS;
-      if (c < vcols) o_buf[((size_t)(t0 + t) * d.heads + h) * D + c0 + c] = so[i];
+  }
+  if (producer) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    write_back(chunks - 1);
+  } else {
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const uint32_t col = c0 + grp * NC + c;
+#pragma unroll
+      for (int i = 0; i < RB; ++i)
+        if (col < D) *reinterpret_cast<ulonglong2 *>(state + (size_t)col * DP + i * 32 + l8 * 4) = make_ulonglong2(s[c][2 * i], s[c][2 * i + 1]);
     }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-#pragma unroll
-  for (int c = 0; c < NC; ++c)
-#pragma unroll
-    for (int i = 0; i < RB; ++i)
-      if (on[c]) *reinterpret_cast<float4 *>(state + (size_t)(c0 + grp * NC + c) * DP + i * 32 + l8 * 4) = s[c][i];
 }
 
-// Norm over every head's outputs, norm weight and gate: one warp per (row, head).
+// Norm over every head's outputs, norm weight and gate: LPH lanes per (row, head), each with its channels in registers
+// (four consecutive ones at a time where the sizes allow it).
+template <int LPH, bool VEC>
 __global__ void __launch_bounds__(256) delta_output_kernel(const __grid_constant__ DeltaArgs a, const float *__restrict__ o_buf, void *out, int out_fmt,
                                                            uint32_t ld_out) {
+  constexpr int PER = VEC ? 4 : 1, MAXU = VEC ? 2 : 8;  // units per lane: LPH * MAXU * PER >= 256 channels for the widest heads
   pdl_launch_dependents();
   pdl_wait();
   const greta_delta_rule &d = a.d;
-  const uint32_t i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, D = d.dim;
-  if (i >= a.rows.M * d.heads) return;
-  const uint32_t m = i / d.heads, h = i % d.heads;
-  const float *o = o_buf + (size_t)i * D;
-  float q = 0.f;
-  for (uint32_t c = lane; c < D; c += 32) q = fmaf(o[c], o[c], q);
-  const float inv = 1.f / sqrtf(warp_sum(q) / (float)D + d.eps);
-  for (uint32_t c = lane; c < D; c += 32)
-    store_out(out, out_fmt, (size_t)m * ld_out + h * D + c, o[c] * inv * d.norm[(size_t)h * D + c] * d.gate[(size_t)m * d.ld + h * D + c]);
+  const uint32_t i = (blockIdx.x * 256 + threadIdx.x) / LPH, l = threadIdx.x % LPH, D = d.dim;
+  const bool on = i < a.rows.M * d.heads;
+  const uint32_t m = on ? i / d.heads : 0, h = on ? i % d.heads : 0;
+  const float *o = o_buf + (size_t)(on ? i : 0) * D;
+  float v[MAXU][PER], q = 0.f;
+#pragma unroll
+  for (int u = 0; u < MAXU; ++u) {
+    const uint32_t c = (u * LPH + l) * PER;
+#pragma unroll
+    for (int e = 0; e < PER; ++e) v[u][e] = 0.f;
+    if (on && c < D) {
+      if (VEC) {
+        const float4 t = *reinterpret_cast<const float4 *>(o + c);
+        v[u][0] = t.x, v[u][PER > 1 ? 1 : 0] = t.y, v[u][PER > 1 ? 2 : 0] = t.z, v[u][PER > 1 ? 3 : 0] = t.w;
+      } else {
+        v[u][0] = o[c];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < PER; ++e) q = fmaf(v[u][e], v[u][e], q);
+  }
+#pragma unroll
+  for (int off = LPH / 2; off > 0; off >>= 1) q += __shfl_xor_sync(0xffffffffu, q, off);
+  const float inv = 1.f / sqrtf(q / (float)D + d.eps);
+#pragma unroll
+  for (int u = 0; u < MAXU; ++u) {
+    const uint32_t c = (u * LPH + l) * PER;
+    if (!on || c >= D) continue;
+    float y[PER];
+    const float *g = d.gate + (size_t)m * d.ld + h * D + c, *n = d.norm + (size_t)h * D + c;
+#pragma unroll
+    for (int e = 0; e < PER; ++e) y[e] = v[u][e] * inv * n[e] * g[e];
+    const size_t at = (size_t)m * ld_out + h * D + c;
+    if (VEC && out_fmt == GRETA_OUT_BF16) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[PER > 1 ? 1 : 0]), hi = __floats2bfloat162_rn(y[PER > 2 ? 2 : 0], y[PER > 3 ? 3 : 0]);
+      uint2 w;
+      w.x = *reinterpret_cast<const uint32_t *>(&lo);
+      w.y = *reinterpret_cast<const uint32_t *>(&hi);
+      *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(out) + at) = w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < PER; ++e) store_out(out, out_fmt, at + e, y[e]);
+    }
+  }
 }
 
 int check_delta(const char *what, const greta_delta_rule *d, const greta_rows *r) {
@@ -265,7 +407,7 @@ int check_delta(const char *what, const greta_delta_rule *d, const greta_rows *r
 
 template <int RB, int NC>
 int launch_scan(cudaStream_t s, const DeltaArgs &a, float *o_buf, int vec) {
-  using C = ScanCfg<RB>;
+  using C = ScanCfg<RB, NC>;
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -273,7 +415,7 @@ int launch_scan(cudaStream_t s, const DeltaArgs &a, float *o_buf, int vec) {
     GRETA_CUDA_TRY(cudaFuncSetAttribute(delta_scan_kernel<RB, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
     attr_set[dev] = true;
   }
-  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC>, dim3(a.d.heads, (a.d.dim + C::COLS - 1) / C::COLS), dim3(C::COLS / NC * 8), C::SMEM, s, a, o_buf, vec));
+  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC>, dim3(a.d.heads, (a.d.dim + C::COLS - 1) / C::COLS), dim3(C::THREADS), C::SMEM, s, a, o_buf, vec));
   return launched("delta_scan_kernel");
 }
 template <int RB>
@@ -318,10 +460,10 @@ int greta_cuda_delta_scan(greta_stream_t stream, const greta_delta_rule *d, cons
   const int vec = d->dim % 4 == 0 && d->ld % 4 == 0 && d->ld_decay % 4 == 0 && aligned16(d->r) && aligned16(d->k) && aligned16(d->v) && aligned16(d->a) &&
                   aligned16(d->decay);
   switch (dim32(d->dim) / 32) {
-    case 1: return launch_scan<1, 1>(s, a, o_buf, vec);
-    case 2: return launch_scan<2, 1>(s, a, o_buf, vec);
-    case 3: return launch_scan<3, 1>(s, a, o_buf, vec);
-    case 4: return launch_scan<4, 1>(s, a, o_buf, vec);
+    case 1: return launch_scan<1, 2>(s, a, o_buf, vec);
+    case 2: return launch_scan<2, 2>(s, a, o_buf, vec);
+    case 3: return launch_scan<3, 2>(s, a, o_buf, vec);
+    case 4: return launch_scan<4, 2>(s, a, o_buf, vec);
     case 5: return launch_scan<5, 1>(s, a, o_buf, vec);
     case 6: return launch_scan<6, 1>(s, a, o_buf, vec);
     case 7: return launch_scan<7, 1>(s, a, o_buf, vec);
@@ -334,7 +476,16 @@ int greta_cuda_delta_output(greta_stream_t stream, const greta_delta_rule *d, co
   if (int rc = check_delta("delta_output", d, &rows)) return rc;
   GRETA_REQUIRE(o_buf && out && d->norm && d->gate, "delta_output: null pointer");
   const DeltaArgs a{*d, rows};
-  GRETA_CUDA_TRY(launch_pdl(delta_output_kernel, dim3((M * d->heads + 7) / 8), dim3(256), 0, (cudaStream_t)stream, a, o_buf, out, out_fmt, ld_out));
+  cudaStream_t s = (cudaStream_t)stream;
+  const uint32_t D = d->dim, pairs = M * d->heads;
+  const bool vec = D % 4 == 0 && d->ld % 4 == 0 && ld_out % 4 == 0 && aligned16(o_buf) && aligned16(d->gate) && aligned16(d->norm) && aligned16(out);
+  auto grid = [&](uint32_t lanes) { return dim3((pairs + 256 / lanes - 1) / (256 / lanes)); };
+  if (vec && D <= 64)
+    GRETA_CUDA_TRY(launch_pdl(delta_output_kernel<16, true>, grid(16), dim3(256), 0, s, a, o_buf, out, out_fmt, ld_out));
+  else if (vec)
+    GRETA_CUDA_TRY(launch_pdl(delta_output_kernel<32, true>, grid(32), dim3(256), 0, s, a, o_buf, out, out_fmt, ld_out));
+  else
+    GRETA_CUDA_TRY(launch_pdl(delta_output_kernel<32, false>, grid(32), dim3(256), 0, s, a, o_buf, out, out_fmt, ld_out));
   return launched("delta_output_kernel");
 }
 

@@ -3,11 +3,17 @@
 // bf16: tensor cores.  The weight rows are the 128-row operand of tcgen05.mma and TN tokens its N dimension, so a thread
 // of the epilogue owns one weight row (one segment, one bias) and a warp stores 32 consecutive outputs of a token.
 // Persistent CTAs, one per SM, walk the tiles with the token tiles innermost: the CTAs in flight share a few weight row
-// tiles, which are read from HBM once.  Roles (192 threads): warp 0 TMA producer of both operands (128-byte swizzle, 64
-// columns per stage), warp 1 MMA issuer (one lane), warps 2-5 epilogue.  Two accumulators in TMEM: a tile's epilogue
-// runs under the next tile's MMAs.  Every mbarrier wait is bounded (see greta_cuda_linear_gemm_status).
+// tiles, which are read from HBM once.  Roles (320 threads): warp 0 TMA producer of both operands (128-byte swizzle, 64
+// columns per stage), warp 1 MMA issuer (one lane), warps 2-9 epilogue, two per TMEM lane quadrant.  Two accumulators in
+// TMEM: a tile's epilogue runs under the next tile's MMAs.  Every mbarrier wait is bounded (see
+// greta_cuda_linear_gemm_status).
+// Where there are fewer tiles than SMs, a cluster of 2, 4 or 8 CTAs shares a tile's K loop: every CTA leaves its partial
+// tile in its shared memory and finishes a share of the tokens, adding the partial sums in rank order through distributed
+// shared memory.
 //
 // fp32: plain 64 x 64 tiles of 32-bit FMAs, for models that run in 32-bit.
+#include <cooperative_groups.h>
+
 #include <algorithm>
 
 #include "dense_device.cuh"
@@ -26,10 +32,53 @@ struct DCfg {
   static constexpr int A_BYTES = TILE_N * BK * 2, B_BYTES = TN * BK * 2, STAGE = A_BYTES + B_BYTES;
   static constexpr int ST = TN == 256 ? 4 : TN == 128 ? 6 : 8;
   static constexpr int COLS = 2 * TN < 32 ? 32 : 2 * TN;  // two accumulators; a power of two
-  static constexpr int THREADS = 192;
+  static constexpr int EPI_WARPS = TN >= 64 ? 8 : 4;
+  static constexpr int THREADS = 64 + EPI_WARPS * 32;
   static constexpr size_t SMEM = (size_t)ST * STAGE + 1024 + 256;
   static_assert(COLS <= 512 && SMEM <= 232448, "tile configuration");
 };
+
+// 32 consecutive tokens (from m on, cnt of them present) of one weight row: bias, activation, store.
+template <int ACT>
+__device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
+  const size_t base = (size_t)m * g.ld + g.col0 + r;
+  if (g.accumulate) {
+    float *o = static_cast<float *>(g.out) + base;
+    float old[32];
+#pragma unroll
+    for (int j = 0; j < 32; ++j) old[j] = j < cnt ? o[(size_t)j * g.ld] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      if (j < cnt) o[(size_t)j * g.ld] = old[j] + apply_act(ACT, __uint_as_float(v[j]) + bias);
+  } else if (g.out_fmt == GRETA_OUT_F32) {
+    float *o = static_cast<float *>(g.out) + base;
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      if (j < cnt) o[(size_t)j * g.ld] = apply_act(ACT, __uint_as_float(v[j]) + bias);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(ACT, __uint_as_float(v[j]) + bias), g.pair_offset);
+  }
+}
+__device__ __forceinline__ void finish_row(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
+  switch (g.act) {
+    case GRETA_ACT_GELU_ERF: finish_row_act<GRETA_ACT_GELU_ERF>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_SIGMOID: finish_row_act<GRETA_ACT_SIGMOID>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_TANH: finish_row_act<GRETA_ACT_TANH>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_DELTA_DECAY: finish_row_act<GRETA_ACT_DELTA_DECAY>(g, r, bias, m, cnt, v); break;
+    default: finish_row_act<GRETA_ACT_NONE>(g, r, bias, m, cnt, v); break;
+  }
+}
+
+// A copy still in flight must not outlive the CTA: after an abort the producer gives the last ones a bounded chance to land.
+__device__ __forceinline__ void drain_copies(uint64_t *full, uint32_t issued, uint32_t stages) {
+  for (uint32_t j = issued > stages ? issued - stages : 0; j < issued; ++j) {
+    const long long t0 = clock64();
+    while (!mbar_try_wait(&full[j % stages], (j / stages) & 1) && clock64() - t0 < 20000000ll) {
+    }
+  }
+}
 
 template <int TN>
 __global__ void __launch_bounds__(DCfg<TN>::THREADS, 1)
@@ -53,7 +102,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
     }
     for (int b = 0; b < 2; ++b) {
       mbar_init(&acc_full[b], 1);
-      mbar_init(&acc_empty[b], 4);
+      mbar_init(&acc_empty[b], C::EPI_WARPS);
     }
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -91,13 +140,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
           }
         }
       }
-      if (*abort_flag) {  // a bounded chance for the copies in flight to land before the CTA exits
-        for (uint32_t j = issued > (uint32_t)ST ? issued - ST : 0; j < issued; ++j) {
-          const long long t0 = clock64();
-          while (!mbar_try_wait(&full[j % ST], (j / ST) & 1) && clock64() - t0 < 20000000ll) {
-          }
-        }
-      }
+      if (*abort_flag) drain_copies(full, issued, ST);
     }
   } else if (warp == 1) {
     if (lane == 0) {
@@ -128,12 +171,11 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
       }
     }
   } else {
-    const int quad = warp & 3;
+    constexpr int SHARE = TN / (C::EPI_WARPS / 4);  // tokens per warp
+    const int quad = warp & 3, c_begin = ((warp - 2) >> 2) * SHARE;
     uint32_t it = 0;
     for (uint32_t t = blockIdx.x; t < tiles; t += gridDim.x, ++it) {
       const uint32_t b = it & 1, m0 = (t % tok_tiles) * TN, row = (t / tok_tiles) * TILE_N + quad * 32 + lane;
-      if (!mbar_wait(&acc_full[b], (it >> 1) & 1, abort_flag, 400 + b)) break;
-      tc_fence_after();
       greta_out_segment g{};
       uint32_t r = 0;
       float bias = 0.f;
@@ -142,36 +184,22 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
         r = row - g.row0;
         if (g.bias) bias = __ldg(g.bias + r);
       }
+      if (!mbar_wait(&acc_full[b], (it >> 1) & 1, abort_flag, 400 + b)) break;
+      tc_fence_after();
 #pragma unroll 1
-      for (int c = 0; c < TN; c += 32) {
+      for (int c = c_begin; c < c_begin + SHARE; c += 32) {
         uint32_t v[32];
         __syncwarp();
         if (m0 + c < M) {
           tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + b * TN + c, v);
           tmem_ld_wait();
         }
-        if (c + 32 >= TN) {  // accumulator read: the issuer may overwrite it
+        if (c + 32 >= c_begin + SHARE) {  // this warp's share is read: the issuer may overwrite it
           tc_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&acc_empty[b]);
         }
-        if (row < N && m0 + c < M) {
-          const uint32_t cnt = min(32u, M - m0 - c);
-          const size_t base = (size_t)(m0 + c) * g.ld + g.col0 + r;
-          if (g.accumulate) {
-            float *o = static_cast<float *>(g.out) + base;
-            float old[32];
-#pragma unroll
-            for (int j = 0; j < 32; ++j) old[j] = j < cnt ? o[(size_t)j * g.ld] : 0.f;
-#pragma unroll
-            for (int j = 0; j < 32; ++j)
-              if (j < cnt) o[(size_t)j * g.ld] = old[j] + apply_act(g.act, __uint_as_float(v[j]) + bias);
-          } else {
-#pragma unroll
-            for (int j = 0; j < 32; ++j)
-              if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(g.act, __uint_as_float(v[j]) + bias), g.pair_offset);
-          }
-        }
+        if (row < N && m0 + c < M) finish_row(g, r, bias, m0 + c, min(32u, M - m0 - c), v);
       }
     }
   }
@@ -180,6 +208,132 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
   if (warp == 1) {
     tc_fence_after();
     tmem_dealloc(tmem_base, C::COLS);
+  }
+}
+
+// One tile per cluster, its K loop shared by the cluster's CTAs.  Same roles; warps 2-9 first leave the partial tile
+// [token][128 rows] in the idle ring, then finish tokens rank * TN / S ...
+template <int TN>
+__global__ void __launch_bounds__(DCfg<TN>::THREADS, 1)
+linear_tc_split_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ Segments sg,
+                       uint32_t M, uint32_t N, uint32_t K) {
+  namespace cg = cooperative_groups;
+  using C = DCfg<TN>;
+  constexpr int ST = C::ST, COLS = TN < 32 ? 32 : TN;
+  static_assert((size_t)TN * TILE_N * 4 <= (size_t)ST * C::STAGE, "the partial tile reuses the ring");
+  cg::cluster_group cl = cg::this_cluster();
+  const uint32_t S = cl.num_blocks(), rank = cl.block_rank();
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t *smem = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint64_t *bars = reinterpret_cast<uint64_t *>(smem + (size_t)ST * C::STAGE);
+  uint64_t *full = bars, *empty = bars + ST, *acc_full = bars + 2 * ST;
+  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(acc_full + 1);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+  float *part = reinterpret_cast<float *>(smem);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint32_t KT = (K + BK - 1) / BK, tok_tiles = (M + TN - 1) / TN, tile = blockIdx.x / S;
+  const uint32_t n0 = (tile / tok_tiles) * TILE_N, m0 = (tile % tok_tiles) * TN;
+  const uint32_t kt0 = KT * rank / S, kt1 = KT * (rank + 1) / S;  // the plan leaves every CTA some stages
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < ST; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
+    }
+    mbar_init(acc_full, 1);
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_w) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_x) : "memory");
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  pdl_launch_dependents();
+  pdl_wait();
+
+  if (warp == 0) {
+    if (lane == 0) {
+      uint32_t issued = 0, s = 0, ph = 1;
+      for (uint32_t kt = kt0; kt < kt1; ++kt) {
+        if (!mbar_wait(&empty[s], ph, abort_flag, 100 + s)) break;
+        uint8_t *st = smem + (size_t)s * C::STAGE;
+        mbar_arrive_expect_tx(&full[s], C::STAGE);
+        tma_load_2d(st, &tmap_w, (int)(kt * BK), (int)n0, &full[s]);
+        tma_load_2d(st + C::A_BYTES, &tmap_x, (int)(kt * BK), (int)m0, &full[s]);
+        ++issued;
+        if (++s == ST) {
+          s = 0;
+          ph ^= 1;
+        }
+      }
+      if (*abort_flag) drain_copies(full, issued, ST);
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc = instr_desc_bf16(TILE_N, TN);
+      const uint32_t lo0 = smem_desc_lo(smem_u32(smem));
+      uint32_t s = 0, ph = 0;
+      bool ok = true;
+      for (uint32_t kt = kt0; kt < kt1; ++kt) {
+        ok = mbar_wait(&full[s], ph, abort_flag, 200 + s);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t w_lo = lo0 + s * (C::STAGE >> 4), x_lo = w_lo + (C::A_BYTES >> 4);
+#pragma unroll
+        for (int k16 = 0; k16 < BK / 16; ++k16)
+          umma_f16(tmem_base, w_lo + k16 * 2, x_lo + k16 * 2, SMEM_DESC_HI_SW128, idesc, (kt > kt0 || k16) ? 1u : 0u);
+        umma_commit(&empty[s]);
+        if (++s == ST) {
+          s = 0;
+          ph ^= 1;
+        }
+      }
+      if (ok) umma_commit(acc_full);
+    }
+  } else {
+    constexpr int SHARE = TN / (C::EPI_WARPS / 4);
+    const int quad = warp & 3, c_begin = ((warp - 2) >> 2) * SHARE;
+    if (mbar_wait(acc_full, 0, abort_flag, 400)) {  // every stage has been loaded and multiplied: the ring is idle
+      tc_fence_after();
+#pragma unroll 1
+      for (int c = c_begin; c < c_begin + SHARE; c += 32) {
+        uint32_t v[32];
+        __syncwarp();
+        tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + c, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) part[(size_t)(c + j) * TILE_N + quad * 32 + lane] = __uint_as_float(v[j]);
+      }
+    }
+  }
+  tc_fence_before();
+  __syncwarp();
+  cl.sync();
+  if (warp >= 2) {
+    const uint32_t per = TN / S, wq = (warp - 2) & 3, half = (warp - 2) >> 2, halves = C::EPI_WARPS / 4;
+    const uint32_t row_l = wq * 32 + lane, row = n0 + row_l;
+    if (row < N) {
+      const greta_out_segment g = sg.s[segment_of(sg, row)];
+      for (uint32_t j = half; j < per; j += halves) {
+        const uint32_t c = rank * per + j, m = m0 + c;
+        if (m >= M) break;
+        float z = 0.f;
+        for (uint32_t r = 0; r < S; ++r) z += *cl.map_shared_rank(part + (size_t)c * TILE_N + row_l, r);
+        store_segment(g, row, m, z);
+      }
+    }
+  }
+  __syncwarp();
+  cl.sync();  // no CTA leaves while another reads its shared memory
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, COLS);
   }
 }
 
@@ -239,21 +393,45 @@ int make_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, u
 }
 
 template <int TN>
-int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, const void *x, uint32_t ldx, uint32_t M) {
+int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, const void *x, uint32_t ldx, uint32_t M, uint32_t split) {
   using C = DCfg<TN>;
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
     GRETA_CUDA_TRY(cudaFuncSetAttribute(linear_tc_kernel<TN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+    GRETA_CUDA_TRY(cudaFuncSetAttribute(linear_tc_split_kernel<TN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
     attr_set[dev] = true;
   }
   CUtensorMap mw, mx;
   if (int rc = make_map(&mw, l->w, l->K, l->N, l->ldw, TILE_N)) return rc;  // columns past K read as zero in both operands
   if (int rc = make_map(&mx, x, l->K, M, ldx, TN)) return rc;
   const uint32_t tiles = ((l->N + TILE_N - 1) / TILE_N) * ((M + TN - 1) / TN);
+  if (split > 1) {
+    GRETA_CUDA_TRY(launch_pdl_cluster(linear_tc_split_kernel<TN>, dim3(tiles * split), dim3(C::THREADS), split, C::SMEM, s, mw, mx, sg, M, l->N, l->K));
+    return launched("linear_tc_split_kernel");
+  }
   GRETA_CUDA_TRY(launch_pdl(linear_tc_kernel<TN>, dim3(std::min(tiles, (uint32_t)sm_count())), dim3(C::THREADS), C::SMEM, s, mw, mx, sg, M, l->N, l->K));
   return launched("linear_tc_kernel");
+}
+
+// Token tile and K split for a product: the widest tile whose tiles (times the CTAs that share one) fill most SMs.
+void plan_dense(uint32_t M, uint32_t N, uint32_t K, uint32_t *tn, uint32_t *split) {
+  const uint32_t row_tiles = (N + TILE_N - 1) / TILE_N, KT = (K + BK - 1) / BK, sms = (uint32_t)sm_count();
+  uint32_t best = 0;
+  for (uint32_t t : {256u, 128u, 64u, 32u}) {
+    if (t > 32 && M <= t / 2) continue;  // mostly padding
+    const uint32_t tiles = row_tiles * ((M + t - 1) / t);
+    uint32_t s = 1;
+    while (s < 8 && tiles * s * 2 <= sms && KT >= s * 2 * 4) s *= 2;
+    const uint32_t fill = std::min(sms, tiles * s);
+    if (fill * 10 > best * 12 || best == 0) {  // a narrower tile has to fill clearly more SMs
+      best = fill;
+      *tn = t;
+      *split = s;
+    }
+    if (best * 10 >= sms * 8) break;
+  }
 }
 
 }  // namespace
@@ -273,13 +451,12 @@ int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *l, const v
     return launched("linear_f32_kernel");
   }
   GRETA_REQUIRE(ldx >= l->K && ldx % 8 == 0, "linear_gemm: ldx=%u K=%u", ldx, l->K);
-  // the widest token tile that still gives most SMs a tile
-  const uint32_t row_tiles = (l->N + TILE_N - 1) / TILE_N;
-  auto enough = [&](uint32_t tn) { return row_tiles * ((M + tn - 1) / tn) >= 120 && M > tn / 2; };
-  if (enough(256)) return launch_dense<256>(s, l, sg, x, ldx, M);
-  if (enough(128)) return launch_dense<128>(s, l, sg, x, ldx, M);
-  if (enough(64)) return launch_dense<64>(s, l, sg, x, ldx, M);
-  return launch_dense<32>(s, l, sg, x, ldx, M);
+  uint32_t tn = 32, split = 1;
+  plan_dense(M, l->N, l->K, &tn, &split);
+  if (tn == 256) return launch_dense<256>(s, l, sg, x, ldx, M, split);
+  if (tn == 128) return launch_dense<128>(s, l, sg, x, ldx, M, split);
+  if (tn == 64) return launch_dense<64>(s, l, sg, x, ldx, M, split);
+  return launch_dense<32>(s, l, sg, x, ldx, M, split);
 }
 
 int greta_cuda_linear_gemm_status(int *code) {

@@ -16,6 +16,7 @@ using namespace greta;
 namespace {
 
 constexpr int GV_THREADS = 256, GV_WARPS = 8;
+constexpr bool PREFETCH = true;
 
 template <typename WT>
 struct W8;  // 8 consecutive weights as stored
@@ -49,7 +50,7 @@ struct W8<float> {
 template <typename WT, int MR, int R>
 __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__restrict__ W, uint32_t N, uint32_t K, uint32_t ldw, Segments sg,
                                                                  const float *x, uint32_t ldx, const float *__restrict__ ln_w,
-                                                                 const float *__restrict__ ln_b, float eps, uint32_t M, uint32_t chunk) {
+                                                                 const float *__restrict__ ln_b, float eps, uint32_t M, uint32_t chunk, int vec) {
   extern __shared__ float4 xs[];  // [MR][2][chunk / 8]
   __shared__ float red[32], stat[MR][2];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -62,6 +63,15 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
   if (any0) {
 #pragma unroll
     for (int r = 0; r < R; ++r) first[r].load(wrow[r]);
+  }
+  if (PREFETCH) {  // the rest of the rows starts its way from HBM to L2 while this CTA still waits for its input
+    const uint32_t row_bytes = ldw * (uint32_t)sizeof(WT);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const char *p = reinterpret_cast<const char *>(W + (size_t)min(n0 + r, N - 1) * ldw);
+      for (uint32_t b = 512 * sizeof(WT) / 2 + lane * 128; b < min(row_bytes, 16384u); b += 32 * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(p + b));
+    }
   }
   pdl_launch_dependents();
   pdl_wait();
@@ -113,6 +123,24 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
       const float *xr = x + (size_t)m * ldx;
       const bool row = (uint32_t)m < M;
       const float mean = ln_w && row ? stat[m][0] : 0.f, inv = ln_w && row ? stat[m][1] : 1.f;
+      if (vec && row) {  // four columns are one slot of a plane
+        for (uint32_t k = threadIdx.x * 4; k < kc; k += GV_THREADS * 4) {
+          const uint32_t col = k0 + k;
+          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (col < K) {
+            v = *reinterpret_cast<const float4 *>(xr + col);
+            if (ln_w) {
+              const float4 w = __ldg(reinterpret_cast<const float4 *>(ln_w + col)), b = __ldg(reinterpret_cast<const float4 *>(ln_b + col));
+              v.x = (v.x - mean) * inv * w.x + b.x;
+              v.y = (v.y - mean) * inv * w.y + b.y;
+              v.z = (v.z - mean) * inv * w.z + b.z;
+              v.w = (v.w - mean) * inv * w.w + b.w;
+            }
+          }
+          reinterpret_cast<float4 *>(xd)[((k >> 2) & 1) * plane + (k >> 3)] = v;
+        }
+        continue;
+      }
       for (uint32_t k = threadIdx.x; k < kc; k += GV_THREADS) {
         const uint32_t col = k0 + k;
         float v = 0.f;
@@ -154,7 +182,7 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
       step(first, k);
       k += 256;
     }
-    constexpr int UN = R >= 4 ? 2 : 4;  // steps in flight
+    constexpr int UN = MR > 2 ? (R >= 4 ? 2 : 4) : R >= 4 ? 2 : R == 2 ? 4 : 8;  // steps in flight
     for (; k + (UN - 1) * 256 < kc; k += UN * 256) {
       W8<WT> w[UN][R];
 #pragma unroll
@@ -184,12 +212,51 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
   if (m < min(M, (uint32_t)MR) && row < N) store_segment(sg.s[segment_of(sg, row)], row, m, mine);
 }
 
+// One CTA per row; rows of up to 8192 columns (a multiple of 4) are read once and kept in registers.
 __global__ void __launch_bounds__(256) layer_norm_kernel(const float *__restrict__ x, const float *__restrict__ w, const float *__restrict__ b, float eps,
-                                                         void *out, int out_fmt, uint32_t D, uint32_t ld) {
+                                                         void *out, int out_fmt, uint32_t D, uint32_t ld, int vec) {
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   const float *xr = x + (size_t)blockIdx.x * D;
+  if (vec) {
+    constexpr int U = 8;
+    float4 v[U];
+    float s = 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t k = (u * 256 + threadIdx.x) * 4;
+      v[u] = k < D ? *reinterpret_cast<const float4 *>(xr + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+      s += (v[u].x + v[u].y) + (v[u].z + v[u].w);
+    }
+    const float mean = block_sum_all(s, red) / (float)D;
+    float q = 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if ((u * 256 + threadIdx.x) * 4 >= D) continue;
+      v[u].x -= mean, v[u].y -= mean, v[u].z -= mean, v[u].w -= mean;
+      q = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, q))));
+    }
+    const float inv = 1.f / sqrtf(block_sum_all(q, red) / (float)D + eps);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t k = (u * 256 + threadIdx.x) * 4;
+      if (k >= D) continue;
+      const float4 g = *reinterpret_cast<const float4 *>(w + k), h = *reinterpret_cast<const float4 *>(b + k);
+      const float4 y = make_float4(v[u].x * inv * g.x + h.x, v[u].y * inv * g.y + h.y, v[u].z * inv * g.z + h.z, v[u].w * inv * g.w + h.w);
+      const size_t at = (size_t)blockIdx.x * ld + k;
+      if (out_fmt == GRETA_OUT_F32) {
+        *reinterpret_cast<float4 *>(static_cast<float *>(out) + at) = y;
+      } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(y.x, y.y), hi = __floats2bfloat162_rn(y.z, y.w);
+        uint2 p;
+        p.x = *reinterpret_cast<const uint32_t *>(&lo);
+        p.y = *reinterpret_cast<const uint32_t *>(&hi);
+        *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(out) + at) = p;
+      }
+    }
+    return;
+  }
   float s = 0.f;
   for (uint32_t k = threadIdx.x; k < D; k += 256) s += xr[k];
   const float mean = block_sum_all(s, red) / (float)D;
@@ -242,8 +309,9 @@ int launch_gemv(cudaStream_t s, const greta_linear *l, const Segments &sg, const
     attr_set[dev] = true;
   }
   const uint32_t grid = (l->N + GV_WARPS * R - 1) / (GV_WARPS * R);
+  const int vec = l->K % 4 == 0 && ldx % 4 == 0 && aligned16(x) && (!ln_w || (aligned16(ln_w) && aligned16(ln_b)));
   GRETA_CUDA_TRY(launch_pdl(linear_gemv_kernel<WT, MR, R>, dim3(grid), dim3(GV_THREADS), smem, s, static_cast<const WT *>(l->w), l->N, l->K, l->ldw, sg, x,
-                            ldx, ln_w, ln_b, eps, M, chunk));
+                            ldx, ln_w, ln_b, eps, M, chunk, vec));
   return launched("linear_gemv_kernel");
 }
 template <typename WT, int MR>
@@ -302,7 +370,8 @@ int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w,
   if (M == 0) return GRETA_OK;
   GRETA_REQUIRE(x && w && b && out && D && ld_out >= D, "layer_norm: bad argument");
   GRETA_REQUIRE(out_fmt == GRETA_OUT_F32 || out_fmt == GRETA_OUT_BF16, "layer_norm: output format %d", out_fmt);
-  GRETA_CUDA_TRY(launch_pdl(layer_norm_kernel, dim3(M), dim3(256), 0, (cudaStream_t)stream, x, w, b, eps, out, out_fmt, D, ld_out));
+  const int vec = D <= 8192 && D % 4 == 0 && ld_out % 4 == 0 && aligned16(x) && aligned16(w) && aligned16(b) && aligned16(out);
+  GRETA_CUDA_TRY(launch_pdl(layer_norm_kernel, dim3(M), dim3(256), 0, (cudaStream_t)stream, x, w, b, eps, out, out_fmt, D, ld_out, vec));
   return launched("layer_norm_kernel");
 }
 

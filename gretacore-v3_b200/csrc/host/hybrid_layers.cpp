@@ -4,8 +4,8 @@
 //   1. LN -> every input projection of mixer and feed-forward (w_in), activations in the epilogue
 //   2. the mixer's core: windowed attention over the cache, or the delta rule over the state
 //   3. [mixer | feed-forward] columns -> both output projections and the residual (w_out)
-// For up to 8 rows (decode, short portions) 1 and 3 are GEMVs with the norm fused in: three kernels per layer and decode step.
-// More rows run on the tensor cores (bf16) behind one layer-norm kernel.  The residual stream, the projections that enter a
+// For a single row (decode; up to 8 in fp32) 1 and 3 are GEMVs with the norm fused in: three kernels per layer and decode
+// step.  More rows run on the tensor cores (bf16) behind one layer-norm kernel.  The residual stream, the projections that enter a
 // mixer, scores, states and norms are fp32 in either mode.
 //
 // Caches and states belong to the scheduler's sequence slots and hold no trace of earlier sequences: positions in front of a
@@ -29,7 +29,8 @@ namespace {
 
 inline cudaStream_t H(gcore::rt::GretaStream *s) { return static_cast<GretaStreamCuda *>(s)->handle(); }
 inline uint32_t up(uint32_t n, uint32_t to) { return (n + to - 1) / to * to; }
-constexpr uint32_t FEW_ROWS = 8;       // rows up to which the linears run as GEMVs
+constexpr uint32_t FEW_ROWS = 8;       // fp32 weights: rows up to which the linears run as GEMVs
+constexpr uint32_t FEW_ROWS_BF16 = 1;  // bf16: the tensor-core kernel streams the weights as fast for two rows as the GEMV for one
 constexpr uint32_t MMA_MIN_ROWS = 16;  // portions from which attention runs on the tensor cores
 
 #define GRETA_TRY(call, what)                                                \
@@ -267,7 +268,7 @@ bool BlockScheduler::allocate_hybrid_activations(std::string *err) {
   if (!zeroed(a.x, (size_t)R * D * 4) || !zeroed(a.tokens, (size_t)R * 4) || !zeroed(a.d_pos, 2 * (size_t)B * 4) || !zeroed(a.d_next, (size_t)B * 4) ||
       !zeroed(a.out_tokens, (size_t)B * max_seq_ * 4) || !zeroed(logits_, (size_t)B * c.vocab_size * 4))
     return false;
-  const size_t few = bf16 ? std::min(R, FEW_ROWS) : R;
+  const size_t few = bf16 ? std::min(R, FEW_ROWS_BF16) : R;
   if (!zeroed(w.h, (size_t)R * w.h_ld * cb) || !zeroed(w.proj, (size_t)R * proj * 4) || !zeroed(w.cat, few * cat * 4) ||
       (bf16 && !zeroed(w.cat16, (size_t)R * cat * 2)) || !zeroed(w.q, (size_t)R * q * 4) || !zeroed(w.x_rows, (size_t)64 * D * 4) ||
       !zeroed(w.logits_rows, (size_t)64 * c.vocab_size * 4))
@@ -311,7 +312,7 @@ bool BlockScheduler::hybrid_layer(size_t layer, const greta_rows &rows, std::str
   HybridLayerBuffers &b = hybrid_[layer];
   HybridActivations &w = hact_;
   cudaStream_t s = H(stream_);
-  const bool bf16 = c.weight_type == GretaDataType::BF16, few = rows.M <= FEW_ROWS, decode = rows.d_pos != nullptr;
+  const bool bf16 = c.weight_type == GretaDataType::BF16, few = rows.M <= (bf16 ? FEW_ROWS_BF16 : FEW_ROWS), decode = rows.d_pos != nullptr;
   const bool delta = m.kind == MixerKind::GENERAL_DELTA;
   const int fmt = bf16 ? GRETA_FMT_BF16 : GRETA_FMT_F32;
   const uint32_t D = c.dim, HD = m.heads * m.dim;
@@ -456,7 +457,7 @@ bool BlockScheduler::hybrid_logits(const float *x, uint32_t n, float *logits, st
   head.ldw = head_ld_;
   head.n_segments = 1;
   head.seg[0] = greta_out_segment{0, c.vocab_size, GRETA_ACT_NONE, GRETA_OUT_F32, 0, nullptr, logits, c.vocab_size, 0, 0};
-  if (n <= FEW_ROWS) {
+  if (n <= (bf16 ? FEW_ROWS_BF16 : FEW_ROWS)) {
     GRETA_TRY(greta_cuda_linear_gemv(s, &head, x, c.dim, fp(output_norm_), fp(final_norm_b_), c.rms_eps, n), "lm head");
     return true;
   }

@@ -28,6 +28,27 @@ struct WinArgs {
 __device__ __forceinline__ uint32_t cache_row(const greta_window_attn &a, uint32_t p) {
   return p < a.keep_first ? p : a.keep_first + (p - a.keep_first) % a.ring;
 }
+// Keys that a row (or a tile of rows from position i0 on, up to i1) may see, as a list: the kept positions in front of the
+// window, then the window; and where they lie in the cache (one division per list, none per key).
+struct KeyList {
+  uint32_t kept, lo, total, keep, ring, p0, base;
+  __device__ __forceinline__ KeyList(const greta_window_attn &a, uint32_t i0, uint32_t i1) {
+    lo = a.window && i0 + 1 > a.window ? i0 + 1 - a.window : 0;
+    kept = min(a.keep_first, lo);
+    total = kept + (i1 - lo + 1);
+    keep = a.keep_first;
+    ring = a.ring;
+    p0 = max(lo, keep);
+    base = (p0 - keep) % ring;
+  }
+  __device__ __forceinline__ uint32_t position(uint32_t t) const { return t < kept ? t : lo + (t - kept); }
+  __device__ __forceinline__ uint32_t row(uint32_t t) const {
+    const uint32_t p = position(t);
+    if (p < keep) return p;
+    const uint32_t o = base + (p - p0);  // p - p0 < ring: a ring holds every position that is seen
+    return keep + (o >= ring ? o - ring : o);
+  }
+};
 template <typename CT>
 __device__ __forceinline__ CT to_cache(float v);
 template <>
@@ -93,8 +114,72 @@ __device__ __forceinline__ void store_cache(const greta_window_attn &a, uint32_t
     if (lane + 32 * i < d8) dst[lane + 32 * i] = to_cache<CT>(v[i]);
 }
 
-template <typename CT>
+// A warp takes one head unit through CV_ROWS consecutive rows: the convolution's weights and its window of projected rows
+// stay in registers, every projected value is read once.  TAPS 0: no convolution; CH: 32-channel groups of the widest head.
+constexpr int CV_ROWS = 16;
+template <typename CT, int TAPS, int CH>
 __global__ void __launch_bounds__(256) conv_norm_kernel(const __grid_constant__ WinArgs w, float *__restrict__ q_out) {
+  constexpr int W = TAPS > 1 ? TAPS : 1;
+  pdl_launch_dependents();
+  pdl_wait();
+  const greta_window_attn &a = w.a;
+  const uint32_t u = blockIdx.x * 8 + (threadIdx.x >> 5), m0 = blockIdx.y * CV_ROWS, m1 = min(m0 + CV_ROWS, w.rows.M), slot = w.rows.slot0;
+  const int lane = threadIdx.x & 31;
+  const uint32_t HK = a.heads + a.kv_heads, C = HK * a.dim + a.kv_heads * a.vdim;
+  if (u >= HK + a.kv_heads) return;
+  const bool is_v = u >= HK;
+  const uint32_t d = is_v ? a.vdim : a.dim, d8 = up8(d), c0 = unit_col(a, u) + lane;
+  float cw[CH][W], win[CH][W];  // win[.][j]: the projected value W - 1 - j rows back
+#pragma unroll
+  for (int i = 0; i < CH; ++i)
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      const bool on = lane + 32 * i < (int)d;
+      cw[i][j] = TAPS && on ? a.conv[(size_t)(c0 + 32 * i) * TAPS + j] : 1.f;
+      win[i][j] = 0.f;
+      const uint32_t back = W - 1 - j, p = w.rows.pos0 + m0;
+      if (back && on && back <= p) {
+        const uint32_t q = p - back;
+        win[i][j] = back <= m0 ? a.proj[(size_t)(m0 - back) * a.ld_proj + c0 + 32 * i] : a.history[((size_t)slot * W + q % W) * C + c0 + 32 * i];
+      }
+    }
+  float cur[CH];
+#pragma unroll
+  for (int i = 0; i < CH; ++i) cur[i] = lane + 32 * i < (int)d ? a.proj[(size_t)m0 * a.ld_proj + c0 + 32 * i] : 0.f;
+  for (uint32_t m = m0; m < m1; ++m) {
+    float v[8], q = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+      win[i][W - 1] = cur[i];
+      cur[i] = m + 1 < m1 && lane + 32 * i < (int)d ? a.proj[(size_t)(m + 1) * a.ld_proj + c0 + 32 * i] : 0.f;  // the next row travels meanwhile
+      float y = 0.f;
+#pragma unroll
+      for (int j = 0; j < W; ++j) y = fmaf(cw[i][j], win[i][j], y);
+#pragma unroll
+      for (int j = 0; j + 1 < W; ++j) win[i][j] = win[i][j + 1];
+      v[i] = lane + 32 * i < (int)d ? y : 0.f;
+      q = fmaf(v[i], v[i], q);
+    }
+    if (!is_v) {
+      const float inv = 1.f / sqrtf(warp_sum(q) / (float)d + a.eps);
+#pragma unroll
+      for (int i = 0; i < CH; ++i) v[i] *= inv;
+    }
+    if (u < a.heads) {
+      float *dst = q_out + ((size_t)m * a.heads + u) * d8;
+#pragma unroll
+      for (int i = 0; i < CH; ++i)
+        if (lane + 32 * i < (int)d8) dst[lane + 32 * i] = v[i];
+    } else {
+      store_cache<CT>(a, slot, w.rows.pos0 + m, is_v ? u - HK : u - a.heads, is_v, lane, v);
+    }
+  }
+}
+// Any number of taps: one warp per (row, head unit).
+template <typename CT>
+__global__ void __launch_bounds__(256) conv_norm_any_kernel(const __grid_constant__ WinArgs w, float *__restrict__ q_out) {
   pdl_launch_dependents();
   pdl_wait();
   const greta_window_attn &a = w.a;
@@ -133,7 +218,7 @@ __device__ __forceinline__ float score(const greta_window_attn &a, uint32_t h, f
   return s;
 }
 
-constexpr int WR_KEYS = 64, WR_THREADS = 256;
+constexpr int WR_KEYS = 128, WR_THREADS = 256, KPG = WR_KEYS / 32;  // keys of a pass, keys per group of eight lanes
 
 // grid (splits, kv heads * head passes, rows), cluster (splits, 1, 1); HN query heads of one key/value head per CTA.
 template <typename CT, int HN, bool FUSED>
@@ -155,8 +240,8 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   pdl_launch_dependents();
   pdl_wait();
   const uint32_t slot = w.rows.d_pos ? w.rows.slot0 + m : w.rows.slot0, i = w.rows.d_pos ? w.rows.d_pos[m] : w.rows.pos0 + m;
-  const uint32_t lo = a.window && i + 1 > a.window ? i + 1 - a.window : 0, kept = min(a.keep_first, lo), total = kept + (i - lo + 1);
-  const uint32_t per = (total + S - 1) / S, t_begin = min(total, split * per), t_end = min(total, t_begin + per);
+  const KeyList keys(a, i, i);
+  const uint32_t total = keys.total, per = (total + S - 1) / S, t_begin = min(total, split * per), t_end = min(total, t_begin + per);
   const uint32_t rows = a.keep_first + a.ring;
   const CT *kc = static_cast<const CT *>(a.k_cache) + ((size_t)slot * a.kv_heads + g) * rows * d8;
   const CT *vc = static_cast<const CT *>(a.v_cache) + ((size_t)slot * a.kv_heads + g) * rows * v8;
@@ -201,7 +286,6 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   }
   __syncthreads();  // also: this CTA's cache row is visible to it
 
-  auto position = [&](uint32_t t) { return t < kept ? t : lo + (t - kept); };
   const uint32_t pr = threadIdx.x % tpp, kg = threadIdx.x / tpp;
   const bool pv = pr < pairs && kg < KG;
   float acc[HN][2];
@@ -209,43 +293,70 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   for (int h = 0; h < HN; ++h) acc[h][0] = acc[h][1] = 0.f;
   for (uint32_t t0 = t_begin; t0 < t_end; t0 += WR_KEYS) {
     const uint32_t n = min((uint32_t)WR_KEYS, t_end - t0);
-    const uint32_t l8 = threadIdx.x & 7, grp = threadIdx.x >> 3;  // 32 groups of 8 lanes, a key each
-    for (uint32_t e = grp; e < WR_KEYS; e += WR_THREADS / 8) {
-      const bool on = e < n;
-      const uint32_t j = position(t0 + (on ? e : 0));
-      const CT *kr = kc + (size_t)cache_row(a, j) * d8;
-      float dot[HN];
+    const uint32_t l8 = threadIdx.x & 7, grp = threadIdx.x >> 3;  // 32 groups of 8 lanes, KPG keys each
+    uint32_t krow[KPG];
+    float dot[KPG][HN];
 #pragma unroll
-      for (int h = 0; h < HN; ++h) dot[h] = 0.f;
-      for (uint32_t c = l8 * 8; c < d8; c += 64) {
-        float k[8];
-        load8(kr + c, k);
+    for (int e = 0; e < KPG; ++e) {
+      const uint32_t t = grp + e * 32;
+      krow[e] = keys.row(t0 + (t < n ? t : 0));
 #pragma unroll
-        for (int h = 0; h < HN; ++h) {
-          const float4 qa = *reinterpret_cast<const float4 *>(sq + h * d8 + c), qb = *reinterpret_cast<const float4 *>(sq + h * d8 + c + 4);
-          dot[h] = fmaf(k[0], qa.x, fmaf(k[1], qa.y, fmaf(k[2], qa.z, fmaf(k[3], qa.w, dot[h]))));
-          dot[h] = fmaf(k[4], qb.x, fmaf(k[5], qb.y, fmaf(k[6], qb.z, fmaf(k[7], qb.w, dot[h]))));
-        }
-      }
-      float mine = 0.f;
+      for (int h = 0; h < HN; ++h) dot[e][h] = 0.f;
+    }
+    for (uint32_t c = l8 * 8; c < d8; c += 64) {
+      float k[KPG][8];
+#pragma unroll
+      for (int e = 0; e < KPG; ++e) load8(kc + (size_t)krow[e] * d8 + c, k[e]);
 #pragma unroll
       for (int h = 0; h < HN; ++h) {
-        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 1);
-        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 2);
-        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 4);
-        if (l8 == (uint32_t)h) mine = dot[h];
+        const float4 qa = *reinterpret_cast<const float4 *>(sq + h * d8 + c), qb = *reinterpret_cast<const float4 *>(sq + h * d8 + c + 4);
+#pragma unroll
+        for (int e = 0; e < KPG; ++e) {
+          float x = dot[e][h];
+          x = fmaf(k[e][0], qa.x, fmaf(k[e][1], qa.y, fmaf(k[e][2], qa.z, fmaf(k[e][3], qa.w, x))));
+          dot[e][h] = fmaf(k[e][4], qb.x, fmaf(k[e][5], qb.y, fmaf(k[e][6], qb.z, fmaf(k[e][7], qb.w, x))));
+        }
       }
-      if (l8 < hn) sp[l8 * WR_KEYS + e] = on ? score(a, h0 + l8, mine, i - j) : -INFINITY;
+    }
+#pragma unroll
+    for (int e = 0; e < KPG; ++e)
+#pragma unroll
+      for (int h = 0; h < HN; ++h) {
+        float x = dot[e][h];
+        x += __shfl_xor_sync(0xffffffffu, x, 1);
+        x += __shfl_xor_sync(0xffffffffu, x, 2);
+        dot[e][h] = x + __shfl_xor_sync(0xffffffffu, x, 4);
+      }
+    // the group's KPG * HN scores are finished by its eight lanes
+#pragma unroll
+    for (int r = 0; r < (KPG * HN + 7) / 8; ++r) {
+      const uint32_t id = l8 + 8 * r, e = id / HN, h = id % HN;
+      float mine = 0.f;
+#pragma unroll
+      for (int x = 0; x < KPG * HN; ++x)
+        if (id == (uint32_t)x) mine = dot[x / HN][x % HN];
+      const uint32_t t = grp + e * 32;
+      if (id < (uint32_t)(KPG * HN) && h < hn) sp[h * WR_KEYS + t] = t < n ? score(a, h0 + h, mine, i - keys.position(t0 + t)) : -INFINITY;
     }
     __syncthreads();
     if (warp < (int)hn) {
       float *s = sp + warp * WR_KEYS;
-      const float a0 = s[lane], a1 = s[lane + 32], old = sm[warp];
-      const float mx = fmaxf(old, warp_max(fmaxf(a0, a1)));
-      const float p0 = expf(a0 - mx), p1 = expf(a1 - mx), f = expf(old - mx);
-      s[lane] = p0;
-      s[lane + 32] = p1;
-      const float sum = warp_sum(p0 + p1);
+      const float old = sm[warp];
+      float x[KPG], mx = old, sum = 0.f;
+#pragma unroll
+      for (int e = 0; e < KPG; ++e) {
+        x[e] = s[lane + 32 * e];
+        mx = fmaxf(mx, x[e]);
+      }
+      mx = warp_max(mx);
+      const float f = expf(old - mx);
+#pragma unroll
+      for (int e = 0; e < KPG; ++e) {
+        x[e] = expf(x[e] - mx);
+        s[lane + 32 * e] = x[e];
+        sum += x[e];
+      }
+      sum = warp_sum(sum);
       __syncwarp();
       if (lane == 0) {
         sm[warp] = mx;
@@ -261,9 +372,9 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
           acc[h][0] *= sf[h];
           acc[h][1] *= sf[h];
         }
-#pragma unroll 4
+#pragma unroll 8
       for (uint32_t e = kg; e < n; e += KG) {
-        const float2 v = load2(vc + (size_t)cache_row(a, position(t0 + e)) * v8 + pr * 2);
+        const float2 v = load2(vc + (size_t)keys.row(t0 + e) * v8 + pr * 2);
 #pragma unroll
         for (int h = 0; h < HN; ++h) {
           const float p = sp[h * WR_KEYS + e];
@@ -377,16 +488,15 @@ __global__ void __launch_bounds__(WM_THREADS) window_mma_kernel(const __grid_con
     const float2 q = *reinterpret_cast<const float2 *>(q_in + ((size_t)(m0 + r) * a.heads + h) * d8 + 2 * c);
     *reinterpret_cast<uint32_t *>(qs + (size_t)r * ROWP + c * 4) = half2_bits(q.x, q.y);
   }
-  const uint32_t lo = a.window && i0 + 1 > a.window ? i0 + 1 - a.window : 0, kept = min(a.keep_first, lo), total = kept + (i1 - lo + 1);
-  const uint32_t ntiles = (total + WM_K - 1) / WM_K;
-  auto position = [&](uint32_t t) { return t < kept ? t : lo + (t - kept); };
+  const KeyList keys(a, i0, i1);
+  const uint32_t total = keys.total, ntiles = (total + WM_K - 1) / WM_K;
   auto stage = [&](uint32_t t, int buf) {
     if (t < ntiles) {
       const uint32_t kchunks = d8 / 8, per = kchunks + v8 / 8;
       for (uint32_t e = threadIdx.x; e < WM_K * per; e += WM_THREADS) {
         const uint32_t r = e / per, c = e % per, idx = t * WM_K + r;
         const bool on = idx < total;
-        const uint32_t cr = cache_row(a, position(on ? idx : 0));
+        const uint32_t cr = keys.row(on ? idx : 0);
         if (c < kchunks)
           cp16z(kt + (size_t)(buf * WM_K + r) * ROWP + c * 16, kc + (size_t)cr * d8 + c * 8, on);
         else
@@ -436,7 +546,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_mma_kernel(const __grid_con
     for (int n = 0; n < WM_K / 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const uint32_t idx = t * WM_K + n * 8 + 2 * tq + (e & 1), j = position(idx), i = qi[e >> 1];
+        const uint32_t idx = t * WM_K + n * 8 + 2 * tq + (e & 1), j = keys.position(idx), i = qi[e >> 1];
         float z = s[n][e] * c1;
         if (cap) z = cap2 - 2.f * cap2 * rcp(1.f + ex2(z));
         if (bias) z -= r1 * lg2(1.f + r2 * (float)(int)(i - j));
@@ -513,6 +623,32 @@ int check_win(const char *what, const greta_window_attn *a, const greta_rows *r)
   return GRETA_OK;
 }
 
+template <typename CT, int TAPS>
+int launch_conv_taps(cudaStream_t s, const WinArgs &w, float *q) {
+  const uint32_t d = std::max(w.a.dim, w.a.vdim);
+  const dim3 grid((w.a.heads + 2 * w.a.kv_heads + 7) / 8, (w.rows.M + CV_ROWS - 1) / CV_ROWS);
+  if (d <= 64)
+    GRETA_CUDA_TRY(launch_pdl(conv_norm_kernel<CT, TAPS, 2>, grid, dim3(256), 0, s, w, q));
+  else if (d <= 128)
+    GRETA_CUDA_TRY(launch_pdl(conv_norm_kernel<CT, TAPS, 4>, grid, dim3(256), 0, s, w, q));
+  else
+    GRETA_CUDA_TRY(launch_pdl(conv_norm_kernel<CT, TAPS, 8>, grid, dim3(256), 0, s, w, q));
+  return launched("conv_norm_kernel");
+}
+template <typename CT>
+int launch_conv(cudaStream_t s, const WinArgs &w, float *q) {
+  switch (w.a.conv ? w.a.taps : 0) {
+    case 0: return launch_conv_taps<CT, 0>(s, w, q);
+    case 1: return launch_conv_taps<CT, 1>(s, w, q);
+    case 2: return launch_conv_taps<CT, 2>(s, w, q);
+    case 3: return launch_conv_taps<CT, 3>(s, w, q);
+    case 4: return launch_conv_taps<CT, 4>(s, w, q);
+    default: break;
+  }
+  GRETA_CUDA_TRY(launch_pdl(conv_norm_any_kernel<CT>, dim3((w.a.heads + 2 * w.a.kv_heads + 7) / 8, w.rows.M), dim3(256), 0, s, w, q));
+  return launched("conv_norm_any_kernel");
+}
+
 template <typename CT, int HN, bool FUSED>
 int launch_rows(cudaStream_t s, const WinArgs &w, const float *q, void *out, int out_fmt, uint32_t ld_out, uint32_t splits) {
   const greta_window_attn &a = w.a;
@@ -533,7 +669,9 @@ int launch_rows(cudaStream_t s, const WinArgs &w, const float *q, void *out, int
 }
 template <typename CT, bool FUSED>
 int pick_heads(cudaStream_t s, const WinArgs &w, const float *q, void *out, int out_fmt, uint32_t ld_out, uint32_t splits) {
-  const uint32_t HG = w.a.heads / w.a.kv_heads;
+  // heads per CTA: all that share a key/value head, fewer where the grid would leave SMs idle
+  uint32_t HG = w.a.heads / w.a.kv_heads;
+  while (HG > 1 && (uint64_t)w.rows.M * w.a.kv_heads * splits * ((w.a.heads / w.a.kv_heads + HG / 2 - 1) / (HG / 2)) <= 160) HG /= 2;
   if (HG == 1) return launch_rows<CT, 1, FUSED>(s, w, q, out, out_fmt, ld_out, splits);
   if (HG == 2) return launch_rows<CT, 2, FUSED>(s, w, q, out, out_fmt, ld_out, splits);
   if (HG <= 4) return launch_rows<CT, 4, FUSED>(s, w, q, out, out_fmt, ld_out, splits);
@@ -564,12 +702,7 @@ int greta_cuda_window_attn_prepare(greta_stream_t stream, const greta_window_att
                 "window_attn_prepare: a portion of %u rows does not fit a ring of %u rows behind a window of %u", rows->M, a->ring, a->window);
   const WinArgs w{*a, *rows};
   cudaStream_t s = (cudaStream_t)stream;
-  const dim3 grid((a->heads + 2 * a->kv_heads + 7) / 8, rows->M);
-  if (a->cache_fmt == GRETA_FMT_F16)
-    GRETA_CUDA_TRY(launch_pdl(conv_norm_kernel<__half>, grid, dim3(256), 0, s, w, q_out));
-  else
-    GRETA_CUDA_TRY(launch_pdl(conv_norm_kernel<float>, grid, dim3(256), 0, s, w, q_out));
-  if (int rc = launched("conv_norm_kernel")) return rc;
+  if (int rc = a->cache_fmt == GRETA_FMT_F16 ? launch_conv<__half>(s, w, q_out) : launch_conv<float>(s, w, q_out)) return rc;
   if (!a->conv) return GRETA_OK;
   const uint32_t C = (a->heads + a->kv_heads) * a->dim + a->kv_heads * a->vdim;
   GRETA_CUDA_TRY(launch_pdl(conv_history_kernel, dim3((C + 255) / 256, std::min(rows->M, a->taps)), dim3(256), 0, s, w));
@@ -582,10 +715,10 @@ int greta_cuda_window_attn(greta_stream_t stream, const greta_window_attn *a, co
   GRETA_REQUIRE(out && max_len && (q || (rows->d_pos && a->proj)), "window_attn: null pointer");
   const WinArgs w{*a, *rows};
   cudaStream_t s = (cudaStream_t)stream;
-  // CTAs per row: enough to fill the GPU, at least two key tiles each, at most a portable cluster
+  // CTAs per row: enough to fill the GPU, at least 64 keys each, at most a portable cluster
   const uint32_t keys = a->window ? std::min(max_len, a->keep_first + a->window) : max_len;
   uint32_t splits = 1;
-  while (splits < 8 && (uint64_t)rows->M * a->kv_heads * splits < 148 && keys > splits * 2 * WR_KEYS) splits *= 2;
+  while (splits < 8 && (uint64_t)rows->M * a->kv_heads * splits < 148 && keys > splits * 64) splits *= 2;
   if (a->cache_fmt == GRETA_FMT_F16)
     return q ? pick_heads<__half, false>(s, w, q, out, out_fmt, ld_out, splits) : pick_heads<__half, true>(s, w, q, out, out_fmt, ld_out, splits);
   return q ? pick_heads<float, false>(s, w, q, out, out_fmt, ld_out, splits) : pick_heads<float, true>(s, w, q, out, out_fmt, ld_out, splits);

@@ -113,7 +113,7 @@ def test_linear_segments_activations_and_formats(g, gemm, fmt):
 def test_linear_gemm_tiles_and_residual(g, M):
     """Every token-tile width, several tiles per CTA, K that is no multiple of a stage, sums added to what is there."""
     rng = np.random.default_rng(M)
-    for N, K in ((20000, 100), (4000, 264), (300, 520)):
+    for N, K in ((20000, 100), (4000, 264), (300, 520), (200, 2100), (700, 1100)):
         W, x = bf16_round(rng.normal(0, 1 / np.sqrt(K), (N, K))), bf16_round(rng.normal(size=(M, K)))
         resid = rng.normal(size=(M, N)).astype(np.float32)
         got = run_linear(g, W, x, g.FMT_BF16, [(N, 0, None, g.OUT_F32)], True, resid=resid)[0]
