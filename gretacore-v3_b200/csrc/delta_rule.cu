@@ -178,22 +178,20 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
     if (c < chunks) {
       const uint32_t t0 = c * TC, n = min((uint32_t)TC + 1, T - t0);
       float *b = sm + (c % 3) * BUF;
-      const uint32_t unit = vec ? 4 : 1, per = D / unit, vper = vec ? vcols / 4 : vcols, tok = 4 * per + vper;
       for (uint32_t t = pw; t < n; t += C::PW) {
         const size_t m = t0 + t, at = m * d.ld + (size_t)h * D;
         float *dst = b + t * ROW;
-        for (uint32_t j = lane; j < tok; j += 32) {
-          const uint32_t which = j < 4 * per ? j / per : 4, e = (j - which * per) * unit;
-          const float *src = which == 0 ? d.decay + m * d.ld_decay + (size_t)h * D
-                             : which == 1 ? d.k + at
-                             : which == 2 ? d.a + at
-                             : which == 3 ? d.r + at
-                                          : d.v + at + c0;
-          float *to = dst + (which < 4 ? which * DP : 5 * DP) + e;
-          if (vec)
-            cp16(to, src + e);
-          else
-            cp4(to, src + e);
+        const float *src[4] = {d.decay + m * d.ld_decay + (size_t)h * D, d.k + at, d.a + at, d.r + at};
+        if (vec) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            for (uint32_t e = lane * 4; e < D; e += 128) cp16(dst + i * DP + e, src[i] + e);
+          if (lane * 4 < (int)vcols) cp16(dst + 5 * DP + lane * 4, d.v + at + c0 + lane * 4);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            for (uint32_t e = lane; e < D; e += 32) cp4(dst + i * DP + e, src[i] + e);
+          if (lane < (int)vcols) cp4(dst + 5 * DP + lane, d.v + at + c0 + lane);
         }
       }
     }
@@ -203,8 +201,12 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
     if (c >= chunks) return;
     const int n = (int)min((uint32_t)TC, T - c * TC);
     float *b = sm + (c % 3) * BUF;
-    for (int t = pw; t < n; t += C::PW) {
+    for (int t = pw; t < TC; t += C::PW) {
       float *row = b + t * ROW;
+      if (t >= n) {  // past the end of the portion: a token that leaves the state as it is
+        for (int e = lane; e < 5 * DP + COLS + 4; e += 32) row[e] = e < DP ? 1.f : 0.f;
+        continue;
+      }
       float k[RB], kk = 0.f, next_k = 0.f, next_ak = 0.f;
 #pragma unroll
       for (int i = 0; i < RB; ++i) {
@@ -284,47 +286,59 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
     } else {
       const float *b = sm + (ch % 3) * BUF;
       float *out = so + (ch & 1) * TC * COLS;
-      const int n = (int)min((uint32_t)TC, T - ch * TC);
-#pragma unroll 2
-      for (int t = 0; t < n; ++t) {
-        const float *row = b + t * ROW;
-        f32x2 x[NC], o[NC], v2[NC], nc2[NC];
-        float v[NC];
+#pragma unroll 1
+      for (int t8 = 0; t8 < TC; t8 += 8) {  // eight tokens of straight-line code; their outputs leave together
+        float o[NC][8];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-          v[c] = row[5 * DP + grp * NC + c];
-          v2[c] = pack2(v[c], v[c]);
-          nc2[c] = pack2(nc[c], nc[c]);
-          x[c] = o[c] = 0ull;
-        }
-#pragma unroll
-        for (int i = 0; i < RB; ++i) {
-          const ulonglong2 kw = lds2(row + 4 * DP + i * 32 + l8 * 4);
+        for (int j = 0; j < 8; ++j) {
+          const float *row = b + (t8 + j) * ROW;
+          f32x2 x[NC], y[NC], v2[NC], nc2[NC];
+          float v[NC];
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
-            x[c] = fma2(kw.x, s[c][2 * i], x[c]);
-            x[c] = fma2(kw.y, s[c][2 * i + 1], x[c]);
+            v[c] = row[5 * DP + grp * NC + c];
+            v2[c] = pack2(v[c], v[c]);
+            nc2[c] = pack2(nc[c], nc[c]);
+            x[c] = y[c] = 0ull;
           }
-        }
 #pragma unroll
-        for (int i = 0; i < RB; ++i) {
-          const int at = i * 32 + l8 * 4;
-          const ulonglong2 w = lds2(row + at), k = lds2(row + DP + at), ak = lds2(row + 2 * DP + at), r = lds2(row + 3 * DP + at);
+          for (int i = 0; i < RB; ++i) {
+            const ulonglong2 kw = lds2(row + 4 * DP + i * 32 + l8 * 4);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              x[c] = fma2(kw.x, s[c][2 * i], x[c]);
+              x[c] = fma2(kw.y, s[c][2 * i + 1], x[c]);
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < RB; ++i) {
+            const int at = i * 32 + l8 * 4;
+            const ulonglong2 w = lds2(row + at), k = lds2(row + DP + at), ak = lds2(row + 2 * DP + at), r = lds2(row + 3 * DP + at);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              s[c][2 * i] = fma2(ak.x, nc2[c], fma2(k.x, v2[c], mul2(w.x, s[c][2 * i])));
+              s[c][2 * i + 1] = fma2(ak.y, nc2[c], fma2(k.y, v2[c], mul2(w.y, s[c][2 * i + 1])));
+              y[c] = fma2(r.x, s[c][2 * i], y[c]);
+              y[c] = fma2(r.y, s[c][2 * i + 1], y[c]);
+            }
+          }
+          const float2 nx = *reinterpret_cast<const float2 *>(row + 5 * DP + COLS);
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
-            s[c][2 * i] = fma2(w.x, s[c][2 * i], fma2(k.x, v2[c], mul2(ak.x, nc2[c])));
-            s[c][2 * i + 1] = fma2(w.y, s[c][2 * i + 1], fma2(k.y, v2[c], mul2(ak.y, nc2[c])));
-            o[c] = fma2(r.x, s[c][2 * i], o[c]);
-            o[c] = fma2(r.y, s[c][2 * i + 1], o[c]);
+            nc[c] = -(sum8(sum_halves(x[c])) + fmaf(nx.y, nc[c], nx.x * v[c]));
+            o[c][j] = sum_halves(y[c]);
           }
         }
-        const float2 nx = *reinterpret_cast<const float2 *>(row + 5 * DP + COLS);
+        // lane j of the group receives the total of token t8 + j: halves of the tokens change places three times
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-          const float ahead = sum8(sum_halves(x[c]));
-          nc[c] = -fmaf(nx.y, nc[c], fmaf(nx.x, v[c], ahead));
-          const float y = sum8(sum_halves(o[c]));
-          if (l8 == c) out[t * COLS + grp * NC + c] = y;
+          float q4[4], q2[2];
+          const bool b4 = l8 & 4, b2 = l8 & 2, b1 = l8 & 1;
+#pragma unroll
+          for (int j = 0; j < 4; ++j) q4[j] = (b4 ? o[c][j + 4] : o[c][j]) + __shfl_xor_sync(0xffffffffu, b4 ? o[c][j] : o[c][j + 4], 4);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) q2[j] = (b2 ? q4[j + 2] : q4[j]) + __shfl_xor_sync(0xffffffffu, b2 ? q4[j] : q4[j + 2], 2);
+          out[(t8 + l8) * COLS + grp * NC + c] = (b1 ? q2[1] : q2[0]) + __shfl_xor_sync(0xffffffffu, b1 ? q2[0] : q2[1], 1);
         }
       }
     }

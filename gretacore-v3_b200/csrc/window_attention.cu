@@ -88,11 +88,37 @@ __device__ __forceinline__ float conv_channel(const greta_window_attn &a, uint32
 __device__ __forceinline__ void conv_head(const greta_window_attn &a, uint32_t m, uint32_t slot, uint32_t p, uint32_t first, uint32_t c0, uint32_t d,
                                           bool norm, int lane, float (&v)[8]) {
   float q = 0.f;
+  if (a.conv && a.taps <= 4) {  // all loads in flight before the first is used
+    const uint32_t C = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
+    float u[8][4], cw[8][4];
+    const float *past[4];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const uint32_t c = lane + 32 * i;
-    v[i] = c < d ? conv_channel(a, m, slot, p, first, c0 + c) : 0.f;
-    q = fmaf(v[i], v[i], q);
+    for (int back = 0; back < 4; ++back) {
+      const bool on = back < (int)a.taps && back <= (int)p;
+      const uint32_t at = p - back;
+      past[back] = !on ? nullptr : at >= first ? a.proj + (size_t)(m - back) * a.ld_proj + c0 : a.history + ((size_t)slot * a.taps + at % a.taps) * C + c0;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int back = 0; back < 4; ++back) {
+        const uint32_t c = lane + 32 * i;
+        const bool on = c < d && past[back];
+        u[i][back] = on ? past[back][c] : 0.f;
+        cw[i][back] = on ? a.conv[(size_t)(c0 + c) * a.taps + a.taps - 1 - back] : 0.f;
+      }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      v[i] = fmaf(cw[i][0], u[i][0], fmaf(cw[i][1], u[i][1], fmaf(cw[i][2], u[i][2], cw[i][3] * u[i][3])));
+      q = fmaf(v[i], v[i], q);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const uint32_t c = lane + 32 * i;
+      v[i] = c < d ? conv_channel(a, m, slot, p, first, c0 + c) : 0.f;
+      q = fmaf(v[i], v[i], q);
+    }
   }
   if (norm) {
     const float inv = 1.f / sqrtf(warp_sum(q) / (float)d + a.eps);
@@ -245,6 +271,14 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   const uint32_t rows = a.keep_first + a.ring;
   const CT *kc = static_cast<const CT *>(a.k_cache) + ((size_t)slot * a.kv_heads + g) * rows * d8;
   const CT *vc = static_cast<const CT *>(a.v_cache) + ((size_t)slot * a.kv_heads + g) * rows * v8;
+  {  // this CTA's keys and values start their way to L2
+    const uint32_t kl = (d8 * (uint32_t)sizeof(CT) + 127) / 128, vl = (v8 * (uint32_t)sizeof(CT) + 127) / 128;
+    for (uint32_t e = threadIdx.x; e < (t_end - t_begin) * (kl + vl); e += WR_THREADS) {
+      const uint32_t r = keys.row(t_begin + e / (kl + vl)), l = e % (kl + vl);
+      const char *p = l < kl ? reinterpret_cast<const char *>(kc + (size_t)r * d8) + l * 128 : reinterpret_cast<const char *>(vc + (size_t)r * v8) + (l - kl) * 128;
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(p));
+    }
+  }
   if (FUSED) {
     const uint32_t C = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
     float *hist = a.conv ? a.history + ((size_t)slot * a.taps + i % a.taps) * C : nullptr;
