@@ -5,11 +5,13 @@
 // so eight lanes hold one column in registers (row i * 32 + lane8 * 4 + e in register 4 i + e) and a step is two dot
 // products over eight lanes and one update.  Rows past dim are padding: every vector is zero there, so they stay zero.
 //
-// The scan looks one token ahead so that no step waits for a reduction it has just started: with S' the state before token t,
-//   k'^T S_j = (k' * w)^T S'_j + (k'.k) v_j - (k'.ak) c_j      (k' the next token's key)
-// and the first term needs only S', one step earlier than the state it belongs to.  Producer warps stage the tokens' vectors
-// (cp.async), derive ak, k' * w and the two scalars, and write the outputs back, one chunk ahead of and behind the warps that
-// hold the state.
+// The scan takes four tokens at a time, so that one reduction serves four tokens.  With W(a..b) the product of the decays of
+// tokens a..b of such a block (0..3) and S the state before it,
+//   c_i = (k_i W(0..i-1))^T S_j + sum_{j<i} P_ij v_j - Q_ij c_j          P, Q: (k_i W(j+1..i-1)) . k_j, ... . ak_j
+//   o_i = (r_i W(0..i))^T S_j   + sum_{j<=i} R_ij v_j - T_ij c_j         R, T: (r_i W(j+1..i)) . k_j, ... . ak_j
+//   S_j <- W(0..3) S_j + sum_i (k_i W(i+1..3)) v_i - (ak_i W(i+1..3)) c_i
+// The 17 vectors and 32 scalars of a block are the same for every column; producer warps derive them from the staged
+// tokens one chunk ahead of the warps that hold the state.  No decay is ever divided by.
 #include <algorithm>
 
 #include "dense_device.cuh"
@@ -145,23 +147,43 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 __device__ __forceinline__ ulonglong2 lds2(const float *p) { return *reinterpret_cast<const ulonglong2 *>(p); }
 
 // The recurrence over a portion: grid (heads, column groups).  A CTA keeps 32 columns of one head in the registers of its
-// first warps, NC columns per group of eight lanes, and walks the tokens in chunks of TC; three chunk buffers rotate.
+// first warps, NC columns per group of eight lanes, and walks the tokens in chunks of TC = a block per producer warp.
 template <int RB, int NC>
 struct ScanCfg {
   static constexpr int DP = RB * 32, COLS = 32;
-  static constexpr int TC = RB <= 4 ? 16 : 8;
-  static constexpr int ROW = 5 * DP + COLS + 4;   // floats of a staged token: w, k, ak, r, k' * w, v, {k'.k, k'.ak}
-  static constexpr int BUF = (TC + 1) * ROW;      // one more token: its key is the last one's k'
+  static constexpr int TC = RB <= 4 ? 16 : 8, NB = TC / 4;
+  static constexpr int RAW_ROW = 4 * DP + COLS, RAW = TC * RAW_ROW;   // a staged token: w, k, a, r, v
+  static constexpr int SCAL = 17 * DP, VT = SCAL + 48;                // of a block: 17 vectors, {P, -Q | R | -T}, v [column][4]
+  static constexpr int BLK = VT + 4 * COLS, DER = NB * BLK;
   static constexpr int CW = COLS / (4 * NC), PW = 4, THREADS = (CW + PW) * 32;
-  static constexpr size_t SMEM = (size_t)(3 * BUF + 2 * TC * COLS) * 4;
+  static constexpr size_t SMEM = (size_t)(2 * RAW + 2 * DER + 2 * TC * COLS) * 4;
   static_assert(SMEM <= 232448, "chunk buffers exceed shared memory");
 };
+// Four values over the eight lanes of a group: lane l8 receives the total of value l8 >> 1.
+__device__ __forceinline__ float sum8_of4(const float (&v)[4], int l8) {
+  const bool b4 = l8 & 4, b2 = l8 & 2;
+  const float p0 = (b4 ? v[2] : v[0]) + __shfl_xor_sync(0xffffffffu, b4 ? v[0] : v[2], 4);
+  const float p1 = (b4 ? v[3] : v[1]) + __shfl_xor_sync(0xffffffffu, b4 ? v[1] : v[3], 4);
+  const float q = (b2 ? p1 : p0) + __shfl_xor_sync(0xffffffffu, b2 ? p0 : p1, 2);
+  return q + __shfl_xor_sync(0xffffffffu, q, 1);
+}
+// 32 values over the 32 lanes of a warp: lane l receives the total of value l.
+__device__ __forceinline__ float sum32_of32(float (&v)[32], int lane) {
+#pragma unroll
+  for (int n = 16; n >= 1; n >>= 1) {
+    const bool up = lane & n;
+#pragma unroll
+    for (int j = 0; j < n; ++j) v[j] = (up ? v[j + n] : v[j]) + __shfl_xor_sync(0xffffffffu, up ? v[j] : v[j + n], n);
+  }
+  return v[0];
+}
+
 template <int RB, int NC>
 __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(const __grid_constant__ DeltaArgs a, float *__restrict__ o_buf, int vec) {
   using C = ScanCfg<RB, NC>;
-  constexpr int DP = C::DP, TC = C::TC, ROW = C::ROW, COLS = C::COLS, BUF = C::BUF;
+  constexpr int DP = C::DP, TC = C::TC, COLS = C::COLS;
   extern __shared__ __align__(16) float sm[];
-  float *so = sm + 3 * BUF;  // [2][TC][COLS]
+  float *derived = sm + 2 * C::RAW, *so = derived + 2 * C::DER;  // so: [2][TC][COLS]
   const greta_delta_rule &d = a.d;
   const uint32_t h = blockIdx.x, c0 = blockIdx.y * COLS, D = d.dim, T = a.rows.M;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
@@ -169,71 +191,99 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
   const int pw = warp - C::CW;
   const uint32_t vcols = min((uint32_t)COLS, D - c0), chunks = (T + TC - 1) / TC;
   float *state = d.state + ((size_t)a.rows.slot0 * d.heads + h) * D * DP;
-  for (int i = threadIdx.x; i < 3 * BUF; i += C::THREADS) sm[i] = 0.f;
+  for (int i = threadIdx.x; i < 2 * C::RAW + 2 * C::DER; i += C::THREADS) sm[i] = 0.f;
   pdl_launch_dependents();
   pdl_wait();
   __syncthreads();
 
-  auto stage = [&](uint32_t c) {  // producer warps: the chunk's tokens and one more
+  auto stage = [&](uint32_t c) {  // producer warps
     if (c < chunks) {
-      const uint32_t t0 = c * TC, n = min((uint32_t)TC + 1, T - t0);
-      float *b = sm + (c % 3) * BUF;
+      const uint32_t t0 = c * TC, n = min((uint32_t)TC, T - t0);
+      float *b = sm + (c & 1) * C::RAW;
       for (uint32_t t = pw; t < n; t += C::PW) {
         const size_t m = t0 + t, at = m * d.ld + (size_t)h * D;
-        float *dst = b + t * ROW;
+        float *dst = b + t * C::RAW_ROW;
         const float *src[4] = {d.decay + m * d.ld_decay + (size_t)h * D, d.k + at, d.a + at, d.r + at};
         if (vec) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
             for (uint32_t e = lane * 4; e < D; e += 128) cp16(dst + i * DP + e, src[i] + e);
-          if (lane * 4 < (int)vcols) cp16(dst + 5 * DP + lane * 4, d.v + at + c0 + lane * 4);
+          if (lane * 4 < (int)vcols) cp16(dst + 4 * DP + lane * 4, d.v + at + c0 + lane * 4);
         } else {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
             for (uint32_t e = lane; e < D; e += 32) cp4(dst + i * DP + e, src[i] + e);
-          if (lane < (int)vcols) cp4(dst + 5 * DP + lane, d.v + at + c0 + lane);
+          if (lane < (int)vcols) cp4(dst + 4 * DP + lane, d.v + at + c0 + lane);
         }
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  auto prepare = [&](uint32_t c) {  // producer warps, once the chunk has landed: ak, k' * w, k'.k, k'.ak
-    if (c >= chunks) return;
-    const int n = (int)min((uint32_t)TC, T - c * TC);
-    float *b = sm + (c % 3) * BUF;
-    for (int t = pw; t < TC; t += C::PW) {
-      float *row = b + t * ROW;
-      if (t >= n) {  // past the end of the portion: a token that leaves the state as it is
-        for (int e = lane; e < 5 * DP + COLS + 4; e += 32) row[e] = e < DP ? 1.f : 0.f;
-        continue;
-      }
-      float k[RB], kk = 0.f, next_k = 0.f, next_ak = 0.f;
-#pragma unroll
-      for (int i = 0; i < RB; ++i) {
-        k[i] = row[DP + i * 32 + lane];
-        kk = fmaf(k[i], k[i], kk);
-      }
-      const float inv2 = 1.f / (warp_sum(kk) + 1e-6f);
-#pragma unroll
-      for (int i = 0; i < RB; ++i) {
-        const int e = i * 32 + lane;
-        const float k1 = row[ROW + DP + e], ak = row[2 * DP + e] * k[i] * inv2;
-        row[2 * DP + e] = ak;
-        row[4 * DP + e] = k1 * row[e];
-        next_k = fmaf(k1, k[i], next_k);
-        next_ak = fmaf(k1, ak, next_ak);
-      }
-      next_k = warp_sum(next_k);
-      next_ak = warp_sum(next_ak);
-      if (lane == 0) {
-        row[5 * DP + COLS] = next_k;
-        row[5 * DP + COLS + 1] = next_ak;
-      }
-    }
-  };
   auto landed = [&]() {  // the chunk before the last one staged is complete for every producer
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     asm volatile("bar.sync 1, %0;" ::"n"(C::PW * 32) : "memory");
+  };
+  auto prepare = [&](uint32_t c) {  // producer warp pw: block pw of the chunk, once it has landed
+    if (c >= chunks || pw >= C::NB) return;
+    const int n = (int)min((uint32_t)TC, T - c * TC) - pw * 4;  // tokens of the block that exist; the others leave the state as it is
+    const float *raw = sm + (c & 1) * C::RAW + pw * 4 * C::RAW_ROW;
+    float *der = derived + (c & 1) * C::DER + pw * C::BLK;
+    float inv2[4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      float kk = 0.f;
+#pragma unroll
+      for (int i = 0; i < RB; ++i) {
+        const float k = raw[t * C::RAW_ROW + DP + i * 32 + lane];
+        kk = fmaf(k, k, kk);
+      }
+      inv2[t] = kk;
+    }
+#pragma unroll
+    for (int t = 0; t < 4; ++t) inv2[t] = 1.f / (warp_sum(inv2[t]) + 1e-6f);
+    float acc[32];
+#pragma unroll
+    for (int j = 0; j < 32; ++j) acc[j] = 0.f;
+#pragma unroll
+    for (int i = 0; i < RB; ++i) {
+      const int e = i * 32 + lane;
+      float w[4], k[4], ak[4], r[4];
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        const float *row = raw + t * C::RAW_ROW + e;
+        const bool on = t < n;
+        w[t] = on ? row[0] : 1.f;
+        k[t] = on ? row[DP] : 0.f;
+        ak[t] = on ? row[2 * DP] * k[t] * inv2[t] : 0.f;
+        r[t] = on ? row[3 * DP] : 0.f;
+      }
+      const float w01 = w[0] * w[1], w12 = w[1] * w[2], w23 = w[2] * w[3], w02 = w01 * w[2], w13 = w12 * w[3];
+      float *o = der + e;
+      o[0] = k[0], o[DP] = k[1] * w[0], o[2 * DP] = k[2] * w01, o[3 * DP] = k[3] * w02;
+      o[4 * DP] = r[0] * w[0], o[5 * DP] = r[1] * w01, o[6 * DP] = r[2] * w02, o[7 * DP] = r[3] * (w02 * w[3]);
+      o[8 * DP] = w[0] * w13;
+      o[9 * DP] = k[0] * w13, o[10 * DP] = k[1] * w23, o[11 * DP] = k[2] * w[3], o[12 * DP] = k[3];
+      o[13 * DP] = -ak[0] * w13, o[14 * DP] = -ak[1] * w23, o[15 * DP] = -ak[2] * w[3], o[16 * DP] = -ak[3];
+      // left factors of the pairs (i, j): P, Q (1,0) (2,0) (2,1) (3,0) (3,1) (3,2); R, T (0,0) (1,0) (1,1) (2,0) .. (3,3)
+      const float pl[6] = {k[1], k[2] * w[1], k[2], k[3] * w12, k[3] * w[2], k[3]};
+      const float rl[10] = {r[0], r[1] * w[1], r[1], r[2] * w12, r[2] * w[2], r[2], r[3] * w13, r[3] * w23, r[3] * w[3], r[3]};
+      constexpr int pj[6] = {0, 0, 1, 0, 1, 2}, rj[10] = {0, 0, 1, 0, 1, 2, 0, 1, 2, 3};
+#pragma unroll
+      for (int x = 0; x < 6; ++x) {
+        acc[x] = fmaf(pl[x], k[pj[x]], acc[x]);
+        acc[6 + x] = fmaf(-pl[x], ak[pj[x]], acc[6 + x]);
+      }
+#pragma unroll
+      for (int x = 0; x < 10; ++x) {
+        acc[12 + x] = fmaf(rl[x], k[rj[x]], acc[12 + x]);
+        acc[22 + x] = fmaf(-rl[x], ak[rj[x]], acc[22 + x]);
+      }
+    }
+    const float total = sum32_of32(acc, lane);
+    const int x = lane < 12 ? 0 : (lane - 12) % 10, ri = x < 1 ? 0 : x < 3 ? 1 : x < 6 ? 2 : 3;  // upper triangles of R and T stay zero
+    der[C::SCAL + (lane < 12 ? lane : (lane < 22 ? 16 : 32) + ri * 4 + x - ri * (ri + 1) / 2)] = total;
+    const float *v = raw + 4 * DP + lane;
+    *reinterpret_cast<float4 *>(der + C::VT + lane * 4) = make_float4(v[0], v[C::RAW_ROW], v[2 * C::RAW_ROW], v[3 * C::RAW_ROW]);
   };
   auto write_back = [&](uint32_t c) {
     const uint32_t n = min((uint32_t)TC, T - c * TC);
@@ -244,7 +294,6 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
 
   const int grp = threadIdx.x >> 3;  // state warps: columns c0 + grp * NC ..
   f32x2 s[NC][2 * RB];
-  float nc[NC];
   if (producer) {
     stage(0);
     stage(1);
@@ -264,19 +313,6 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
     }
   }
   __syncthreads();
-  if (!producer) {  // the first token's c
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      f32x2 x = 0ull;
-#pragma unroll
-      for (int i = 0; i < RB; ++i) {
-        const ulonglong2 k = lds2(sm + DP + i * 32 + l8 * 4);
-        x = fma2(k.x, s[c][2 * i], x);
-        x = fma2(k.y, s[c][2 * i + 1], x);
-      }
-      nc[c] = -sum8(sum_halves(x));
-    }
-  }
   for (uint32_t ch = 0; ch < chunks; ++ch) {
     if (producer) {
       stage(ch + 2);
@@ -284,61 +320,79 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
       prepare(ch + 1);
       if (ch) write_back(ch - 1);
     } else {
-      const float *b = sm + (ch % 3) * BUF;
       float *out = so + (ch & 1) * TC * COLS;
 #pragma unroll 1
-      for (int t8 = 0; t8 < TC; t8 += 8) {  // eight tokens of straight-line code; their outputs leave together
-        float o[NC][8];
+      for (int blk = 0; blk < C::NB; ++blk) {
+        const float *b = derived + (ch & 1) * C::DER + blk * C::BLK;
+        float x[NC][4], o[NC][4];
+        {
+          f32x2 xs[NC][4], rs[NC][4];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const float *row = b + (t8 + j) * ROW;
-          f32x2 x[NC], y[NC], v2[NC], nc2[NC];
-          float v[NC];
+          for (int c = 0; c < NC; ++c)
 #pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            v[c] = row[5 * DP + grp * NC + c];
-            v2[c] = pack2(v[c], v[c]);
-            nc2[c] = pack2(nc[c], nc[c]);
-            x[c] = y[c] = 0ull;
-          }
+            for (int t = 0; t < 4; ++t) xs[c][t] = rs[c][t] = 0ull;
 #pragma unroll
-          for (int i = 0; i < RB; ++i) {
-            const ulonglong2 kw = lds2(row + 4 * DP + i * 32 + l8 * 4);
+          for (int i = 0; i < RB; ++i)
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-              x[c] = fma2(kw.x, s[c][2 * i], x[c]);
-              x[c] = fma2(kw.y, s[c][2 * i + 1], x[c]);
+            for (int t = 0; t < 4; ++t) {
+              const ulonglong2 k = lds2(b + t * DP + i * 32 + l8 * 4), r = lds2(b + (4 + t) * DP + i * 32 + l8 * 4);
+#pragma unroll
+              for (int c = 0; c < NC; ++c) {
+                xs[c][t] = fma2(k.y, s[c][2 * i + 1], fma2(k.x, s[c][2 * i], xs[c][t]));
+                rs[c][t] = fma2(r.y, s[c][2 * i + 1], fma2(r.x, s[c][2 * i], rs[c][t]));
+              }
             }
-          }
 #pragma unroll
-          for (int i = 0; i < RB; ++i) {
-            const int at = i * 32 + l8 * 4;
-            const ulonglong2 w = lds2(row + at), k = lds2(row + DP + at), ak = lds2(row + 2 * DP + at), r = lds2(row + 3 * DP + at);
+          for (int c = 0; c < NC; ++c)
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-              s[c][2 * i] = fma2(ak.x, nc2[c], fma2(k.x, v2[c], mul2(w.x, s[c][2 * i])));
-              s[c][2 * i + 1] = fma2(ak.y, nc2[c], fma2(k.y, v2[c], mul2(w.y, s[c][2 * i + 1])));
-              y[c] = fma2(r.x, s[c][2 * i], y[c]);
-              y[c] = fma2(r.y, s[c][2 * i + 1], y[c]);
+            for (int t = 0; t < 4; ++t) {
+              x[c][t] = sum_halves(xs[c][t]);
+              o[c][t] = sum_halves(rs[c][t]);
             }
-          }
-          const float2 nx = *reinterpret_cast<const float2 *>(row + 5 * DP + COLS);
-#pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            nc[c] = -(sum8(sum_halves(x[c])) + fmaf(nx.y, nc[c], nx.x * v[c]));
-            o[c][j] = sum_halves(y[c]);
-          }
         }
-        // lane j of the group receives the total of token t8 + j: halves of the tokens change places three times
+        // P10 P20 P21 P30 | P31 P32 -Q10 -Q20 | -Q21 -Q30 -Q31 -Q32
+        const float4 s0 = lds4(b + C::SCAL), s1 = lds4(b + C::SCAL + 4), s2 = lds4(b + C::SCAL + 8);
+        const float4 R = lds4(b + C::SCAL + 16 + (l8 >> 1) * 4), Tn = lds4(b + C::SCAL + 32 + (l8 >> 1) * 4);  // of this lane's token
+        float4 v[NC], cc[NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-          float q4[4], q2[2];
-          const bool b4 = l8 & 4, b2 = l8 & 2, b1 = l8 & 1;
+          v[c] = lds4(b + C::VT + (grp * NC + c) * 4);
+          const float q = sum8_of4(x[c], l8);
+          const int base = lane & 24;
+          cc[c].x = __shfl_sync(0xffffffffu, q, base);
+          cc[c].y = fmaf(s1.z, cc[c].x, fmaf(s0.x, v[c].x, __shfl_sync(0xffffffffu, q, base + 2)));
+          cc[c].z = fmaf(s2.x, cc[c].y, fmaf(s1.w, cc[c].x, fmaf(s0.z, v[c].y, fmaf(s0.y, v[c].x, __shfl_sync(0xffffffffu, q, base + 4)))));
+          const float p3 = fmaf(s1.y, v[c].z, fmaf(s1.x, v[c].y, fmaf(s0.w, v[c].x, __shfl_sync(0xffffffffu, q, base + 6))));
+          cc[c].w = fmaf(s2.w, cc[c].z, fmaf(s2.z, cc[c].y, fmaf(s2.y, cc[c].x, p3)));
+        }
 #pragma unroll
-          for (int j = 0; j < 4; ++j) q4[j] = (b4 ? o[c][j + 4] : o[c][j]) + __shfl_xor_sync(0xffffffffu, b4 ? o[c][j] : o[c][j + 4], 4);
+        for (int i = 0; i < RB; ++i) {
+          const int at = i * 32 + l8 * 4;
+          const ulonglong2 w = lds2(b + 8 * DP + at);
 #pragma unroll
-          for (int j = 0; j < 2; ++j) q2[j] = (b2 ? q4[j + 2] : q4[j]) + __shfl_xor_sync(0xffffffffu, b2 ? q4[j] : q4[j + 2], 2);
-          out[(t8 + l8) * COLS + grp * NC + c] = (b1 ? q2[1] : q2[0]) + __shfl_xor_sync(0xffffffffu, b1 ? q2[0] : q2[1], 1);
+          for (int c = 0; c < NC; ++c) {
+            s[c][2 * i] = mul2(w.x, s[c][2 * i]);
+            s[c][2 * i + 1] = mul2(w.y, s[c][2 * i + 1]);
+          }
+#pragma unroll
+          for (int t = 0; t < 4; ++t) {
+            const ulonglong2 k = lds2(b + (9 + t) * DP + at), ak = lds2(b + (13 + t) * DP + at);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              const float vt = t == 0 ? v[c].x : t == 1 ? v[c].y : t == 2 ? v[c].z : v[c].w;
+              const float ct = t == 0 ? cc[c].x : t == 1 ? cc[c].y : t == 2 ? cc[c].z : cc[c].w;
+              const f32x2 v2 = pack2(vt, vt), c2 = pack2(ct, ct);
+              s[c][2 * i] = fma2(ak.x, c2, fma2(k.x, v2, s[c][2 * i]));
+              s[c][2 * i + 1] = fma2(ak.y, c2, fma2(k.y, v2, s[c][2 * i + 1]));
+            }
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          float y = sum8_of4(o[c], l8);
+          y = fmaf(R.x, v[c].x, fmaf(R.y, v[c].y, fmaf(R.z, v[c].z, fmaf(R.w, v[c].w, y))));
+          y = fmaf(Tn.x, cc[c].x, fmaf(Tn.y, cc[c].y, fmaf(Tn.z, cc[c].z, fmaf(Tn.w, cc[c].w, y))));
+          if (!(l8 & 1)) out[(blk * 4 + (l8 >> 1)) * COLS + grp * NC + c] = y;
         }
       }
     }
@@ -422,14 +476,19 @@ int check_delta(const char *what, const greta_delta_rule *d, const greta_rows *r
 template <int RB, int NC>
 int launch_scan(cudaStream_t s, const DeltaArgs &a, float *o_buf, int vec) {
   using C = ScanCfg<RB, NC>;
+  // A grid that fits the SMs asks for more than half of an SM's shared memory: CTAs that become resident while the previous
+  // kernel drains would otherwise pair up on the SMs that fall idle first, and the pairs would set the pace.
+  constexpr size_t ALONE = 118 * 1024;
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-    GRETA_CUDA_TRY(cudaFuncSetAttribute(delta_scan_kernel<RB, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM));
+    GRETA_CUDA_TRY(cudaFuncSetAttribute(delta_scan_kernel<RB, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(C::SMEM, ALONE)));
     attr_set[dev] = true;
   }
-  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC>, dim3(a.d.heads, (a.d.dim + C::COLS - 1) / C::COLS), dim3(C::THREADS), C::SMEM, s, a, o_buf, vec));
+  const dim3 grid(a.d.heads, (a.d.dim + C::COLS - 1) / C::COLS);
+  const size_t smem = grid.x * grid.y <= (uint32_t)sm_count() ? std::max(C::SMEM, ALONE) : C::SMEM;
+  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC>, grid, dim3(C::THREADS), smem, s, a, o_buf, vec));
   return launched("delta_scan_kernel");
 }
 template <int RB>
@@ -474,8 +533,8 @@ int greta_cuda_delta_scan(greta_stream_t stream, const greta_delta_rule *d, cons
   const int vec = d->dim % 4 == 0 && d->ld % 4 == 0 && d->ld_decay % 4 == 0 && aligned16(d->r) && aligned16(d->k) && aligned16(d->v) && aligned16(d->a) &&
                   aligned16(d->decay);
   switch (dim32(d->dim) / 32) {
-    case 1: return launch_scan<1, 2>(s, a, o_buf, vec);
-    case 2: return launch_scan<2, 2>(s, a, o_buf, vec);
+    case 1: return launch_scan<1, 4>(s, a, o_buf, vec);
+    case 2: return launch_scan<2, 4>(s, a, o_buf, vec);
     case 3: return launch_scan<3, 2>(s, a, o_buf, vec);
     case 4: return launch_scan<4, 2>(s, a, o_buf, vec);
     case 5: return launch_scan<5, 1>(s, a, o_buf, vec);

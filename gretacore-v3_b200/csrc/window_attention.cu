@@ -64,8 +64,12 @@ __device__ __forceinline__ void load8(const float *p, float (&f)[8]) {
   const float4 a = *reinterpret_cast<const float4 *>(p), b = *reinterpret_cast<const float4 *>(p + 4);
   f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
 }
-__device__ __forceinline__ float2 load2(const __half *p) { return __half22float2(*reinterpret_cast<const __half2 *>(p)); }
-__device__ __forceinline__ float2 load2(const float *p) { return *reinterpret_cast<const float2 *>(p); }
+__device__ __forceinline__ float4 load4(const __half *p) {
+  const uint2 u = *reinterpret_cast<const uint2 *>(p);
+  const float2 a = h2_to_f2(u.x), b = h2_to_f2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
 
 // Convolved channel c of the token at position p, activation row m of the launch; rows of the launch that belong to the same
 // sequence start at position first.
@@ -244,7 +248,7 @@ __device__ __forceinline__ float score(const greta_window_attn &a, uint32_t h, f
   return s;
 }
 
-constexpr int WR_KEYS = 128, WR_THREADS = 256, KPG = WR_KEYS / 32;  // keys of a pass, keys per group of eight lanes
+constexpr int WR_KEYS = 256, WR_THREADS = 256, KPG = 4;  // keys of a pass; keys that a group of eight lanes has in flight
 
 // grid (splits, kv heads * head passes, rows), cluster (splits, 1, 1); HN query heads of one key/value head per CTA.
 template <typename CT, int HN, bool FUSED>
@@ -253,7 +257,7 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   const greta_window_attn &a = w.a;
   extern __shared__ __align__(16) float smem[];
   const uint32_t d8 = up8(a.dim), v8 = up8(a.vdim), HG = a.heads / a.kv_heads, passes = (HG + HN - 1) / HN;
-  const uint32_t pairs = v8 / 2, tpp = (pairs + 31) / 32 * 32, KG = WR_THREADS / tpp;
+  const uint32_t quads = v8 / 4, tpp = (quads + 31) / 32 * 32, KG = WR_THREADS / tpp;
   float *sq = smem;                          // [HN][d8]
   float *sp = sq + HN * d8;                  // [HN][WR_KEYS] scores, then weights
   float *so = sp + HN * WR_KEYS;             // [HN][v8] this CTA's unnormalised output
@@ -321,71 +325,73 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   __syncthreads();  // also: this CTA's cache row is visible to it
 
   const uint32_t pr = threadIdx.x % tpp, kg = threadIdx.x / tpp;
-  const bool pv = pr < pairs && kg < KG;
-  float acc[HN][2];
+  const bool pv = pr < quads && kg < KG;
+  float acc[HN][4];
 #pragma unroll
-  for (int h = 0; h < HN; ++h) acc[h][0] = acc[h][1] = 0.f;
+  for (int h = 0; h < HN; ++h) acc[h][0] = acc[h][1] = acc[h][2] = acc[h][3] = 0.f;
   for (uint32_t t0 = t_begin; t0 < t_end; t0 += WR_KEYS) {
     const uint32_t n = min((uint32_t)WR_KEYS, t_end - t0);
     const uint32_t l8 = threadIdx.x & 7, grp = threadIdx.x >> 3;  // 32 groups of 8 lanes, KPG keys each
-    uint32_t krow[KPG];
-    float dot[KPG][HN];
+    for (uint32_t part = 0; part < n; part += 32 * KPG) {
+      uint32_t krow[KPG];
+      float dot[KPG][HN];
 #pragma unroll
-    for (int e = 0; e < KPG; ++e) {
-      const uint32_t t = grp + e * 32;
-      krow[e] = keys.row(t0 + (t < n ? t : 0));
+      for (int e = 0; e < KPG; ++e) {
+        const uint32_t t = part + grp + e * 32;
+        krow[e] = keys.row(t0 + (t < n ? t : 0));
 #pragma unroll
-      for (int h = 0; h < HN; ++h) dot[e][h] = 0.f;
-    }
-    for (uint32_t c = l8 * 8; c < d8; c += 64) {
-      float k[KPG][8];
+        for (int h = 0; h < HN; ++h) dot[e][h] = 0.f;
+      }
+      for (uint32_t c = l8 * 8; c < d8; c += 64) {
+        float k[KPG][8];
 #pragma unroll
-      for (int e = 0; e < KPG; ++e) load8(kc + (size_t)krow[e] * d8 + c, k[e]);
+        for (int e = 0; e < KPG; ++e) load8(kc + (size_t)krow[e] * d8 + c, k[e]);
 #pragma unroll
-      for (int h = 0; h < HN; ++h) {
-        const float4 qa = *reinterpret_cast<const float4 *>(sq + h * d8 + c), qb = *reinterpret_cast<const float4 *>(sq + h * d8 + c + 4);
+        for (int h = 0; h < HN; ++h) {
+          const float4 qa = *reinterpret_cast<const float4 *>(sq + h * d8 + c), qb = *reinterpret_cast<const float4 *>(sq + h * d8 + c + 4);
 #pragma unroll
-        for (int e = 0; e < KPG; ++e) {
-          float x = dot[e][h];
-          x = fmaf(k[e][0], qa.x, fmaf(k[e][1], qa.y, fmaf(k[e][2], qa.z, fmaf(k[e][3], qa.w, x))));
-          dot[e][h] = fmaf(k[e][4], qb.x, fmaf(k[e][5], qb.y, fmaf(k[e][6], qb.z, fmaf(k[e][7], qb.w, x))));
+          for (int e = 0; e < KPG; ++e) {
+            float x = dot[e][h];
+            x = fmaf(k[e][0], qa.x, fmaf(k[e][1], qa.y, fmaf(k[e][2], qa.z, fmaf(k[e][3], qa.w, x))));
+            dot[e][h] = fmaf(k[e][4], qb.x, fmaf(k[e][5], qb.y, fmaf(k[e][6], qb.z, fmaf(k[e][7], qb.w, x))));
+          }
         }
       }
-    }
 #pragma unroll
-    for (int e = 0; e < KPG; ++e)
+      for (int e = 0; e < KPG; ++e)
 #pragma unroll
-      for (int h = 0; h < HN; ++h) {
-        float x = dot[e][h];
-        x += __shfl_xor_sync(0xffffffffu, x, 1);
-        x += __shfl_xor_sync(0xffffffffu, x, 2);
-        dot[e][h] = x + __shfl_xor_sync(0xffffffffu, x, 4);
+        for (int h = 0; h < HN; ++h) {
+          float x = dot[e][h];
+          x += __shfl_xor_sync(0xffffffffu, x, 1);
+          x += __shfl_xor_sync(0xffffffffu, x, 2);
+          dot[e][h] = x + __shfl_xor_sync(0xffffffffu, x, 4);
+        }
+      // the group's KPG * HN scores are finished by its eight lanes
+#pragma unroll
+      for (int r = 0; r < (KPG * HN + 7) / 8; ++r) {
+        const uint32_t id = l8 + 8 * r, e = id / HN, h = id % HN;
+        float mine = 0.f;
+#pragma unroll
+        for (int x = 0; x < KPG * HN; ++x)
+          if (id == (uint32_t)x) mine = dot[x / HN][x % HN];
+        const uint32_t t = part + grp + e * 32;
+        if (id < (uint32_t)(KPG * HN) && h < hn) sp[h * WR_KEYS + t] = t < n ? score(a, h0 + h, mine, i - keys.position(t0 + t)) : -INFINITY;
       }
-    // the group's KPG * HN scores are finished by its eight lanes
-#pragma unroll
-    for (int r = 0; r < (KPG * HN + 7) / 8; ++r) {
-      const uint32_t id = l8 + 8 * r, e = id / HN, h = id % HN;
-      float mine = 0.f;
-#pragma unroll
-      for (int x = 0; x < KPG * HN; ++x)
-        if (id == (uint32_t)x) mine = dot[x / HN][x % HN];
-      const uint32_t t = grp + e * 32;
-      if (id < (uint32_t)(KPG * HN) && h < hn) sp[h * WR_KEYS + t] = t < n ? score(a, h0 + h, mine, i - keys.position(t0 + t)) : -INFINITY;
     }
     __syncthreads();
     if (warp < (int)hn) {
       float *s = sp + warp * WR_KEYS;
       const float old = sm[warp];
-      float x[KPG], mx = old, sum = 0.f;
+      float x[WR_KEYS / 32], mx = old, sum = 0.f;
 #pragma unroll
-      for (int e = 0; e < KPG; ++e) {
-        x[e] = s[lane + 32 * e];
+      for (int e = 0; e < WR_KEYS / 32; ++e) {
+        x[e] = lane + 32 * e < (int)n ? s[lane + 32 * e] : -INFINITY;
         mx = fmaxf(mx, x[e]);
       }
       mx = warp_max(mx);
       const float f = expf(old - mx);
 #pragma unroll
-      for (int e = 0; e < KPG; ++e) {
+      for (int e = 0; e < WR_KEYS / 32; ++e) {
         x[e] = expf(x[e] - mx);
         s[lane + 32 * e] = x[e];
         sum += x[e];
@@ -402,19 +408,20 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
     if (pv) {
 #pragma unroll
       for (int h = 0; h < HN; ++h)
-        if (h < (int)hn) {
-          acc[h][0] *= sf[h];
-          acc[h][1] *= sf[h];
-        }
+        if (h < (int)hn)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) acc[h][x] *= sf[h];
 #pragma unroll 8
       for (uint32_t e = kg; e < n; e += KG) {
-        const float2 v = load2(vc + (size_t)keys.row(t0 + e) * v8 + pr * 2);
+        const float4 v = load4(vc + (size_t)keys.row(t0 + e) * v8 + pr * 4);
 #pragma unroll
         for (int h = 0; h < HN; ++h) {
           const float p = sp[h * WR_KEYS + e];
           if (h < (int)hn) {
             acc[h][0] = fmaf(p, v.x, acc[h][0]);
             acc[h][1] = fmaf(p, v.y, acc[h][1]);
+            acc[h][2] = fmaf(p, v.z, acc[h][2]);
+            acc[h][3] = fmaf(p, v.w, acc[h][3]);
           }
         }
       }
@@ -423,10 +430,9 @@ __global__ void __launch_bounds__(WR_THREADS) window_rows_kernel(const __grid_co
   }
   if (pv)
 #pragma unroll
-    for (int h = 0; h < HN; ++h) {
-      sx[((size_t)kg * HN + h) * v8 + pr * 2] = acc[h][0];
-      sx[((size_t)kg * HN + h) * v8 + pr * 2 + 1] = acc[h][1];
-    }
+    for (int h = 0; h < HN; ++h)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) sx[((size_t)kg * HN + h) * v8 + pr * 4 + x] = acc[h][x];
   __syncthreads();
   for (uint32_t e = threadIdx.x; e < hn * v8; e += WR_THREADS) {
     float t = 0.f;
@@ -686,7 +692,7 @@ int launch_conv(cudaStream_t s, const WinArgs &w, float *q) {
 template <typename CT, int HN, bool FUSED>
 int launch_rows(cudaStream_t s, const WinArgs &w, const float *q, void *out, int out_fmt, uint32_t ld_out, uint32_t splits) {
   const greta_window_attn &a = w.a;
-  const uint32_t d8 = up8(a.dim), v8 = up8(a.vdim), tpp = (v8 / 2 + 31) / 32 * 32, KG = WR_THREADS / tpp;
+  const uint32_t d8 = up8(a.dim), v8 = up8(a.vdim), tpp = (v8 / 4 + 31) / 32 * 32, KG = WR_THREADS / tpp;
   const size_t smem = ((size_t)HN * (d8 + WR_KEYS + v8 + (size_t)KG * v8) + 3 * HN) * 4;
   static bool attr_set[64] = {};
   int dev = 0;
