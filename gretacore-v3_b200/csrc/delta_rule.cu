@@ -123,39 +123,16 @@ __device__ __forceinline__ void cp4(void *dst, const void *src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-typedef unsigned long long f32x2;  // two floats for the packed 32-bit arithmetic
-__device__ __forceinline__ f32x2 pack2(float a, float b) {
-  f32x2 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
-  return d;
-}
-__device__ __forceinline__ float sum_halves(f32x2 v) {
-  float a, b;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
-  return a + b;
-}
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-  f32x2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ ulonglong2 lds2(const float *p) { return *reinterpret_cast<const ulonglong2 *>(p); }
-
 // The recurrence over a portion: grid (heads, column groups).  A CTA keeps 32 columns of one head in the registers of its
 // first warps, NC columns per group of eight lanes, and walks the tokens in chunks of TC = a block per producer warp.
 template <int RB, int NC>
 struct ScanCfg {
   static constexpr int DP = RB * 32, COLS = 32;
-  static constexpr int TC = RB <= 4 ? 16 : 8, NB = TC / 4;
+  static constexpr int TC = RB <= 2 ? 32 : RB <= 4 ? 16 : 8, NB = TC / 4;
   static constexpr int RAW_ROW = 4 * DP + COLS, RAW = TC * RAW_ROW;   // a staged token: w, k, a, r, v
   static constexpr int SCAL = 17 * DP, VT = SCAL + 48;                // of a block: 17 vectors, {P, -Q | R | -T}, v [column][4]
   static constexpr int BLK = VT + 4 * COLS, DER = NB * BLK;
-  static constexpr int CW = COLS / (4 * NC), PW = 4, THREADS = (CW + PW) * 32;
+  static constexpr int CW = COLS / (4 * NC), PW = NB < 4 ? 4 : NB, THREADS = (CW + PW) * 32;
   static constexpr size_t SMEM = (size_t)(2 * RAW + 2 * DER + 2 * TC * COLS) * 4;
   static_assert(SMEM <= 232448, "chunk buffers exceed shared memory");
 };
@@ -207,7 +184,9 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
         if (vec) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
-            for (uint32_t e = lane * 4; e < D; e += 128) cp16(dst + i * DP + e, src[i] + e);
+#pragma unroll
+            for (int j = 0; j < (DP + 127) / 128; ++j)
+              if (lane * 4 + j * 128 < (int)D) cp16(dst + i * DP + lane * 4 + j * 128, src[i] + lane * 4 + j * 128);
           if (lane * 4 < (int)vcols) cp16(dst + 4 * DP + lane * 4, d.v + at + c0 + lane * 4);
         } else {
 #pragma unroll
@@ -293,7 +272,7 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
   };
 
   const int grp = threadIdx.x >> 3;  // state warps: columns c0 + grp * NC ..
-  f32x2 s[NC][2 * RB];
+  float4 s[NC][RB];
   if (producer) {
     stage(0);
     stage(1);
@@ -305,10 +284,7 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
       const uint32_t col = c0 + grp * NC + c;
 #pragma unroll
       for (int i = 0; i < RB; ++i) {
-        const bool on = col < D && a.rows.pos0;
-        const ulonglong2 v = on ? *reinterpret_cast<const ulonglong2 *>(state + (size_t)col * DP + i * 32 + l8 * 4) : make_ulonglong2(0ull, 0ull);
-        s[c][2 * i] = v.x;
-        s[c][2 * i + 1] = v.y;
+        s[c][i] = col < D && a.rows.pos0 ? *reinterpret_cast<const float4 *>(state + (size_t)col * DP + i * 32 + l8 * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
     }
   }
@@ -325,31 +301,21 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
       for (int blk = 0; blk < C::NB; ++blk) {
         const float *b = derived + (ch & 1) * C::DER + blk * C::BLK;
         float x[NC][4], o[NC][4];
-        {
-          f32x2 xs[NC][4], rs[NC][4];
 #pragma unroll
-          for (int c = 0; c < NC; ++c)
+        for (int c = 0; c < NC; ++c)
 #pragma unroll
-            for (int t = 0; t < 4; ++t) xs[c][t] = rs[c][t] = 0ull;
+          for (int t = 0; t < 4; ++t) x[c][t] = o[c][t] = 0.f;
 #pragma unroll
-          for (int i = 0; i < RB; ++i)
+        for (int i = 0; i < RB; ++i)
 #pragma unroll
-            for (int t = 0; t < 4; ++t) {
-              const ulonglong2 k = lds2(b + t * DP + i * 32 + l8 * 4), r = lds2(b + (4 + t) * DP + i * 32 + l8 * 4);
+          for (int t = 0; t < 4; ++t) {
+            const float4 k = lds4(b + t * DP + i * 32 + l8 * 4), r = lds4(b + (4 + t) * DP + i * 32 + l8 * 4);
 #pragma unroll
-              for (int c = 0; c < NC; ++c) {
-                xs[c][t] = fma2(k.y, s[c][2 * i + 1], fma2(k.x, s[c][2 * i], xs[c][t]));
-                rs[c][t] = fma2(r.y, s[c][2 * i + 1], fma2(r.x, s[c][2 * i], rs[c][t]));
-              }
+            for (int c = 0; c < NC; ++c) {
+              x[c][t] = dot4(k, s[c][i], x[c][t]);
+              o[c][t] = dot4(r, s[c][i], o[c][t]);
             }
-#pragma unroll
-          for (int c = 0; c < NC; ++c)
-#pragma unroll
-            for (int t = 0; t < 4; ++t) {
-              x[c][t] = sum_halves(xs[c][t]);
-              o[c][t] = sum_halves(rs[c][t]);
-            }
-        }
+          }
         // P10 P20 P21 P30 | P31 P32 -Q10 -Q20 | -Q21 -Q30 -Q31 -Q32
         const float4 s0 = lds4(b + C::SCAL), s1 = lds4(b + C::SCAL + 4), s2 = lds4(b + C::SCAL + 8);
         const float4 R = lds4(b + C::SCAL + 16 + (l8 >> 1) * 4), Tn = lds4(b + C::SCAL + 32 + (l8 >> 1) * 4);  // of this lane's token
@@ -368,22 +334,20 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
 #pragma unroll
         for (int i = 0; i < RB; ++i) {
           const int at = i * 32 + l8 * 4;
-          const ulonglong2 w = lds2(b + 8 * DP + at);
+          const float4 w = lds4(b + 8 * DP + at);
 #pragma unroll
-          for (int c = 0; c < NC; ++c) {
-            s[c][2 * i] = mul2(w.x, s[c][2 * i]);
-            s[c][2 * i + 1] = mul2(w.y, s[c][2 * i + 1]);
-          }
+          for (int c = 0; c < NC; ++c) s[c][i] = make_float4(w.x * s[c][i].x, w.y * s[c][i].y, w.z * s[c][i].z, w.w * s[c][i].w);
 #pragma unroll
           for (int t = 0; t < 4; ++t) {
-            const ulonglong2 k = lds2(b + (9 + t) * DP + at), ak = lds2(b + (13 + t) * DP + at);
+            const float4 k = lds4(b + (9 + t) * DP + at), ak = lds4(b + (13 + t) * DP + at);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
               const float vt = t == 0 ? v[c].x : t == 1 ? v[c].y : t == 2 ? v[c].z : v[c].w;
               const float ct = t == 0 ? cc[c].x : t == 1 ? cc[c].y : t == 2 ? cc[c].z : cc[c].w;
-              const f32x2 v2 = pack2(vt, vt), c2 = pack2(ct, ct);
-              s[c][2 * i] = fma2(ak.x, c2, fma2(k.x, v2, s[c][2 * i]));
-              s[c][2 * i + 1] = fma2(ak.y, c2, fma2(k.y, v2, s[c][2 * i + 1]));
+              s[c][i].x = fmaf(ak.x, ct, fmaf(k.x, vt, s[c][i].x));
+              s[c][i].y = fmaf(ak.y, ct, fmaf(k.y, vt, s[c][i].y));
+              s[c][i].z = fmaf(ak.z, ct, fmaf(k.z, vt, s[c][i].z));
+              s[c][i].w = fmaf(ak.w, ct, fmaf(k.w, vt, s[c][i].w));
             }
           }
         }
@@ -407,7 +371,7 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC>::THREADS) delta_scan_kernel(co
       const uint32_t col = c0 + grp * NC + c;
 #pragma unroll
       for (int i = 0; i < RB; ++i)
-        if (col < D) *reinterpret_cast<ulonglong2 *>(state + (size_t)col * DP + i * 32 + l8 * 4) = make_ulonglong2(s[c][2 * i], s[c][2 * i + 1]);
+        if (col < D) *reinterpret_cast<float4 *>(state + (size_t)col * DP + i * 32 + l8 * 4) = s[c][i];
     }
   }
 }
@@ -533,8 +497,8 @@ int greta_cuda_delta_scan(greta_stream_t stream, const greta_delta_rule *d, cons
   const int vec = d->dim % 4 == 0 && d->ld % 4 == 0 && d->ld_decay % 4 == 0 && aligned16(d->r) && aligned16(d->k) && aligned16(d->v) && aligned16(d->a) &&
                   aligned16(d->decay);
   switch (dim32(d->dim) / 32) {
-    case 1: return launch_scan<1, 4>(s, a, o_buf, vec);
-    case 2: return launch_scan<2, 4>(s, a, o_buf, vec);
+    case 1: return launch_scan<1, 2>(s, a, o_buf, vec);
+    case 2: return launch_scan<2, 2>(s, a, o_buf, vec);
     case 3: return launch_scan<3, 2>(s, a, o_buf, vec);
     case 4: return launch_scan<4, 2>(s, a, o_buf, vec);
     case 5: return launch_scan<5, 1>(s, a, o_buf, vec);
