@@ -54,7 +54,7 @@ int main(int argc, char **argv) {
   if (model.empty() || out_dir.empty() || (dtype != "bfloat16" && dtype != "float32"))
     return complain("usage: trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N", 2);
   gcore::cli::Session s;
-  if (!s.open(model, dtype == "float32", kSlots, max_tokens, &err)) return complain(err);
+  if (!s.open(model, dtype == "float32", kSlots, max_tokens, &err, 16384)) return complain(err);
   auto &sched = s.scheduler;
   const size_t V = s.config.vocab_size;
 

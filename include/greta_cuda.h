@@ -455,7 +455,7 @@ GRETA_API int greta_cuda_linear_gemv(greta_stream_t stream, const greta_linear *
 /* Many rows.  BF16: tensor cores (tcgen05), x is bf16 [M][ldx], ldx a multiple of 8 and its columns K .. ldw-1 zero where
  * ldx >= ldw.  F32: true 32-bit products on the CUDA cores, x is fp32 [M][ldx], ldx >= ldw, zero-padded. */
 GRETA_API int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *lin, const void *x, uint32_t ldx, uint32_t M);
-/* Same contract as greta_cuda_gemm_status, for the kernels of greta_cuda_linear_gemm. */
+/* greta_cuda_gemm_status for the kernels of greta_cuda_linear_gemm. */
 GRETA_API int greta_cuda_linear_gemm_status(int *code);
 /* y = (x - mean) / sqrt(var + eps) * w + b per row of D values; out fp32 or bf16 (GRETA_OUT_*), row stride ld_out. */
 GRETA_API int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w, const float *b, float eps, void *out, int out_fmt,
