@@ -42,8 +42,10 @@ int main(int argc, char **argv) {
   }
   if (model.empty() || prompts.empty() || (dtype != "bfloat16" && dtype != "float32"))
     return complain("usage: greta_infer --model DIR|FILE.gguf --tokens 1,2,3[;4,5] [--max-tokens N] [--dtype bfloat16|float32] [--eos ID] [--max-seq N]", 2);
+  size_t longest = 0;
+  for (const auto &p : prompts) longest = std::max(longest, p.size());
   gcore::cli::Session s;
-  if (!s.open(model, dtype == "float32", prompts.size(), max_seq, &err)) return complain(err);
+  if (!s.open(model, dtype == "float32", prompts.size(), max_seq, &err, 0, longest + (size_t)std::max(sp.max_tokens, 1))) return complain(err);
   std::vector<std::vector<int32_t>> out;
   if (prompts.size() == 1) {
     gcore::inference::GenerationStats st;

@@ -13,9 +13,9 @@ struct Session {
   inference::BlockScheduler scheduler;
   inference::Generator generator;
 
-  // fp32: run an unquantised design in true 32-bit.  max_seq: positions of a sequence, 0 for as many as the model has; a model
-  // with no more than `roomy` of them gets them all.
-  bool open(const std::string &path, bool fp32, size_t batch, size_t max_seq, std::string *err, size_t roomy = 0) {
+  // fp32: run an unquantised design in true 32-bit.  max_seq: positions of a sequence; 0: as many as the model has or, where
+  // nothing bounds them, `needed`.  A model with no more than `roomy` positions gets them all.
+  bool open(const std::string &path, bool fp32, size_t batch, size_t max_seq, std::string *err, size_t roomy = 0, size_t needed = 0) {
     std::unique_ptr<inference::WeightLoader> loader = inference::create_weight_loader(path, err);
     if (!loader) return false;
     config = loader->get_config();
@@ -25,6 +25,7 @@ struct Session {
       *err = "32-bit computation: only unquantised model folders run in it";
       return false;
     }
+    if (!max_seq && config.default_seq_len) max_seq = needed ? needed : config.default_seq_len;
     const size_t seq = max_seq && config.max_seq_len > roomy ? std::min<size_t>(max_seq, config.max_seq_len) : config.max_seq_len;
     return scheduler.init(config, err) && scheduler.allocate_weights(err) && scheduler.load_weights(*loader, err) &&
            scheduler.allocate_activations(batch, seq, err) && generator.init(config, &scheduler, err);

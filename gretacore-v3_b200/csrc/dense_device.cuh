@@ -12,12 +12,15 @@ struct Segments {
 };
 
 __device__ __forceinline__ float act_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float apply_act(int act, float z) {
+__device__ __forceinline__ float act_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float apply_act(int act, float z, float rate = 0.f) {
   switch (act) {
     case GRETA_ACT_GELU_ERF: return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
     case GRETA_ACT_SIGMOID: return act_sigmoid(z);
     case GRETA_ACT_TANH: return tanhf(z);
     case GRETA_ACT_DELTA_DECAY: return expf(-0.60653065971263342f * act_sigmoid(z));
+    case GRETA_ACT_RELU2: return z > 0.f ? z * z : 0.f;
+    case GRETA_ACT_SOFTPLUS_DECAY: return expf(-rate * act_softplus(z));
     default: return z;
   }
 }
@@ -30,6 +33,8 @@ __device__ __forceinline__ int segment_of(const Segments &sg, uint32_t row) {
 __device__ __forceinline__ void store_out(void *out, int fmt, size_t idx, float v, uint32_t pair_offset = 0) {
   if (fmt == GRETA_OUT_F32) {
     static_cast<float *>(out)[idx] = v;
+  } else if (fmt == GRETA_OUT_F16) {
+    static_cast<__half *>(out)[idx] = __float2half_rn(v);
   } else {
     const __nv_bfloat16 hi = __float2bfloat16_rn(v);
     static_cast<__nv_bfloat16 *>(out)[idx] = hi;
@@ -39,7 +44,7 @@ __device__ __forceinline__ void store_out(void *out, int fmt, size_t idx, float 
 __device__ __forceinline__ void store_segment(const greta_out_segment &g, uint32_t row, uint32_t m, float z) {
   const uint32_t r = row - g.row0;
   if (g.bias) z += __ldg(g.bias + r);
-  z = apply_act(g.act, z);
+  z = apply_act(g.act, z, g.rate ? __ldg(g.rate + r) : 0.f);
   const size_t idx = (size_t)m * g.ld + g.col0 + r;
   if (g.accumulate)
     static_cast<float *>(g.out)[idx] += z;

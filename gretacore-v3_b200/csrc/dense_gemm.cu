@@ -1,6 +1,6 @@
 // Dense linears on many activation rows (prompts and long portions).
 //
-// bf16: tensor cores.  The weight rows are the 128-row operand of tcgen05.mma and TN tokens its N dimension, so a thread
+// bf16 or fp16: tensor cores.  The weight rows are the 128-row operand of tcgen05.mma and TN tokens its N dimension, so a thread
 // of the epilogue owns one weight row (one segment, one bias) and a warp stores 32 consecutive outputs of a token.
 // Persistent CTAs, one per SM, walk the tiles with the token tiles innermost: the CTAs in flight share a few weight row
 // tiles, which are read from HBM once.  Roles (320 threads): warp 0 TMA producer of both operands (128-byte swizzle, 64
@@ -42,6 +42,7 @@ struct DCfg {
 template <int ACT>
 __device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
   const size_t base = (size_t)m * g.ld + g.col0 + r;
+  const float rate = ACT == GRETA_ACT_SOFTPLUS_DECAY ? __ldg(g.rate + r) : 0.f;
   if (g.accumulate) {
     float *o = static_cast<float *>(g.out) + base;
     float old[32];
@@ -49,16 +50,16 @@ __device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint3
     for (int j = 0; j < 32; ++j) old[j] = j < cnt ? o[(size_t)j * g.ld] : 0.f;
 #pragma unroll
     for (int j = 0; j < 32; ++j)
-      if (j < cnt) o[(size_t)j * g.ld] = old[j] + apply_act(ACT, __uint_as_float(v[j]) + bias);
+      if (j < cnt) o[(size_t)j * g.ld] = old[j] + apply_act(ACT, __uint_as_float(v[j]) + bias, rate);
   } else if (g.out_fmt == GRETA_OUT_F32) {
     float *o = static_cast<float *>(g.out) + base;
 #pragma unroll
     for (int j = 0; j < 32; ++j)
-      if (j < cnt) o[(size_t)j * g.ld] = apply_act(ACT, __uint_as_float(v[j]) + bias);
+      if (j < cnt) o[(size_t)j * g.ld] = apply_act(ACT, __uint_as_float(v[j]) + bias, rate);
   } else {
 #pragma unroll
     for (int j = 0; j < 32; ++j)
-      if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(ACT, __uint_as_float(v[j]) + bias), g.pair_offset);
+      if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(ACT, __uint_as_float(v[j]) + bias, rate), g.pair_offset);
   }
 }
 __device__ __forceinline__ void finish_row(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
@@ -67,6 +68,8 @@ __device__ __forceinline__ void finish_row(const greta_out_segment &g, uint32_t 
     case GRETA_ACT_SIGMOID: finish_row_act<GRETA_ACT_SIGMOID>(g, r, bias, m, cnt, v); break;
     case GRETA_ACT_TANH: finish_row_act<GRETA_ACT_TANH>(g, r, bias, m, cnt, v); break;
     case GRETA_ACT_DELTA_DECAY: finish_row_act<GRETA_ACT_DELTA_DECAY>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_RELU2: finish_row_act<GRETA_ACT_RELU2>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_SOFTPLUS_DECAY: finish_row_act<GRETA_ACT_SOFTPLUS_DECAY>(g, r, bias, m, cnt, v); break;
     default: finish_row_act<GRETA_ACT_NONE>(g, r, bias, m, cnt, v); break;
   }
 }
@@ -83,7 +86,7 @@ __device__ __forceinline__ void drain_copies(uint64_t *full, uint32_t issued, ui
 template <int TN>
 __global__ void __launch_bounds__(DCfg<TN>::THREADS, 1)
 linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ Segments sg, uint32_t M,
-                 uint32_t N, uint32_t K) {
+                 uint32_t N, uint32_t K, uint32_t idesc) {
   using C = DCfg<TN>;
   constexpr int ST = C::ST;
   extern __shared__ uint8_t smem_raw[];
@@ -144,7 +147,6 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc = instr_desc_bf16(TILE_N, TN);
       const uint32_t lo0 = smem_desc_lo(smem_u32(smem));
       uint32_t s = 0, ph = 0, it = 0;
       bool ok = true;
@@ -216,7 +218,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
 template <int TN>
 __global__ void __launch_bounds__(DCfg<TN>::THREADS, 1)
 linear_tc_split_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ Segments sg,
-                       uint32_t M, uint32_t N, uint32_t K) {
+                       uint32_t M, uint32_t N, uint32_t K, uint32_t idesc) {
   namespace cg = cooperative_groups;
   using C = DCfg<TN>;
   constexpr int ST = C::ST, COLS = TN < 32 ? 32 : TN;
@@ -276,7 +278,6 @@ linear_tc_split_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc = instr_desc_bf16(TILE_N, TN);
       const uint32_t lo0 = smem_desc_lo(smem_u32(smem));
       uint32_t s = 0, ph = 0;
       bool ok = true;
@@ -375,7 +376,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float *__restrict
   }
 }
 
-int make_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, uint32_t ld, uint32_t box_rows) {
+int make_map(CUtensorMap *map, int fmt, const void *base, uint32_t cols, uint32_t rows, uint32_t ld, uint32_t box_rows) {
   EncodeTiledFn enc = encode_tiled();
   if (!enc) {
     set_error("linear_gemm: cuTensorMapEncodeTiled is not available from this driver");
@@ -383,7 +384,7 @@ int make_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, u
   }
   const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(cuuint64_t)ld * 2};
   const cuuint32_t box[2] = {BK, box_rows}, estr[2] = {1, 1};
-  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+  const CUresult r = enc(map, fmt == GRETA_FMT_F16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                          CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) {
     set_error("linear_gemm: cuTensorMapEncodeTiled failed with code %d", (int)r);
@@ -404,14 +405,15 @@ int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, cons
     attr_set[dev] = true;
   }
   CUtensorMap mw, mx;
-  if (int rc = make_map(&mw, l->w, l->K, l->N, l->ldw, TILE_N)) return rc;  // columns past K read as zero in both operands
-  if (int rc = make_map(&mx, x, l->K, M, ldx, TN)) return rc;
+  if (int rc = make_map(&mw, l->fmt, l->w, l->K, l->N, l->ldw, TILE_N)) return rc;  // columns past K read as zero in both operands
+  if (int rc = make_map(&mx, l->fmt, x, l->K, M, ldx, TN)) return rc;
   const uint32_t tiles = ((l->N + TILE_N - 1) / TILE_N) * ((M + TN - 1) / TN);
+  const uint32_t idesc = l->fmt == GRETA_FMT_F16 ? instr_desc_f16(TILE_N, TN) : instr_desc_bf16(TILE_N, TN);  // both operands are of one type
   if (split > 1) {
-    GRETA_CUDA_TRY(launch_pdl_cluster(linear_tc_split_kernel<TN>, dim3(tiles * split), dim3(C::THREADS), split, C::SMEM, s, mw, mx, sg, M, l->N, l->K));
+    GRETA_CUDA_TRY(launch_pdl_cluster(linear_tc_split_kernel<TN>, dim3(tiles * split), dim3(C::THREADS), split, C::SMEM, s, mw, mx, sg, M, l->N, l->K, idesc));
     return launched("linear_tc_split_kernel");
   }
-  GRETA_CUDA_TRY(launch_pdl(linear_tc_kernel<TN>, dim3(std::min(tiles, (uint32_t)sm_count())), dim3(C::THREADS), C::SMEM, s, mw, mx, sg, M, l->N, l->K));
+  GRETA_CUDA_TRY(launch_pdl(linear_tc_kernel<TN>, dim3(std::min(tiles, (uint32_t)sm_count())), dim3(C::THREADS), C::SMEM, s, mw, mx, sg, M, l->N, l->K, idesc));
   return launched("linear_tc_kernel");
 }
 

@@ -1,6 +1,6 @@
 // Dense linears on few activation rows (decode and short portions): y[m][n] = act(W[n] . LN(x[m]) + bias), weights in bf16
 // or fp32 streamed once for up to 8 rows, activations and accumulation in fp32; and the small operators around them
-// (layer norm, embedding with learned positions, row gather).
+// (layer and root-mean-square norm, embeddings, row gather).  A norm without an offset (ln_b) is the root-mean-square one.
 //
 // A warp owns R weight rows.  Each lane takes 8 consecutive weights of every row per step (16 bytes of bf16), the
 // activations of the same 8 columns come out of shared memory once for all R rows.  There the two float4 halves of every
@@ -77,9 +77,11 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
   pdl_wait();
   if (ln_w) {
     if (MR == 1) {
-      float s = 0.f;
-      for (uint32_t k = threadIdx.x; k < K; k += GV_THREADS) s += x[k];
-      const float mean = block_sum_all(s, red) / (float)K;
+      float s = 0.f, mean = 0.f;
+      if (ln_b) {
+        for (uint32_t k = threadIdx.x; k < K; k += GV_THREADS) s += x[k];
+        mean = block_sum_all(s, red) / (float)K;
+      }
       float q = 0.f;
       for (uint32_t k = threadIdx.x; k < K; k += GV_THREADS) {
         const float c = x[k] - mean;
@@ -92,9 +94,11 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
       }
     } else if (warp < MR && warp < M) {
       const float *xr = x + (size_t)warp * ldx;
-      float s = 0.f;
-      for (uint32_t k = lane; k < K; k += 32) s += xr[k];
-      const float mean = warp_sum(s) / (float)K;
+      float s = 0.f, mean = 0.f;
+      if (ln_b) {
+        for (uint32_t k = lane; k < K; k += 32) s += xr[k];
+        mean = warp_sum(s) / (float)K;
+      }
       float q = 0.f;
       for (uint32_t k = lane; k < K; k += 32) {
         const float c = xr[k] - mean;
@@ -130,7 +134,8 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
           if (col < K) {
             v = *reinterpret_cast<const float4 *>(xr + col);
             if (ln_w) {
-              const float4 w = __ldg(reinterpret_cast<const float4 *>(ln_w + col)), b = __ldg(reinterpret_cast<const float4 *>(ln_b + col));
+              const float4 w = __ldg(reinterpret_cast<const float4 *>(ln_w + col));
+              const float4 b = ln_b ? __ldg(reinterpret_cast<const float4 *>(ln_b + col)) : make_float4(0.f, 0.f, 0.f, 0.f);
               v.x = (v.x - mean) * inv * w.x + b.x;
               v.y = (v.y - mean) * inv * w.y + b.y;
               v.z = (v.z - mean) * inv * w.z + b.z;
@@ -146,7 +151,7 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
         float v = 0.f;
         if (row && col < K) {
           v = xr[col];
-          if (ln_w) v = (v - mean) * inv * __ldg(ln_w + col) + __ldg(ln_b + col);
+          if (ln_w) v = (v - mean) * inv * __ldg(ln_w + col) + (ln_b ? __ldg(ln_b + col) : 0.f);
         }
         xd[((k >> 2) & 1) * plane * 4 + (k >> 3) * 4 + (k & 3)] = v;
       }
@@ -212,13 +217,14 @@ __global__ void __launch_bounds__(GV_THREADS) linear_gemv_kernel(const WT *__res
   if (m < min(M, (uint32_t)MR) && row < N) store_segment(sg.s[segment_of(sg, row)], row, m, mine);
 }
 
-// One CTA per row; rows of up to 8192 columns (a multiple of 4) are read once and kept in registers.
-__global__ void __launch_bounds__(256) layer_norm_kernel(const float *__restrict__ x, const float *__restrict__ w, const float *__restrict__ b, float eps,
-                                                         void *out, int out_fmt, uint32_t D, uint32_t ld, int vec) {
+// One CTA per row; rows of up to 8192 columns (a multiple of 4) are read once and kept in registers.  RMS: no mean, no offset.
+template <bool RMS>
+__global__ void __launch_bounds__(256) norm_kernel(const float *__restrict__ x, uint32_t ldx, const float *__restrict__ w, const float *__restrict__ b,
+                                                   float eps, void *out, int out_fmt, uint32_t D, uint32_t ld, int vec) {
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
-  const float *xr = x + (size_t)blockIdx.x * D;
+  const float *xr = x + (size_t)blockIdx.x * ldx;
   if (vec) {
     constexpr int U = 8;
     float4 v[U];
@@ -229,7 +235,7 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float *__restrict
       v[u] = k < D ? *reinterpret_cast<const float4 *>(xr + k) : make_float4(0.f, 0.f, 0.f, 0.f);
       s += (v[u].x + v[u].y) + (v[u].z + v[u].w);
     }
-    const float mean = block_sum_all(s, red) / (float)D;
+    const float mean = RMS ? 0.f : block_sum_all(s, red) / (float)D;
     float q = 0.f;
 #pragma unroll
     for (int u = 0; u < U; ++u) {
@@ -242,11 +248,18 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float *__restrict
     for (int u = 0; u < U; ++u) {
       const uint32_t k = (u * 256 + threadIdx.x) * 4;
       if (k >= D) continue;
-      const float4 g = *reinterpret_cast<const float4 *>(w + k), h = *reinterpret_cast<const float4 *>(b + k);
+      const float4 g = *reinterpret_cast<const float4 *>(w + k);
+      const float4 h = RMS ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4 *>(b + k);
       const float4 y = make_float4(v[u].x * inv * g.x + h.x, v[u].y * inv * g.y + h.y, v[u].z * inv * g.z + h.z, v[u].w * inv * g.w + h.w);
       const size_t at = (size_t)blockIdx.x * ld + k;
       if (out_fmt == GRETA_OUT_F32) {
         *reinterpret_cast<float4 *>(static_cast<float *>(out) + at) = y;
+      } else if (out_fmt == GRETA_OUT_F16) {
+        const __half2 lo = __floats2half2_rn(y.x, y.y), hi = __floats2half2_rn(y.z, y.w);
+        uint2 p;
+        p.x = *reinterpret_cast<const uint32_t *>(&lo);
+        p.y = *reinterpret_cast<const uint32_t *>(&hi);
+        *reinterpret_cast<uint2 *>(static_cast<__half *>(out) + at) = p;
       } else {
         const __nv_bfloat162 lo = __floats2bfloat162_rn(y.x, y.y), hi = __floats2bfloat162_rn(y.z, y.w);
         uint2 p;
@@ -257,16 +270,19 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float *__restrict
     }
     return;
   }
-  float s = 0.f;
-  for (uint32_t k = threadIdx.x; k < D; k += 256) s += xr[k];
-  const float mean = block_sum_all(s, red) / (float)D;
+  float mean = 0.f;
+  if (!RMS) {
+    float s = 0.f;
+    for (uint32_t k = threadIdx.x; k < D; k += 256) s += xr[k];
+    mean = block_sum_all(s, red) / (float)D;
+  }
   float q = 0.f;
   for (uint32_t k = threadIdx.x; k < D; k += 256) {
     const float c = xr[k] - mean;
     q = fmaf(c, c, q);
   }
   const float inv = 1.f / sqrtf(block_sum_all(q, red) / (float)D + eps);
-  for (uint32_t k = threadIdx.x; k < D; k += 256) store_out(out, out_fmt, (size_t)blockIdx.x * ld + k, (xr[k] - mean) * inv * w[k] + b[k]);
+  for (uint32_t k = threadIdx.x; k < D; k += 256) store_out(out, out_fmt, (size_t)blockIdx.x * ld + k, (xr[k] - mean) * inv * w[k] + (RMS ? 0.f : b[k]));
 }
 
 template <typename T>
@@ -289,6 +305,17 @@ __global__ void embedding_positions_kernel(const int32_t *__restrict__ tokens, c
   out[i] = v;
 }
 
+template <typename T>
+__global__ void embedding_scaled_kernel(const int32_t *__restrict__ tokens, const T *__restrict__ table, uint32_t ld, float scale, float *__restrict__ out,
+                                        uint32_t M, uint32_t D, uint32_t vocab) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (size_t)M * D) return;
+  const int32_t t = tokens[i / D];
+  out[i] = t >= 0 && (uint32_t)t < vocab ? scale * (float)table[(size_t)t * ld + i % D] : 0.f;
+}
+
 struct RowList {
   uint32_t r[64];
 };
@@ -309,7 +336,7 @@ int launch_gemv(cudaStream_t s, const greta_linear *l, const Segments &sg, const
     attr_set[dev] = true;
   }
   const uint32_t grid = (l->N + GV_WARPS * R - 1) / (GV_WARPS * R);
-  const int vec = l->K % 4 == 0 && ldx % 4 == 0 && aligned16(x) && (!ln_w || (aligned16(ln_w) && aligned16(ln_b)));
+  const int vec = l->K % 4 == 0 && ldx % 4 == 0 && aligned16(x) && (!ln_w || (aligned16(ln_w) && (!ln_b || aligned16(ln_b))));
   GRETA_CUDA_TRY(launch_pdl(linear_gemv_kernel<WT, MR, R>, dim3(grid), dim3(GV_THREADS), smem, s, static_cast<const WT *>(l->w), l->N, l->K, l->ldw, sg, x,
                             ldx, ln_w, ln_b, eps, M, chunk, vec));
   return launched("linear_gemv_kernel");
@@ -336,7 +363,8 @@ namespace greta {
 // Shared argument checks of the dense linears; fills the by-value segment list.
 int check_linear(const char *what, const greta_linear *l, Segments *sg) {
   GRETA_REQUIRE(l && l->w && l->N && l->K, "%s: null or empty linear", what);
-  GRETA_REQUIRE(l->fmt == GRETA_FMT_BF16 || l->fmt == GRETA_FMT_F32, "%s: weight format %d is not dense (BF16 or F32)", what, l->fmt);
+  GRETA_REQUIRE(l->fmt == GRETA_FMT_BF16 || l->fmt == GRETA_FMT_F32 || l->fmt == GRETA_FMT_F16, "%s: weight format %d is not dense (BF16, F16 or F32)", what,
+                l->fmt);
   GRETA_REQUIRE(l->ldw % 64 == 0 && l->ldw >= l->K && aligned16(l->w), "%s: ldw=%u K=%u or a misaligned weight", what, l->ldw, l->K);
   GRETA_REQUIRE(l->n_segments >= 1 && l->n_segments <= GRETA_MAX_SEGMENTS, "%s: %u segments", what, l->n_segments);
   uint32_t row = 0;
@@ -344,6 +372,7 @@ int check_linear(const char *what, const greta_linear *l, Segments *sg) {
     const greta_out_segment &g = l->seg[i];
     GRETA_REQUIRE(g.row0 == row && g.rows && g.out, "%s: segment %u leaves a gap or has no output", what, i);
     GRETA_REQUIRE(!g.accumulate || g.out_fmt == GRETA_OUT_F32, "%s: segment %u accumulates into a format other than fp32", what, i);
+    GRETA_REQUIRE(g.act != GRETA_ACT_SOFTPLUS_DECAY || g.rate, "%s: segment %u has no decay rates", what, i);
     row += g.rows;
     sg->s[i] = g;
   }
@@ -360,7 +389,8 @@ int greta_cuda_linear_gemv(greta_stream_t stream, const greta_linear *l, const f
   Segments sg{};
   if (int rc = check_linear("linear_gemv", l, &sg)) return rc;
   GRETA_REQUIRE(M >= 1 && M <= 8, "linear_gemv: M=%u (1..8)", M);
-  GRETA_REQUIRE(x && ldx >= l->K && (!ln_w == !ln_b), "linear_gemv: bad activations or norm");
+  GRETA_REQUIRE(x && ldx >= l->K && (ln_w || !ln_b), "linear_gemv: bad activations or norm");
+  GRETA_REQUIRE(l->fmt != GRETA_FMT_F16, "linear_gemv: weights must be BF16 or F32");
   cudaStream_t s = (cudaStream_t)stream;
   return l->fmt == GRETA_FMT_BF16 ? pick_m<__nv_bfloat16>(s, l, sg, x, ldx, ln_w, ln_b, eps, M) : pick_m<float>(s, l, sg, x, ldx, ln_w, ln_b, eps, M);
 }
@@ -369,10 +399,21 @@ int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w,
                           uint32_t ld_out) {
   if (M == 0) return GRETA_OK;
   GRETA_REQUIRE(x && w && b && out && D && ld_out >= D, "layer_norm: bad argument");
-  GRETA_REQUIRE(out_fmt == GRETA_OUT_F32 || out_fmt == GRETA_OUT_BF16, "layer_norm: output format %d", out_fmt);
+  GRETA_REQUIRE(out_fmt == GRETA_OUT_F32 || out_fmt == GRETA_OUT_F16 || out_fmt == GRETA_OUT_BF16, "layer_norm: output format %d", out_fmt);
   const int vec = D <= 8192 && D % 4 == 0 && ld_out % 4 == 0 && aligned16(x) && aligned16(w) && aligned16(b) && aligned16(out);
-  GRETA_CUDA_TRY(launch_pdl(layer_norm_kernel, dim3(M), dim3(256), 0, (cudaStream_t)stream, x, w, b, eps, out, out_fmt, D, ld_out, vec));
-  return launched("layer_norm_kernel");
+  GRETA_CUDA_TRY(launch_pdl(norm_kernel<false>, dim3(M), dim3(256), 0, (cudaStream_t)stream, x, D, w, b, eps, out, out_fmt, D, ld_out, vec));
+  return launched("norm_kernel");
+}
+
+int greta_cuda_rms_norm(greta_stream_t stream, const float *x, uint32_t ldx, const float *w, float eps, void *out, int out_fmt, uint32_t M, uint32_t D,
+                        uint32_t ld_out) {
+  if (M == 0) return GRETA_OK;
+  GRETA_REQUIRE(x && w && out && D && ldx >= D && ld_out >= D, "rms_norm: bad argument");
+  GRETA_REQUIRE(out_fmt == GRETA_OUT_F32 || out_fmt == GRETA_OUT_F16 || out_fmt == GRETA_OUT_BF16, "rms_norm: output format %d", out_fmt);
+  const int vec = D <= 8192 && D % 4 == 0 && ldx % 4 == 0 && ld_out % 4 == 0 && aligned16(x) && aligned16(w) && aligned16(out);
+  GRETA_CUDA_TRY(launch_pdl(norm_kernel<true>, dim3(M), dim3(256), 0, (cudaStream_t)stream, x, ldx, w, static_cast<const float *>(nullptr), eps, out, out_fmt,
+                            D, ld_out, vec));
+  return launched("norm_kernel");
 }
 
 int greta_cuda_embedding_positions(greta_stream_t stream, const int32_t *tokens, const void *table, const void *pos_table, int fmt, float *out, uint32_t M,
@@ -388,6 +429,21 @@ int greta_cuda_embedding_positions(greta_stream_t stream, const int32_t *tokens,
     GRETA_CUDA_TRY(launch_pdl(embedding_positions_kernel<float>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, tokens, table, pos_table, out, M, D, vocab,
                               max_positions, d_pos, pos0));
   return launched("embedding_positions_kernel");
+}
+
+int greta_cuda_embedding_scaled(greta_stream_t stream, const int32_t *tokens, const void *table, int fmt, uint32_t ld, float scale, float *out, uint32_t M,
+                                uint32_t D, uint32_t vocab) {
+  if (M == 0 || D == 0) return GRETA_OK;
+  GRETA_REQUIRE(tokens && table && out && ld >= D, "embedding_scaled: bad argument");
+  GRETA_REQUIRE(fmt == GRETA_FMT_BF16 || fmt == GRETA_FMT_F32, "embedding_scaled: table format %d", fmt);
+  const unsigned grid = (unsigned)(((size_t)M * D + 255) / 256);
+  if (fmt == GRETA_FMT_BF16)
+    GRETA_CUDA_TRY(launch_pdl(embedding_scaled_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, tokens,
+                              static_cast<const __nv_bfloat16 *>(table), ld, scale, out, M, D, vocab));
+  else
+    GRETA_CUDA_TRY(launch_pdl(embedding_scaled_kernel<float>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, tokens, static_cast<const float *>(table), ld,
+                              scale, out, M, D, vocab));
+  return launched("embedding_scaled_kernel");
 }
 
 int greta_cuda_gather_rows(greta_stream_t stream, const float *x, uint32_t D, const uint32_t *rows, uint32_t n, float *out) {

@@ -133,7 +133,7 @@ int open_model(ModelConfig k, WeightLoader *loader, int fmt, uint32_t batch, uin
   }
   m->cfg = k;
   const bool ok = m->sched.init(k, &err) && m->sched.allocate_weights(&err) && (!loader || m->sched.load_weights(*loader, &err)) &&
-                  m->sched.allocate_activations(batch, max_seq ? max_seq : k.max_seq_len, &err) && m->gen.init(k, &m->sched, &err);
+                  m->sched.allocate_activations(batch, max_seq ? max_seq : k.default_positions(), &err) && m->gen.init(k, &m->sched, &err);
   if (!ok) return done(false, err);
   *out = m.release();
   return 0;

@@ -74,14 +74,14 @@ def _load(libname, header):
 
 
 # Structures of the dense linears and the mixers (include/greta_cuda.h).
-ACT_NONE, ACT_GELU_ERF, ACT_SIGMOID, ACT_TANH, ACT_DELTA_DECAY = range(5)
-OUT_F32, OUT_BF16, OUT_BF16_PAIR = 0, 2, 10
+ACT_NONE, ACT_GELU_ERF, ACT_SIGMOID, ACT_TANH, ACT_DELTA_DECAY, ACT_RELU2, ACT_SOFTPLUS_DECAY = range(7)
+OUT_F32, OUT_F16, OUT_BF16, OUT_BF16_PAIR = 0, 1, 2, 10
 _U, _F, _P = C.c_uint32, C.c_float, C.c_void_p
 
 
 class OutSegment(C.Structure):
     _fields_ = [("row0", _U), ("rows", _U), ("act", C.c_int), ("out_fmt", C.c_int), ("accumulate", C.c_int), ("bias", _P), ("out", _P), ("ld", _U),
-                ("col0", _U), ("pair_offset", _U)]
+                ("col0", _U), ("pair_offset", _U), ("rate", _P)]
 
 
 class Linear(C.Structure):

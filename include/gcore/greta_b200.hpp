@@ -352,9 +352,20 @@ public:
 
 namespace gcore::inference {
 
-// Layer kinds of the hybrid designs (unquantised weights, one pre-norm per layer, mixer and feed-forward side by side:
-// x += mixer(LN(x)) + ff(LN(x))).  A design is a list of layers; every size and constant is a field here.
-enum class MixerKind { WINDOW_ATTENTION, GENERAL_DELTA };
+// Layer kinds of the hybrid designs (unquantised weights).  A design is a list of layers; every size and constant is a field here.
+enum class MixerKind { WINDOW_ATTENTION, GENERAL_DELTA, LATENT_ATTENTION, GATED_DELTA };
+// Rotary positions: pairs (i, i + dims / 2), or neighbours (interleaved), turned by position * frequency i.
+struct RotarySpec {
+  uint32_t dims = 0;
+  bool interleaved = false;
+  double base = 10000.0;
+  double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;  // YaRN; factor 0 = none
+  bool operator==(const RotarySpec &o) const {
+    return dims == o.dims && interleaved == o.interleaved && base == o.base && factor == o.factor && original == o.original && fast == o.fast && slow == o.slow;
+  }
+  // Frequency of every pair, and the amplitude of cos and sin.
+  std::vector<double> frequencies(double *amplitude) const;
+};
 struct MixerSpec {
   MixerKind kind = MixerKind::WINDOW_ATTENTION;
   uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0;  // general delta: heads and dim only
@@ -362,14 +373,32 @@ struct MixerSpec {
   uint32_t window = 0, keep_first = 0;                  // window 0 = every earlier position
   float scale = 1.0f, softcap = 0.0f;                   // softcap 0 = none
   bool temp = false, distance_bias = false, sink = false;  // per-head vectors that the layer has
-  uint32_t rank = 0;                                    // general delta: width of the low-rank decay path
-  // Projected columns in front of the feed-forward's: attention q|k|v; delta r|k|v|gate|a (the low-rank path follows).
-  uint32_t proj_cols() const { return kind == MixerKind::GENERAL_DELTA ? 5 * heads * dim : (heads + kv_heads) * dim + kv_heads * vdim; }
+  uint32_t rank = 0, gate_rank = 0;                     // delta rules: width of the low-rank decay path (gated: and of the output gate's)
+  uint32_t q_rank = 0, kv_rank = 0, rot_dim = 0;        // latent attention: query latent (0 = direct), key/value latent, rotated part
+  bool gate = false;                                    // latent attention: sigmoid gate on the heads' outputs
+  RotarySpec rotary;
+  // Projected fp32 columns: attention q|k|v; general delta r|k|v|gate|a; latent q or its latent|down|gate; gated delta q|k|v|beta, each
+  // part on a multiple of 4 columns in the last two (the low-rank paths have their own buffers).
+  static uint32_t up4(uint32_t n) { return (n + 3u) & ~3u; }
+  uint32_t q_cols() const { return heads * (dim + rot_dim); }
+  uint32_t down_col() const { return up4(q_rank ? q_rank : q_cols()); }
+  uint32_t gate_col() const { return down_col() + up4(kv_rank + rot_dim); }
+  uint32_t conv_cols() const { return kind == MixerKind::GATED_DELTA ? 2 * kv_heads * dim + heads * vdim : (heads + kv_heads) * dim + kv_heads * vdim; }
+  uint32_t proj_cols() const {
+    switch (kind) {
+      case MixerKind::GENERAL_DELTA: return 5 * heads * dim;
+      case MixerKind::LATENT_ATTENTION: return gate_col() + (gate ? heads * vdim : 0);
+      case MixerKind::GATED_DELTA: return up4(conv_cols()) + heads;
+      default: return conv_cols();
+    }
+  }
   uint32_t out_cols() const { return kind == MixerKind::GENERAL_DELTA ? heads * dim : heads * vdim; }
 };
 struct LayerSpec {
   MixerSpec mixer;
-  uint32_t ff = 0;  // width of the gelu feed-forward; 0 = none
+  uint32_t ff = 0;               // width of the feed-forward; 0 = none
+  int ff_act = 1;                // GRETA_ACT_* between its two products (gelu)
+  bool parallel = true;          // mixer and feed-forward side by side on one norm; false: one after the other, a norm each
 };
 enum class ModelArch { LLAMA, HYBRID };
 
@@ -391,11 +420,18 @@ struct ModelConfig {
   // Tensor parallelism (Megatron style): this process holds shard tp_rank of tp_size.
   uint32_t tp_rank = 0, tp_size = 1;
   // Which layers the scheduler runs.  HYBRID: `layers` describes them, dim is the width, rms_eps the epsilon of every norm,
-  // max_seq_len the number of learned positions, weight_type BF16 or FP32 (FP32: everything in 32-bit).
+  // max_seq_len the number of learned positions (or the most a sequence may have), weight_type BF16 or FP32 (FP32: everything in
+  // 32-bit).
   ModelArch arch = ModelArch::LLAMA;
   std::string architecture;        // name in the model registry
   std::vector<LayerSpec> layers;
   uint32_t prefill_chunk = 2048;   // HYBRID: most positions of a prompt that run at once (longer prompts run in portions)
+  bool learned_positions = true;   // HYBRID: a position table is added to the embedding
+  bool rms_norms = false;          // HYBRID: root-mean-square norms without offsets instead of layer norms
+  bool tied_head = false;          // HYBRID: the LM head is the embedding table
+  float embed_scale = 1.0f;        // HYBRID: factor on the embedding
+  uint32_t default_seq_len = 0;    // positions of a sequence when the caller names no number; 0 = max_seq_len
+  uint32_t default_positions() const { return default_seq_len ? default_seq_len : max_seq_len; }
 
   static ModelConfig llama2_7b() { return ModelConfig{}; }
   static ModelConfig llama2_13b() {
@@ -516,15 +552,22 @@ struct ActivationBuffers {
   gcore::rt::cuda::Buffer tokens, d_pos, d_next, attn_scratch, gemm_ws, out_tokens;
 };
 
-// One layer of a hybrid design: everything that reads the norm's output packed in one weight (w_in), both sublayers' output
-// projections side by side in another (w_out: [mixer | feed-forward] columns), and the sequences' caches or states.
+// One layer of a hybrid design: everything of the mixer that reads the norm's output packed in one weight (w_in), its output
+// projection in another (w_out).  Parallel layers have the feed-forward in the same two (w_out: [mixer | feed-forward] columns),
+// sequential ones in w_up and w_down behind a norm of their own.  And the sequences' caches or states.
 struct HybridLayerBuffers {
   gcore::rt::cuda::Buffer norm_w, norm_b, w_in, w_out;
   uint32_t in_rows = 0, in_ld = 0, out_cols = 0, out_ld = 0, ff_col = 0;  // ff_col: first feed-forward column of w_out
+  gcore::rt::cuda::Buffer norm2_w, w_up, w_down;
+  uint32_t up_ld = 0, down_ld = 0;
   gcore::rt::cuda::Buffer temp, r1, r2, sink, conv;                       // attention, fp32
   gcore::rt::cuda::Buffer w2, w2_packed, w0, a_bias, out_norm;            // general delta; w2 fp32, w2_packed for portions
-  uint32_t w2_ld = 0;
-  gcore::rt::cuda::Buffer k_cache, v_cache, history, state;               // [slots][...]
+  uint32_t w2_ld = 0;                                                     // gated delta: w2 decay, g2 gate, w2_packed both, w0 its bias
+  gcore::rt::cuda::Buffer g2, rate;
+  gcore::rt::cuda::Buffer q_norm, w_uq, kv_norm, w_kv;                    // latent attention
+  uint32_t uq_ld = 0, kv_ld = 0;
+  size_t rotation = 0;                                                    // which of the scheduler's rotation tables
+  gcore::rt::cuda::Buffer k_cache, v_cache, history, state;               // [slots][...]; latent attention: k_cache alone
   uint32_t ring = 0;
 };
 
@@ -611,6 +654,16 @@ private:
   bool load_hybrid_synthetic(uint64_t seed, std::string *err);
   bool hybrid_embed(const int32_t *d_tokens, const greta_rows &rows, std::string *err);
   bool hybrid_layer(size_t layer, const greta_rows &rows, std::string *err);
+  // The steps of a layer.  x_norm_linear: norm of the residual rows, then the linear's segments; from_cat: a product of the mixer's or
+  // feed-forward's columns that adds to the residual.
+  bool x_norm_linear(greta_linear &lin, const gcore::rt::cuda::Buffer &norm_w, const gcore::rt::cuda::Buffer &norm_b, const greta_rows &rows, std::string *err);
+  bool from_cat(const gcore::rt::cuda::Buffer &w, uint32_t cols, uint32_t ld, const greta_rows &rows, std::string *err);
+  bool general_delta_core(size_t layer, const greta_rows &rows, std::string *err);
+  bool window_attention_core(size_t layer, const greta_rows &rows, std::string *err);
+  bool latent_attention_core(size_t layer, const greta_rows &rows, std::string *err);
+  bool gated_delta_core(size_t layer, const greta_rows &rows, std::string *err);
+  bool few_rows(const greta_rows &rows) const;          // the linears run as GEMVs
+  void *cat_buffer(const greta_rows &rows, int *fmt);   // where mixers and feed-forwards leave what the output projections read
   bool hybrid_logits(const float *x, uint32_t n, float *logits, std::string *err);
   // Runs seq_len tokens in portions; after each, `after(first row, rows)` sees its hidden rows in activations_.x.
   bool hybrid_run(const int32_t *tokens, size_t seq_start, size_t seq_len, const std::function<bool(size_t, size_t)> &after, std::string *err);
@@ -634,7 +687,11 @@ private:
   struct HybridActivations {
     gcore::rt::cuda::Buffer h, proj, cat, cat16, q, low, low16, decay, o, x_rows, logits_rows;
     uint32_t h_ld = 0, proj_ld = 0, cat_ld = 0, low_ld = 0, low16_ld = 0, decay_ld = 0;
+    gcore::rt::cuda::Buffer q_latent, latent_scratch, k_expanded, v_expanded, u, gate;  // latent attention; gated delta
+    uint32_t q_latent_ld = 0, u_ld = 0, gate_ld = 0;
   } hact_;
+  std::vector<RotarySpec> rotations_;                    // distinct rotations of the model and their tables
+  std::vector<gcore::rt::cuda::Buffer> rotation_tables_;  // [positions][dims / 2][cos, sin] fp32
   gcore::rt::cuda::Buffer pos_embd_, final_norm_b_;
   uint32_t head_ld_ = 0;
   uint64_t weight_bytes_ = 0;

@@ -430,9 +430,17 @@ GRETA_API int greta_cuda_argmax_advance_batch(greta_stream_t stream, const float
  * weight rows with its own bias, activation, destination and storage type, applied in the kernel's epilogue:
  *   out[m * ld + col0 + (n - row0)]  =  act(W[n] . x[m] + bias[n - row0])     (accumulate: added to what is there, fp32)
  * ldw is a multiple of 64 elements; W is 16-byte aligned. */
-enum { GRETA_ACT_NONE = 0, GRETA_ACT_GELU_ERF = 1, GRETA_ACT_SIGMOID = 2, GRETA_ACT_TANH = 3, GRETA_ACT_DELTA_DECAY = 4 /* exp(-exp(-1/2) sigmoid(z)) */ };
-/* Storage of an output: fp32, bf16, or a bf16 pair (hi at the element's place, lo = bf16(z - hi) pair_offset elements on). */
-enum { GRETA_OUT_F32 = 0, GRETA_OUT_BF16 = 2, GRETA_OUT_BF16_PAIR = 10 };
+enum {
+  GRETA_ACT_NONE = 0,
+  GRETA_ACT_GELU_ERF = 1,
+  GRETA_ACT_SIGMOID = 2,
+  GRETA_ACT_TANH = 3,
+  GRETA_ACT_DELTA_DECAY = 4,    /* exp(-exp(-1/2) sigmoid(z)) */
+  GRETA_ACT_RELU2 = 5,          /* max(z, 0)^2 */
+  GRETA_ACT_SOFTPLUS_DECAY = 6  /* exp(-rate softplus(z)), one rate per row of the segment */
+};
+/* Storage of an output: fp32, fp16, bf16, or a bf16 pair (hi at the element's place, lo = bf16(z - hi) pair_offset elements on). */
+enum { GRETA_OUT_F32 = 0, GRETA_OUT_F16 = 1, GRETA_OUT_BF16 = 2, GRETA_OUT_BF16_PAIR = 10 };
 #define GRETA_MAX_SEGMENTS 8
 typedef struct greta_out_segment {
   uint32_t row0, rows;
@@ -440,31 +448,39 @@ typedef struct greta_out_segment {
   const float *bias; /* [rows] or NULL */
   void *out;
   uint32_t ld, col0, pair_offset;
+  const float *rate; /* [rows], GRETA_ACT_SOFTPLUS_DECAY only */
 } greta_out_segment;
 typedef struct greta_linear {
-  int fmt;           /* GRETA_FMT_BF16 or GRETA_FMT_F32 */
+  int fmt;           /* GRETA_FMT_BF16 or GRETA_FMT_F32; greta_cuda_linear_gemm also GRETA_FMT_F16 */
   const void *w;
   uint32_t N, K, ldw;
   uint32_t n_segments;
   greta_out_segment seg[GRETA_MAX_SEGMENTS];
 } greta_linear;
 /* Few rows (1 <= M <= 8): weights streamed once for all rows, activations in fp32 whatever the weights' format.  With
- * ln_w / ln_b the input rows are layer-normalised on the way in (K = width of the norm). x [M][ldx]. */
+ * ln_w / ln_b the input rows are layer-normalised on the way in (K = width of the norm); ln_b NULL: divided by their root
+ * mean square instead (no mean, no offset).  x [M][ldx]. */
 GRETA_API int greta_cuda_linear_gemv(greta_stream_t stream, const greta_linear *lin, const float *x, uint32_t ldx, const float *ln_w,
                                      const float *ln_b, float eps, uint32_t M);
-/* Many rows.  BF16: tensor cores (tcgen05), x is bf16 [M][ldx], ldx a multiple of 8 and its columns K .. ldw-1 zero where
- * ldx >= ldw.  F32: true 32-bit products on the CUDA cores, x is fp32 [M][ldx], ldx >= ldw, zero-padded. */
+/* Many rows.  BF16 / F16: tensor cores (tcgen05), x is of the weights' type, [M][ldx], ldx a multiple of 8; columns past K are
+ * not read.  F32: true 32-bit products on the CUDA cores, x is fp32 [M][ldx], ldx >= ldw, zero-padded. */
 GRETA_API int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *lin, const void *x, uint32_t ldx, uint32_t M);
 /* greta_cuda_gemm_status for the kernels of greta_cuda_linear_gemm. */
 GRETA_API int greta_cuda_linear_gemm_status(int *code);
-/* y = (x - mean) / sqrt(var + eps) * w + b per row of D values; out fp32 or bf16 (GRETA_OUT_*), row stride ld_out. */
+/* y = (x - mean) / sqrt(var + eps) * w + b per row of D values; out fp32, fp16 or bf16 (GRETA_OUT_*), row stride ld_out. */
 GRETA_API int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w, const float *b, float eps, void *out, int out_fmt,
                                     uint32_t M, uint32_t D, uint32_t ld_out);
+/* y = x / sqrt(mean(x^2) + eps) * w per row of D values, rows ldx apart. */
+GRETA_API int greta_cuda_rms_norm(greta_stream_t stream, const float *x, uint32_t ldx, const float *w, float eps, void *out, int out_fmt, uint32_t M,
+                                  uint32_t D, uint32_t ld_out);
 /* out[m] = table[tokens[m]] + pos_table[p], p = d_pos[m] or pos0 + m; tables in fmt BF16 or F32; ids or positions outside
  * their table contribute zeros. */
 GRETA_API int greta_cuda_embedding_positions(greta_stream_t stream, const int32_t *tokens, const void *table, const void *pos_table, int fmt,
                                              float *out, uint32_t M, uint32_t D, uint32_t vocab, uint32_t max_positions, const uint32_t *d_pos,
                                              uint32_t pos0);
+/* out[m] = scale * table[tokens[m]], table rows ld elements apart; ids outside the table give zeros. */
+GRETA_API int greta_cuda_embedding_scaled(greta_stream_t stream, const int32_t *tokens, const void *table, int fmt, uint32_t ld, float scale, float *out,
+                                          uint32_t M, uint32_t D, uint32_t vocab);
 /* out[i] = x[rows[i]], rows of D floats (n <= 64, row numbers on the host). */
 GRETA_API int greta_cuda_gather_rows(greta_stream_t stream, const float *x, uint32_t D, const uint32_t *rows, uint32_t n, float *out);
 
@@ -508,6 +524,47 @@ GRETA_API int greta_cuda_window_attn(greta_stream_t stream, const greta_window_a
 GRETA_API int greta_cuda_window_attn_prefill(greta_stream_t stream, const greta_window_attn *a, const greta_rows *rows, const float *q,
                                              void *out, int out_fmt, uint32_t ld_out);
 
+/* ------------------------------------------------------------------ latent attention
+ * Keys and values of all heads come from one latent per token, c = RMS(down[0 .. rank)) * latent_norm, and one rotated key part
+ * kr = rotate(down[rank .. rank + rot_dim)):
+ *   k_h = W_uk,h c   v_h = W_uv,h c   s = (q_h . k_h + rotate(qr_h) . kr) scale   softmax over j <= i, exp(sink_h) added to the
+ *   denominator (sink NULL: none)   out_h = gate_h * sum p v_h (gate NULL: none)
+ * Only c and kr are cached: [slots][cap][rank16 | rot16] (rank16, rot16: rounded up to 16, zero-padded), F16 or F32.
+ * Rotation: the first rot_dims of the rot_dim channels in pairs, (i, i + rot_dims / 2) or (2 i, 2 i + 1); `rotation` holds cos and
+ * sin (with any amplitude) of the angle of pair i at position p: [positions][rot_dims / 2][2].
+ * w_kv: [heads][dim8] rows of W_uk, then [heads][vdim8] rows of W_uv (dim8, vdim8: rounded up to 8, zero rows), ld_w elements
+ * apart (a multiple of 64), of the cache's type. */
+typedef struct greta_latent_attn {
+  uint32_t heads, dim, rot_dim, vdim, rank;
+  uint32_t rot_dims, interleaved;
+  uint32_t cap, positions;
+  float scale, eps;
+  const float *rotation, *sink, *latent_norm;
+  const float *q;    /* [M][heads][dim + rot_dim], rows ld_q apart, not rotated */
+  uint32_t ld_q;
+  const float *down; /* [M][rank + rot_dim], rows ld_down apart */
+  uint32_t ld_down;
+  const float *gate; /* [M][heads * vdim], rows ld_gate apart */
+  uint32_t ld_gate;
+  int fmt;           /* GRETA_FMT_F16 or GRETA_FMT_F32: cache and w_kv; F32 also selects true 32-bit arithmetic */
+  const void *w_kv;
+  uint32_t ld_w;
+  void *cache;
+} greta_latent_attn;
+GRETA_API uint32_t greta_cuda_latent_row(uint32_t rank, uint32_t rot_dim); /* elements of a cache row */
+/* Norm, rotation and cache write of a portion's rows. */
+GRETA_API int greta_cuda_latent_cache(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows);
+/* Absorbed form (decode and short portions): q_h W_uk,h meets the cached latents themselves, W_uv,h is applied to the weighted sum of
+ * latents.  Writes the rows' cache entries as well.  scratch: greta_cuda_latent_scratch_bytes for at least these rows;
+ * max_len bounds the position of any row plus one. */
+GRETA_API size_t greta_cuda_latent_scratch_bytes(const greta_latent_attn *a, uint32_t M, uint32_t max_len);
+GRETA_API int greta_cuda_latent_absorbed(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, void *scratch, void *out,
+                                         int out_fmt, uint32_t ld_out, uint32_t max_len);
+/* Expanded form (prompts; F16): k [pos0 + M][heads * dim8] and v [pos0 + M][heads * vdim8] in fp16 are the products of the cached
+ * latents with w_kv (greta_cuda_linear_gemm).  The rows' cache entries must be there. */
+GRETA_API int greta_cuda_latent_prefill(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, const void *k, const void *v,
+                                        void *out, int out_fmt, uint32_t ld_out);
+
 /* ------------------------------------------------------------------ generalised delta rule
  * Per head, key dimension = value dimension = dim, state S [dim x dim] in fp32, zero in front of position 0:
  *   u = k / sqrt(k.k + 1e-6);  S <- diag(w) S - (a * u)(u^T S) + k v^T;  o = S^T r
@@ -533,6 +590,47 @@ GRETA_API int greta_cuda_delta_step(greta_stream_t stream, const greta_delta_rul
 GRETA_API int greta_cuda_delta_scan(greta_stream_t stream, const greta_delta_rule *d, const greta_rows *rows, float *o_buf);
 GRETA_API int greta_cuda_delta_output(greta_stream_t stream, const greta_delta_rule *d, const float *o_buf, uint32_t M, void *out, int out_fmt,
                                       uint32_t ld_out);
+
+/* ------------------------------------------------------------------ gated delta rule with a decay per key channel
+ * Per value head h (query / key head h / (heads / kv_heads)), state S [dim x vdim] in fp32, zero in front of position 0:
+ *   S <- diag(g) S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q
+ * out_h = o / rms(o) * norm * gate_h.  Before that q, k and v pass a short causal convolution over time (conv [channels][taps],
+ * no bias, zeros in front of the start) and silu, q and k are divided by sqrt(sum of squares + 1e-6), q times dim^(-1/2).
+ * g = exp(-rate softplus(A2 t + dt_bias)),  gate = sigmoid(G2 t'),  t and t' low-rank activations.
+ * proj: fp32 [M][q: kv_heads*dim | k: kv_heads*dim | v: heads*vdim], C channels; history [slots][taps][C], the projected row of
+ * position p in row p % taps; state [slots][heads][vdim columns][dim32 rows] (dim32: rounded up to 32). */
+typedef struct greta_gated_delta {
+  uint32_t heads, kv_heads, dim, vdim, taps, rank_a, rank_g;
+  float eps;
+  const float *proj;
+  uint32_t ld_proj;
+  const float *conv;
+  float *history;
+  const float *beta;             /* [M][heads], rows ld_beta apart, after the sigmoid */
+  uint32_t ld_beta;
+  const float *norm;             /* [vdim] */
+  float *state;
+  /* one token per sequence */
+  const float *low;              /* [M][t: rank_a at column 0 | t': rank_g at column low_g], rows ld_low apart */
+  uint32_t ld_low, low_g;
+  const float *a2, *g2;          /* [heads*dim][rank_a], [heads*vdim][rank_g] */
+  const float *rate, *dt_bias;   /* [heads*dim] */
+  /* portions */
+  float *u;                      /* [M][C]: q, k, v as they enter the recurrence; written by _prepare */
+  uint32_t ld_u;
+  const float *decay, *gate;     /* [M][heads*dim], [M][heads*vdim] */
+  uint32_t ld_decay, ld_gate;
+} greta_gated_delta;
+GRETA_API size_t greta_cuda_gated_delta_state_bytes(uint32_t heads, uint32_t dim, uint32_t vdim); /* of one sequence */
+/* One new token per sequence (rows->d_pos set): convolution, decay, state update, read-out, norm and gate in one kernel. */
+GRETA_API int greta_cuda_gated_delta_step(greta_stream_t stream, const greta_gated_delta *d, const greta_rows *rows, void *out, int out_fmt,
+                                          uint32_t ld_out);
+/* A portion: convolution, silu and unit norms -> u, and the history's new rows; the recurrence, o -> o_buf fp32 [M][heads*vdim];
+ * norm and gate. */
+GRETA_API int greta_cuda_gated_delta_prepare(greta_stream_t stream, const greta_gated_delta *d, const greta_rows *rows);
+GRETA_API int greta_cuda_gated_delta_scan(greta_stream_t stream, const greta_gated_delta *d, const greta_rows *rows, float *o_buf);
+GRETA_API int greta_cuda_gated_delta_output(greta_stream_t stream, const greta_gated_delta *d, const float *o_buf, uint32_t M, void *out, int out_fmt,
+                                            uint32_t ld_out);
 
 /* ------------------------------------------------------------------ tensor-parallel exchange
  * The reference is single-GPU (hipSetDevice(0), greta_runtime_hip.cpp:153); these are new.
