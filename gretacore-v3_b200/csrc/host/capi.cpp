@@ -172,6 +172,16 @@ int greta_host_check_config(const char *json) {
   ModelConfig k;
   return done(json && config_from_json(json, nullptr, &k, &err), err);
 }
+int greta_host_rotary(uint32_t dims, double base, const double *yarn4, double *freq, double *amplitude) {
+  if (!dims || dims % 2 || !(base > 0) || !freq || !amplitude) return done(false, "rotary: bad argument");
+  RotarySpec s;
+  s.dims = dims;
+  s.base = base;
+  if (yarn4) s.factor = yarn4[0], s.original = yarn4[1], s.fast = yarn4[2], s.slow = yarn4[3];
+  const std::vector<double> f = s.frequencies(amplitude);
+  std::copy(f.begin(), f.end(), freq);
+  return 0;
+}
 int greta_model_destroy(greta_model_t m) {
   delete static_cast<Model *>(m);
   return 0;

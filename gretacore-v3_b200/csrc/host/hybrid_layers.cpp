@@ -150,13 +150,16 @@ bool BlockScheduler::init_hybrid(std::string *err) {
     if (m.kind == MixerKind::LATENT_ATTENTION && (!m.kv_rank || m.kv_rank > 1024 || !m.rot_dim || m.rot_dim > 128))
       return fail(err, "init: latent attention needs a latent of 1..1024 and a rotated part of 1..128");
   }
+  rotations_.clear();
+  for (const LayerSpec &l : c.layers)
+    if (l.mixer.kind == MixerKind::LATENT_ATTENTION && std::find(rotations_.begin(), rotations_.end(), l.mixer.rotary) == rotations_.end())
+      rotations_.push_back(l.mixer.rotary);
   if (gcore::rt::GretaContext::instance().initialize() != gcore::rt::GretaResult::SUCCESS)
     return fail(err, "init: no usable CUDA device (this path has no CPU fallback)");
   vocab_l_ = c.vocab_size;
   stream_ = gcore::rt::GretaContext::instance().create_stream();
   blocks_.clear();
   hybrid_.clear();
-  rotations_.clear();
   initialized_ = true;
   return true;
 }
@@ -260,7 +263,6 @@ bool BlockScheduler::load_hybrid(TensorSource &src, std::string *err) {
       if (!kv.upload(b.w_kv, err)) return false;
       weight_bytes_ += b.w_kv.size();
       b.rotation = std::find(rotations_.begin(), rotations_.end(), m.rotary) - rotations_.begin();
-      if (b.rotation == rotations_.size()) rotations_.push_back(m.rotary);
     } else if (m.kind == MixerKind::GATED_DELTA) {
       if (!rows(mix + "q", GD) || !rows(mix + "k", GD) || !rows(mix + "v", HV) || !rows(mix + "b", m.heads) || !rows(mix + "a1", m.rank) ||
           !rows(mix + "g1", m.gate_rank) || !convolution({{"q", GD}, {"k", GD}, {"v", HV}}) || !vec(mix + "dt_bias", HD, b.w0) ||

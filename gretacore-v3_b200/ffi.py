@@ -103,6 +103,18 @@ class DeltaRule(C.Structure):
                [("ld_decay", _U), ("t", _P), ("ld_t", _U), ("w2", _P), ("w0", _P), ("norm", _P), ("state", _P)]
 
 
+class LatentAttn(C.Structure):
+    _fields_ = [(n, _U) for n in ("heads", "dim", "rot_dim", "vdim", "rank", "rot_dims", "interleaved", "cap", "positions")] + \
+               [("scale", _F), ("eps", _F)] + [(n, _P) for n in ("rotation", "sink", "latent_norm", "q")] + \
+               [("ld_q", _U), ("down", _P), ("ld_down", _U), ("gate", _P), ("ld_gate", _U), ("fmt", C.c_int), ("w_kv", _P), ("ld_w", _U), ("cache", _P)]
+
+
+class GatedDelta(C.Structure):
+    _fields_ = [(n, _U) for n in ("heads", "kv_heads", "dim", "vdim", "taps", "rank_a", "rank_g")] + [("eps", _F), ("proj", _P), ("ld_proj", _U)] + \
+               [(n, _P) for n in ("conv", "history", "beta")] + [("ld_beta", _U), ("norm", _P), ("state", _P), ("low", _P), ("ld_low", _U), ("low_g", _U)] + \
+               [(n, _P) for n in ("a2", "g2", "rate", "dt_bias", "u")] + [("ld_u", _U), ("decay", _P), ("gate", _P), ("ld_decay", _U), ("ld_gate", _U)]
+
+
 def cuda():
     return _load("libgreta_cuda.so", "greta_cuda.h")
 

@@ -61,7 +61,8 @@ GRETA_API int greta_model_create(const greta_model_config *cfg, greta_model_t *o
 GRETA_API int greta_model_create_batch(const greta_model_config *cfg, uint32_t batch, greta_model_t *out);
 /* Model folders (config.json + model.safetensors, read through the model registry) and GGUF files: create, load the weights
  * and allocate `batch` sequences.  fmt: GRETA_FMT_BF16, or GRETA_FMT_F32 to run an unquantised design in true 32-bit (ignored
- * for GGUF files).  max_seq 0: the model's own limit; prefill_chunk 0: the default portion size. */
+ * for GGUF files).  max_seq 0: the model's own limit (8192 where the
+ * design has none); prefill_chunk 0: the default portion size. */
 GRETA_API int greta_model_open(const char *path, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk, greta_model_t *out);
 /* The same from the text of a config.json, without weights: follow with greta_model_load_synthetic. */
 GRETA_API int greta_model_create_from_json(const char *config_json, int fmt, uint32_t batch, uint32_t max_seq, uint32_t prefill_chunk,
@@ -72,6 +73,8 @@ GRETA_API int greta_model_info(greta_model_t m, uint32_t *out5);
 GRETA_API const char *greta_host_architectures(void);
 /* config.json text -> checked, without a device (shape-dependent parts take their defaults). */
 GRETA_API int greta_host_check_config(const char *config_json);
+/* RotarySpec::frequencies: dims / 2 frequencies and the amplitude of cos and sin.  yarn4 = {factor, original, fast, slow}, or NULL. */
+GRETA_API int greta_host_rotary(uint32_t dims, double base, const double *yarn4, double *freq, double *amplitude);
 GRETA_API int greta_model_destroy(greta_model_t m);
 GRETA_API int greta_model_load_synthetic(greta_model_t m, uint64_t seed);                 /* load_synthetic_weights */
 /* BlockScheduler::load_weights from a GGUF file whose projections are stored as Q4_0 / Q8_0: blocks go to the device as
