@@ -515,77 +515,86 @@ def hybrid_config(z, max_positions):
             "layers": [delta if i % 2 == 0 else attn for i in range(z["layers"])]}
 
 
+def model_throughput(pkg, make, vocab, context):
+    """Prefill (512 and 2048 tokens) and decode (batches of 1, 8 and 16 behind `context` tokens) of make(batch), which returns a model
+    without weights.  Device times (events on the model's stream); a model's weights exceed L2, so nothing is served from it between steps."""
+    lib = pkg.ffi.cuda()
+    peak, _ = measured_peak_gbs()
+    res = {}
+    for batch in (1, 8, 16):
+        m = make(batch)
+        m.load_synthetic(1)
+        toks = pkg.model.synth_tokens(1, context, vocab)
+        sampler = ClockSampler(0)
+        sampler.start()
+        t0 = time.time()
+        if batch == 1:
+            for T in (512, 2048):
+                m.forward_timed(toks[:T], 3)
+                res[f"prefill_{T}_tok_per_s"] = round(T / min(m.forward_timed(toks[:T], 5) for _ in range(3)) * 1e3)
+        for b in range(batch):
+            if batch > 1:
+                m.set_sequence(b)
+            m.forward(toks, 0)
+        m.begin_decode(1 if batch == 1 else [1] * batch, context)
+        m.decode_timed(16)
+        n0 = lib.greta_cuda_launch_count()
+        ms = m.decode_timed(128) / 128
+        res[f"decode_b{batch}_tok_per_s"] = round(batch / ms * 1e3)
+        res[f"decode_b{batch}_us_per_step"] = round(ms * 1e3, 1)
+        res[f"decode_b{batch}_weight_stream_frac_of_peak"] = round(m.weight_bytes() / ms / 1e6 / peak, 3)
+        res["launches_per_step"] = (lib.greta_cuda_launch_count() - n0) / 128
+        res["clocks"] = sampler.stop(t0, time.time())
+        res["weight_bytes"] = m.weight_bytes()
+        m.close()
+    return res
+
+
 def hybrid_models(pkg):
     """Prefill and decode throughput of the hybrid design beside the Llama-shaped model of the same width, layers and weight
-    count (Q8_0).  Device times (events on the model's stream); a model's weights exceed L2, so nothing is served from it
-    between steps.  One JSON line per model and size."""
+    count (Q8_0).  One JSON line per model and size."""
     g = pkg.ffi
-    lib = g.cuda()
-    peak, peak_src = measured_peak_gbs()
+    _, peak_src = measured_peak_gbs()
     for name, z in HYBRID_SIZES.items():
-        for design in ("hybrid bf16", "llama q8_0"):
-            res = {}
-            for batch in (1, 8, 16):
-                if design == "hybrid bf16":
-                    m = pkg.model.Model.from_config(hybrid_config(z, 2560), batch=batch)
-                else:
-                    m = pkg.model.Model(dict(dim=z["width"], num_heads=z["heads"], num_heads_kv=z["kv"], num_layers=z["layers"], vocab=HYBRID_VOCAB,
-                                             hidden_dim=z["llama_ff"], head_dim=z["dim"], max_seq=2560, rope_base=10000.0, rms_eps=1e-5),
-                                        weight_fmt=g.FMT_Q8_0, batch=batch)
-                m.load_synthetic(1)
-                toks = pkg.model.synth_tokens(1, HYBRID_CONTEXT, HYBRID_VOCAB)
-                sampler = ClockSampler(0)
-                sampler.start()
-                t0 = time.time()
-                if batch == 1:
-                    for T in (512, 2048):
-                        m.forward_timed(toks[:T], 3)
-                        res[f"prefill_{T}_tok_per_s"] = round(T / min(m.forward_timed(toks[:T], 5) for _ in range(3)) * 1e3)
-                for b in range(batch):
-                    if batch > 1:
-                        m.set_sequence(b)
-                    m.forward(toks, 0)
-                m.begin_decode(1 if batch == 1 else [1] * batch, HYBRID_CONTEXT)
-                m.decode_timed(16)
-                n0 = lib.greta_cuda_launch_count()
-                ms = m.decode_timed(128) / 128
-                res[f"decode_b{batch}_tok_per_s"] = round(batch / ms * 1e3)
-                res[f"decode_b{batch}_us_per_step"] = round(ms * 1e3, 1)
-                res[f"decode_b{batch}_weight_stream_frac_of_peak"] = round(m.weight_bytes() / ms / 1e6 / peak, 3)
-                res["launches_per_step"] = (lib.greta_cuda_launch_count() - n0) / 128
-                res["clocks"] = sampler.stop(t0, time.time())
-                wb = m.weight_bytes()
-                m.close()
-            print(json.dumps({"case": "hybrid_models", "size": name, "design": design, "layers": z["layers"], "weight_bytes": wb, **res,
+        llama = dict(dim=z["width"], num_heads=z["heads"], num_heads_kv=z["kv"], num_layers=z["layers"], vocab=HYBRID_VOCAB, hidden_dim=z["llama_ff"],
+                     head_dim=z["dim"], max_seq=2560, rope_base=10000.0, rms_eps=1e-5)
+        designs = {"hybrid bf16": lambda b: pkg.model.Model.from_config(hybrid_config(z, 2560), batch=b),
+                   "llama q8_0": lambda b: pkg.model.Model(llama, weight_fmt=g.FMT_Q8_0, batch=b)}
+        for design, make in designs.items():
+            res = model_throughput(pkg, make, HYBRID_VOCAB, HYBRID_CONTEXT)
+            print(json.dumps({"case": "hybrid_models", "size": name, "design": design, "layers": z["layers"], **res,
                               "window": HYBRID_WINDOW, "context": HYBRID_CONTEXT, "peak_source": f"of {peak_src}"}), flush=True)
 
 
-def hybrid_kernels(pkg, only=None):
-    """The hybrid design's kernels and the like kernels of the Llama-shaped model, one by one, with the roofline each is held
-    against: HBM bytes, tensor-core FLOPs (bf16), or - the delta-rule scan - fp32 FMA throughput.  Buffers rotate beyond L2."""
-    import ctypes as C
-    g = pkg.ffi
-    lib = g.cuda()
-    peak, _ = measured_peak_gbs()
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            tc = float(json.load(f)["bf16_tflops"])
-    except Exception:
-        tc = 1590.0
-    fma = 148 * 128 * 2 * 1.965e9 / 1e12                     # TFLOP/s of 32-bit FMAs at the maximum clock
-    stream = C.c_void_p()
-    g.check(lib.greta_cuda_stream_create(C.byref(stream)))
-    e0, e1 = C.c_void_p(), C.c_void_p()
-    lib.greta_cuda_event_create(C.byref(e0))
-    lib.greta_cuda_event_create(C.byref(e1))
-    rng = np.random.default_rng(0)
+class KernelBench:
+    """Times single kernels: device buffers, and launches replayed in a graph over copies of the data that together exceed L2."""
 
-    def buf(nbytes, kind="zero"):
-        b = g.DeviceBuffer(int(nbytes), zero=True)
+    def __init__(self, pkg, case, only=None):
+        import ctypes as C
+        self.C, self.case, self.only, self.g = C, case, only, pkg.ffi
+        self.lib = self.g.cuda()
+        self.peak, _ = measured_peak_gbs()
+        try:
+            with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+                self.tc = float(json.load(f)["bf16_tflops"])
+        except Exception:
+            self.tc = 1590.0
+        self.fma = 148 * 128 * 2 * 1.965e9 / 1e12            # TFLOP/s of 32-bit FMAs at the maximum clock
+        self.stream = C.c_void_p()
+        self.g.check(self.lib.greta_cuda_stream_create(C.byref(self.stream)))
+        self.e0, self.e1 = C.c_void_p(), C.c_void_p()
+        self.lib.greta_cuda_event_create(C.byref(self.e0))
+        self.lib.greta_cuda_event_create(C.byref(self.e1))
+        self.rng = np.random.default_rng(0)
+
+    def buf(self, nbytes, kind="zero"):
+        b = self.g.DeviceBuffer(int(nbytes), zero=True)
         if kind == "bf16":
-            block = (np.abs(rng.normal(0, 0.02, 1 << 20)).astype(np.float32).view(np.uint32) >> 16).astype(np.uint16)
+            block = (np.abs(self.rng.normal(0, 0.02, 1 << 20)).astype(np.float32).view(np.uint32) >> 16).astype(np.uint16)
+        elif kind == "f16":
+            block = self.rng.normal(0, 0.5, 1 << 20).astype(np.float16)
         elif kind == "f32":
-            block = rng.normal(0, 0.5, 1 << 20).astype(np.float32)
+            block = self.rng.normal(0, 0.5, 1 << 20).astype(np.float32)
         else:
             return b
         raw = block.view(np.uint8)
@@ -593,48 +602,58 @@ def hybrid_kernels(pkg, only=None):
             b.upload(raw[:min(raw.size, int(nbytes) - at)], at)
         return b
 
-    def report(name, size, launches, copies, hbm=0.0, tensor=0.0, fp32=0.0):
+    def report(self, name, size, launches, copies, hbm=0.0, tensor=0.0, fp32=0.0):
         """launches(i) enqueues copy i; hbm bytes, tensor and fp32 flops of one launch."""
-        if only and only not in name:
+        if self.only and self.only not in name:
             return
+        C, g, lib = self.C, self.g, self.lib
         for i in range(copies):
             launches(i)
-        g.check(lib.greta_cuda_stream_synchronize(stream))
+        g.check(lib.greta_cuda_stream_synchronize(self.stream))
         graph, ex = C.c_void_p(), C.c_void_p()
         reps = max(1, 24 // copies)
-        g.check(lib.greta_cuda_graph_capture_begin(stream))
+        g.check(lib.greta_cuda_graph_capture_begin(self.stream))
         for _ in range(reps):
             for i in range(copies):
                 launches(i)
-        g.check(lib.greta_cuda_graph_capture_end(stream, C.byref(graph)))
+        g.check(lib.greta_cuda_graph_capture_end(self.stream, C.byref(graph)))
         g.check(lib.greta_cuda_graph_instantiate(graph, C.byref(ex)))
         best = 1e30
         for it in range(6):
-            lib.greta_cuda_event_record(e0, stream)
-            lib.greta_cuda_graph_launch(ex, stream)
-            lib.greta_cuda_event_record(e1, stream)
-            lib.greta_cuda_event_synchronize(e1)
+            lib.greta_cuda_event_record(self.e0, self.stream)
+            lib.greta_cuda_graph_launch(ex, self.stream)
+            lib.greta_cuda_event_record(self.e1, self.stream)
+            lib.greta_cuda_event_synchronize(self.e1)
             ms = C.c_float()
-            lib.greta_cuda_event_elapsed_ms(e0, e1, C.byref(ms))
+            lib.greta_cuda_event_elapsed_ms(self.e0, self.e1, C.byref(ms))
             if it >= 3:
                 best = min(best, ms.value)
         lib.greta_cuda_graph_exec_destroy(ex)
         lib.greta_cuda_graph_destroy(graph)
         us = best * 1e3 / (reps * copies)
-        roof = {"hbm": hbm / peak / 1e3, "tensor": tensor / tc / 1e6, "fp32": fp32 / fma / 1e6}
+        roof = {"hbm": hbm / self.peak / 1e3, "tensor": tensor / self.tc / 1e6, "fp32": fp32 / self.fma / 1e6}
         bound = max(roof, key=roof.get)
-        print(json.dumps({"case": "hybrid_kernels", "size": size, "kernel": name, "us": round(us, 2), "bound": bound,
+        print(json.dumps({"case": self.case, "size": size, "kernel": name, "us": round(us, 2), "bound": bound,
                           "roofline_us": round(roof[bound], 2), "frac": round(roof[bound] / us, 3)}), flush=True)
 
-    def dense(N, K, segs):
+    def dense(self, N, K, segs, fmt=None):
+        g = self.g
         ld = (K + 63) // 64 * 64
-        w = buf(N * ld * 2, "bf16")
-        lin = g.Linear(g.FMT_BF16, w.ptr, N, K, ld, len(segs))
+        w = self.buf(N * ld * 2, "bf16" if fmt is None else "f16")
+        lin = g.Linear(g.FMT_BF16 if fmt is None else fmt, w.ptr, N, K, ld, len(segs))
         row = 0
-        for i, (n, act, fmt, out, ldo, acc) in enumerate(segs):
-            lin.seg[i] = g.OutSegment(row, n, act, fmt, acc, None, out.ptr, ldo, 0, 0)
+        for i, (n, act, out_fmt, out, ldo, acc) in enumerate(segs):
+            lin.seg[i] = g.OutSegment(row, n, act, out_fmt, acc, None, out.ptr, ldo, 0, 0)
             row += n
         return w, lin
+
+
+def hybrid_kernels(pkg, only=None):
+    """The hybrid design's kernels and the like kernels of the Llama-shaped model, one by one, with the roofline each is held
+    against: HBM bytes, tensor-core FLOPs (bf16), or - the delta-rule scan - fp32 FMA throughput.  Buffers rotate beyond L2."""
+    import ctypes as C
+    kb = KernelBench(pkg, "hybrid_kernels", only)
+    g, lib, stream, buf, report, dense = kb.g, kb.lib, kb.stream, kb.buf, kb.report, kb.dense
 
     for size, z in HYBRID_SIZES.items():
         D, F, H, G, Dh = z["width"], z["ff"], z["heads"], z["kv"], z["dim"]
@@ -725,6 +744,122 @@ def hybrid_kernels(pkg, only=None):
         report("layer_norm T=2048", size, lambda i: g.check(lib.greta_cuda_layer_norm(stream, xs[i].ptr, ln.ptr, ln.ptr, 1e-6, cat.ptr, g.OUT_BF16, T, D, D)), 8,
                hbm=T * D * 6)
         del caches, att, states, ds, xs
+
+
+LATENT_SIZES = {  # latent heads, query latent, delta heads x 128; ff chosen for the weight count of the hybrid design of that width
+    "2048": dict(width=2048, heads=16, q_rank=768, delta_heads=16, ff=8576, layers=8),
+    "4096": dict(width=4096, heads=32, q_rank=1536, delta_heads=32, ff=17664, layers=4),
+}
+LATENT_DIM, LATENT_ROT, LATENT_RANK, LATENT_LOW = 128, 64, 512, 128
+
+
+def latent_config(z):
+    ff = {"kind": "dense", "ff": z["ff"]}
+    mix = {"heads": z["heads"], "dim": LATENT_DIM, "rot_dim": LATENT_ROT, "vdim": LATENT_DIM, "kv_rank": LATENT_RANK, "scale": (LATENT_DIM + LATENT_ROT) ** -0.5}
+    yarn = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    latent = {"type": "latent_attention", "mlp": ff, "mixer": dict(mix, q_rank=z["q_rank"], rot={"base": 10000.0, "dims": LATENT_ROT, "scaling": yarn})}
+    latent2 = {"type": "latent_attention_2", "mlp": ff, "mixer": dict(mix, rot={"base": 10000.0, "dims": LATENT_ROT})}
+    delta = {"type": "channel_delta", "mlp": ff, "mixer": {"heads": z["delta_heads"], "kv_heads": z["delta_heads"], "dim": 128, "vdim": 128, "conv": 4,
+                                                           "decay_rank": LATENT_LOW, "gate_rank": LATENT_LOW}}
+    return {"architecture": "Tetilorn", "width": z["width"], "vocab": HYBRID_VOCAB, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [[delta, latent, delta, latent2][i % 4] for i in range(z["layers"])]}
+
+
+def latent_models(pkg):
+    """Prefill and decode throughput of the latent attention / gated delta design beside the windowed attention / general delta design of the
+    same width, layers and weight count, both bf16.  One JSON line per model and size."""
+    _, peak_src = measured_peak_gbs()
+    for name, z in LATENT_SIZES.items():
+        designs = {"tetilorn bf16": lambda b: pkg.model.Model.from_config(latent_config(z), batch=b, max_seq=2560),
+                   "bidonex bf16": lambda b: pkg.model.Model.from_config(hybrid_config(HYBRID_SIZES[name], 2560), batch=b)}
+        for design, make in designs.items():
+            res = model_throughput(pkg, make, HYBRID_VOCAB, HYBRID_CONTEXT)
+            print(json.dumps({"case": "latent_models", "size": name, "design": design, "layers": z["layers"], **res, "context": HYBRID_CONTEXT,
+                              "peak_source": f"of {peak_src}"}), flush=True)
+
+
+def latent_kernels(pkg, only=None):
+    """The kernels of the latent attention / gated delta design one by one, each with its roofline (hybrid_kernels measures the like kernels
+    of the design it is compared with)."""
+    import ctypes as C
+    kb = KernelBench(pkg, "latent_kernels", only)
+    g, lib, stream, buf, report, dense = kb.g, kb.lib, kb.stream, kb.buf, kb.report, kb.dense
+    dim, rot, R, low_rank, T = LATENT_DIM, LATENT_ROT, LATENT_RANK, LATENT_LOW, 2048
+    for size, z in LATENT_SIZES.items():
+        D, F, H, Q, HE = z["width"], z["ff"], z["heads"], z["q_rank"], z["delta_heads"]
+        HV, HQ, cap = H * dim, H * (dim + rot), 2560
+        n_in = Q + R + rot + HV                              # query latent | latents | gate
+        x, xb, ln, cat = buf(T * max(D, F) * 4, "f32"), buf(T * max(F, D) * 2), buf(max(D, Q) * 4, "f32"), buf(T * max(F, HV) * 4)
+        res = buf(T * D * 4)
+        ld = (n_in + 3) // 4 * 4
+        proj, qb = buf(T * max(ld, 3 * HE * 128 + HE + 4) * 4, "f32"), buf(T * HQ * 4, "f32")
+        # dense products
+        for label, N, K, act, fmt, out, ldo, acc, cold in (("in (latent)", n_in, D, 0, g.OUT_F32, proj, ld, 0, 4e8), ("queries", HQ, Q, 0, g.OUT_F32, qb, HQ, 0, 2e8),
+                                                           ("up", F, D, g.ACT_RELU2, g.OUT_BF16, cat, F, 0, 4e8), ("down", D, F, 0, g.OUT_F32, res, D, 1, 4e8)):
+            copies = max(2, int(cold // (N * K * 2)))
+            ws = [dense(N, K, [(N, act, fmt, out, ldo, acc)]) for _ in range(copies)]
+            one_row = [g.Linear.from_buffer_copy(l) for _, l in ws]
+            for l in one_row:
+                l.seg[0].out_fmt = g.OUT_F32
+            norm = ln.ptr if label != "down" else None
+            report(f"linear_gemv {label} M=1", size, lambda i: g.check(lib.greta_cuda_linear_gemv(stream, C.byref(one_row[i]), x.ptr, K, norm, None, 1e-6, 1)), copies,
+                   hbm=N * K * 2)
+            for M in (16, 512, T):
+                report(f"linear_gemm {label} T={M}", size, lambda i: g.check(lib.greta_cuda_linear_gemm(stream, C.byref(ws[i][1]), xb.ptr, K, M)), copies,
+                       hbm=N * K * 2 + M * (K * 2 + N * (8 if acc else 2 if fmt == g.OUT_BF16 else 4)), tensor=2.0 * M * N * K)
+            del ws, one_row
+        # latent attention
+        row = lib.greta_cuda_latent_row(R, rot)
+        n_kv = 2 * H * dim
+        for b in (1, 16):
+            n_copy = max(2, int(2e8 // (b * cap * row * 2 + n_kv * R * 2)))
+            caches = [(buf(b * cap * row * 2, "f16"), buf(n_kv * R * 2, "f16")) for _ in range(n_copy)]
+            table, sink = buf(cap * rot * 4, "f32"), buf(H * 4, "f32")
+            att = [g.LatentAttn(H, dim, rot, dim, R, rot, 0, cap, cap, 0.07, 1e-6, table.ptr, sink.ptr, ln.ptr, qb.ptr, HQ, proj.ptr + 4 * Q, ld, proj.ptr + 4 * (Q + R + rot),
+                                ld, g.FMT_F16, w.ptr, R, c.ptr) for c, w in caches]
+            dpos = g.DeviceBuffer.from_numpy(np.full(b, HYBRID_CONTEXT, np.uint32))
+            rows = g.Rows(b, 0, 0, dpos.ptr)
+            scratch = buf(lib.greta_cuda_latent_scratch_bytes(C.byref(att[0]), b, cap))
+            report(f"latent absorbed decode M={b}", size, lambda i: g.check(lib.greta_cuda_latent_absorbed(stream, C.byref(att[i]), C.byref(rows), scratch.ptr, cat.ptr, 0, HV,
+                                                                                                         cap)), n_copy,
+                   hbm=b * HYBRID_CONTEXT * (R + rot) * 2 + n_kv * R * 2, tensor=b * HYBRID_CONTEXT * H * 2.0 * (2 * R + rot))
+            if b == 1:
+                many = g.Rows(T, 0, 0, None)
+                kx, vx = buf(cap * HV * 2, "f16"), buf(cap * HV * 2, "f16")
+                kv = g.Linear(g.FMT_F16, caches[0][1].ptr, n_kv, R, R, 2)
+                kv.seg[0] = g.OutSegment(0, HV, 0, g.OUT_F16, 0, None, kx.ptr, HV, 0, 0)
+                kv.seg[1] = g.OutSegment(HV, HV, 0, g.OUT_F16, 0, None, vx.ptr, HV, 0, 0)
+                qx = buf(T * lib.greta_cuda_latent_query_row(H, dim, rot) * 2)
+                report("latent_prepare T=2048", size, lambda i: g.check(lib.greta_cuda_latent_prepare(stream, C.byref(att[i]), C.byref(many), qx.ptr)), n_copy,
+                       hbm=T * ((R + rot) * 6 + HQ * 6))
+                report("linear_gemm keys and values T=2048", size, lambda i: g.check(lib.greta_cuda_linear_gemm(stream, C.byref(kv), caches[i][0].ptr, row, T)), n_copy,
+                       hbm=T * R * 2 + n_kv * R * 2 + T * n_kv * 2, tensor=2.0 * T * n_kv * R)
+                report("latent_prefill T=2048", size, lambda i: g.check(lib.greta_cuda_latent_prefill(stream, C.byref(att[i]), C.byref(many), qx.ptr, kx.ptr, vx.ptr, cat.ptr,
+                                                                                                    g.OUT_BF16, HV)), 2,
+                       tensor=2.0 * H * (2 * dim + rot) * T * (T + 1) / 2, hbm=T * (HQ * 4 + HV * 10))
+            del caches, att
+        # gated delta rule
+        HD = HE * 128
+        Cc, ldp = 3 * HD, 3 * HD + HE + 4
+        conv, low, w2 = buf(Cc * 16, "f32"), buf(T * 2 * low_rank * 4, "f32"), buf(HD * low_rank * 4, "f32")
+        u, dec, gate, o = buf(T * Cc * 4, "f32"), buf(T * HD * 4, "f32"), buf(T * HD * 4, "f32"), buf(T * HD * 4)
+        states = [(buf(16 * lib.greta_cuda_gated_delta_state_bytes(HE, 128, 128)), buf(16 * 4 * Cc * 4)) for _ in range(max(2, int(2e8 // (16 * HE * 128 * 128 * 4))))]
+        ds = [g.GatedDelta(HE, HE, 128, 128, 4, low_rank, low_rank, 1e-6, proj.ptr, ldp, conv.ptr, h.ptr, proj.ptr + 4 * Cc, ldp, ln.ptr, st.ptr, low.ptr, 2 * low_rank, low_rank,
+                           w2.ptr, w2.ptr, w2.ptr, w2.ptr, u.ptr, Cc, dec.ptr, gate.ptr, HD, HD) for st, h in states]
+        for b in (1, 16):
+            dpos = g.DeviceBuffer.from_numpy(np.full(b, HYBRID_CONTEXT, np.uint32))
+            rows = g.Rows(b, 0, 0, dpos.ptr)
+            report(f"gated_delta_step M={b}", size, lambda i: g.check(lib.greta_cuda_gated_delta_step(stream, C.byref(ds[i]), C.byref(rows), cat.ptr, 0, HD)), len(ds),
+                   hbm=b * HE * 128 * 128 * 8 + 2 * HD * low_rank * 4)
+        many = g.Rows(T, 0, 0, None)
+        report("gated_delta_prepare T=2048", size, lambda i: g.check(lib.greta_cuda_gated_delta_prepare(stream, C.byref(ds[i]), C.byref(many))), len(ds), hbm=T * Cc * 8)
+        report("gated_delta_scan T=2048", size, lambda i: g.check(lib.greta_cuda_gated_delta_scan(stream, C.byref(ds[i]), C.byref(many), o.ptr)), 2, hbm=T * HD * 4 * 5,
+               fp32=2.0 * T * HE * 128 * 128 * 4)
+        report("gated_delta_output T=2048", size, lambda i: g.check(lib.greta_cuda_gated_delta_output(stream, C.byref(ds[i]), o.ptr, T, cat.ptr, g.OUT_BF16, HD)), 2,
+               hbm=T * HD * (4 + 4 + 2))
+        xs = [buf(T * D * 4, "f32") for _ in range(8)]
+        report("rms_norm T=2048", size, lambda i: g.check(lib.greta_cuda_rms_norm(stream, xs[i].ptr, D, ln.ptr, 1e-6, cat.ptr, g.OUT_BF16, T, D, D)), 8, hbm=T * D * 6)
+        del states, ds, xs
 
 
 def run_case(pkg, name):
@@ -838,7 +973,8 @@ def main():
                     help="tensor-parallel exchange of the decode step: fused into the GEMV kernels over peer memory, or NCCL all-reduce")
     ap.add_argument("--case", default=None, help="run a small single-kernel case (gemv_swiglu, gemv_plain, gemm_c2, gemm_small, attn_decode, decode_step, gemv_batch, attn_batch) and exit; "
                          "gemv_shapes prints the GEMV bandwidth of every projection shape; hybrid_models and hybrid_kernels (or "
-                         "hybrid_kernels:<part of a name>) measure the hybrid design beside the Llama-shaped model")
+                         "hybrid_kernels:<part of a name>) measure the hybrid design beside the Llama-shaped model; latent_models and "
+                         "latent_kernels the latent attention / gated delta design beside the hybrid one")
     args = ap.parse_args()
     pkg = load_pkg()
     ranks = pkg.rendezvous.Ranks()
@@ -860,6 +996,14 @@ def main():
     if args.case and args.case.startswith("hybrid_kernels"):
         pkg.ffi.require_device()
         hybrid_kernels(pkg, args.case.partition(":")[2] or None)
+        return
+    if args.case == "latent_models":
+        pkg.ffi.require_device()
+        latent_models(pkg)
+        return
+    if args.case and args.case.startswith("latent_kernels"):
+        pkg.ffi.require_device()
+        latent_kernels(pkg, args.case.partition(":")[2] or None)
         return
     if args.case:
         run_case(pkg, args.case)

@@ -508,7 +508,7 @@ struct GatedArgs {
   greta_gated_delta d;
   greta_rows rows;
 };
-__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + expf(-z)); }
 // Projected channel c of sequence `slot` at position p - back: from the launch's rows (m is the row of position p, rows of this
 // sequence start at position first) or from the history; zero in front of the sequence.
 __device__ __forceinline__ float channel_at(const greta_gated_delta &d, uint32_t C, uint32_t slot, uint32_t m, uint32_t p, uint32_t first, uint32_t back,
@@ -544,30 +544,53 @@ __global__ void __launch_bounds__(256) gated_prepare_kernel(const __grid_constan
         cw[i][j] = on ? d.conv[(size_t)(c0 + 32 * i) * W + j] : 0.f;
         win[i][j] = on && j < W - 1 ? channel_at(d, C, slot, m0, a.rows.pos0 + m0, a.rows.pos0, W - 1 - j, c0 + 32 * i) : 0.f;
       }
-  for (uint32_t m = m0; m < m1; ++m) {
-    float v[CH], q = 0.f;
+  constexpr int RG = 4;  // rows of a group; the next group's loads are in flight while one is computed
+  float cur[RG][CH];
+  auto load = [&](uint32_t m) {
 #pragma unroll
-    for (int i = 0; i < CH; ++i) {
-      const bool on = lane + 32 * i < (int)n;
-      float y = 0.f;
-      if (TAPS) {
-        win[i][W - 1] = on ? d.proj[(size_t)m * d.ld_proj + c0 + 32 * i] : 0.f;
+    for (int r = 0; r < RG; ++r)
 #pragma unroll
-        for (int j = 0; j < W; ++j) y = fmaf(cw[i][j], win[i][j], y);
+      for (int i = 0; i < CH; ++i) cur[r][i] = m + r < m1 && lane + 32 * i < (int)n ? d.proj[(size_t)(m + r) * d.ld_proj + c0 + 32 * i] : 0.f;
+  };
+  if (TAPS) load(m0);
+  for (uint32_t m = m0; m < m1; m += RG) {
+    float v[RG][CH], q[RG];
 #pragma unroll
-        for (int j = 0; j + 1 < W; ++j) win[i][j] = win[i][j + 1];
-      } else if (on) {
-        for (uint32_t j = 0; j < d.taps; ++j)
-          y = fmaf(d.conv[(size_t)(c0 + 32 * i) * d.taps + j], channel_at(d, C, slot, m, a.rows.pos0 + m, a.rows.pos0, d.taps - 1 - j, c0 + 32 * i), y);
+    for (int r = 0; r < RG; ++r) {
+      q[r] = 0.f;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        float y = 0.f;
+        if (TAPS) {
+          win[i][W - 1] = cur[r][i];
+#pragma unroll
+          for (int j = 0; j < W; ++j) y = fmaf(cw[i][j], win[i][j], y);
+#pragma unroll
+          for (int j = 0; j + 1 < W; ++j) win[i][j] = win[i][j + 1];
+        } else if (m + r < m1 && lane + 32 * i < (int)n) {
+          for (uint32_t j = 0; j < d.taps; ++j)
+            y = fmaf(d.conv[(size_t)(c0 + 32 * i) * d.taps + j], channel_at(d, C, slot, m + r, a.rows.pos0 + m + r, a.rows.pos0, d.taps - 1 - j, c0 + 32 * i), y);
+        }
+        v[r][i] = y;
       }
-      v[i] = on ? silu(y) : 0.f;
-      q = fmaf(v[i], v[i], q);
     }
-    float inv = 1.f;
-    if (!is_v) inv = after / sqrtf(warp_sum(q) + 1e-6f);
+    if (TAPS) load(m + RG);
 #pragma unroll
-    for (int i = 0; i < CH; ++i)
-      if (lane + 32 * i < (int)n) d.u[(size_t)m * d.ld_u + c0 + 32 * i] = v[i] * inv;
+    for (int r = 0; r < RG; ++r)
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        v[r][i] = lane + 32 * i < (int)n ? silu(v[r][i]) : 0.f;
+        q[r] = fmaf(v[r][i], v[r][i], q[r]);
+      }
+    if (!is_v) {
+#pragma unroll
+      for (int r = 0; r < RG; ++r) q[r] = after / sqrtf(warp_sum(q[r]) + 1e-6f);
+    }
+#pragma unroll
+    for (int r = 0; r < RG; ++r)
+#pragma unroll
+      for (int i = 0; i < CH; ++i)
+        if (m + r < m1 && lane + 32 * i < (int)n) d.u[(size_t)(m + r) * d.ld_u + c0 + 32 * i] = is_v ? v[r][i] : v[r][i] * q[r];
   }
 }
 __global__ void gated_history_kernel(const __grid_constant__ GatedArgs a) {

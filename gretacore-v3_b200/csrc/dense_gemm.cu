@@ -23,6 +23,7 @@ using namespace greta;
 
 namespace greta {
 int check_linear(const char *what, const greta_linear *l, Segments *sg);
+cudaError_t latent_wait_status(int *code);
 }
 
 namespace {
@@ -464,6 +465,7 @@ int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *l, const v
 int greta_cuda_linear_gemm_status(int *code) {
   GRETA_REQUIRE(code, "linear_gemm_status: null out pointer");
   GRETA_CUDA_TRY(cudaMemcpyFromSymbol(code, g_gemm_error, sizeof(int)));
+  if (*code == 0) GRETA_CUDA_TRY(latent_wait_status(code));
   return GRETA_OK;
 }
 

@@ -339,7 +339,7 @@ bool BlockScheduler::allocate_hybrid_activations(std::string *err) {
     return true;
   };
   uint32_t proj = 4, cat = 64, q = 4, o = 4, low = 0, low16 = 0, hd = 0, q_latent = 0, u = 0, gate = 0;
-  size_t scratch = 0, kx = 0, vx = 0;
+  size_t scratch = 0, qx = 0, kx = 0, vx = 0;
   const uint32_t absorbed = bf16 ? std::max(B, std::min(chunk, MMA_MIN_ROWS - 1)) : R;  // rows that latent attention takes in its absorbed form
   for (uint32_t l = 0; l < c.num_layers; ++l) {
     const MixerSpec &m = c.layers[l].mixer;
@@ -368,6 +368,7 @@ bool BlockScheduler::allocate_hybrid_activations(std::string *err) {
         a.heads = m.heads, a.rank = m.kv_rank, a.rot_dim = m.rot_dim, a.fmt = bf16 ? GRETA_FMT_F16 : GRETA_FMT_F32;
         scratch = std::max(scratch, greta_cuda_latent_scratch_bytes(&a, absorbed, (uint32_t)max_seq_));
         if (bf16 && chunk >= MMA_MIN_ROWS) {
+          qx = std::max(qx, (size_t)R * greta_cuda_latent_query_row(m.heads, m.dim, m.rot_dim) * 2);
           kx = std::max(kx, max_seq_ * m.heads * up(m.dim, 8) * 2);
           vx = std::max(vx, max_seq_ * m.heads * up(m.vdim, 8) * 2);
         }
@@ -397,7 +398,7 @@ bool BlockScheduler::allocate_hybrid_activations(std::string *err) {
               !zeroed(w.decay, (size_t)R * w.decay_ld * 4) || !zeroed(w.o, (size_t)R * o * 4)))
     return false;
   if ((u && (!zeroed(w.u, (size_t)R * u * 4) || !zeroed(w.gate, (size_t)R * gate * 4))) || (q_latent && !zeroed(w.q_latent, (size_t)R * q_latent * cb)) ||
-      (scratch && !zeroed(w.latent_scratch, scratch)) || (kx && (!zeroed(w.k_expanded, kx, GretaDataType::FP16) || !zeroed(w.v_expanded, vx, GretaDataType::FP16))))
+      (scratch && !zeroed(w.latent_scratch, scratch)) || (kx && (!zeroed(w.q_tiles, qx, GretaDataType::FP16) || !zeroed(w.k_expanded, kx, GretaDataType::FP16) || !zeroed(w.v_expanded, vx, GretaDataType::FP16))))
     return false;
   rotation_tables_ = std::vector<Buffer>(rotations_.size());
   for (size_t r = 0; r < rotations_.size(); ++r) {  // angles in double: the tables are as exact as their fp32 entries
@@ -725,14 +726,14 @@ bool BlockScheduler::latent_attention_core(size_t layer, const greta_rows &rows,
     return true;
   }
   // keys and values of every head for all positions so far, then attention over them
-  GRETA_TRY(greta_cuda_latent_cache(s, &a, &rows), "attention inputs");
+  GRETA_TRY(greta_cuda_latent_prepare(s, &a, &rows, w.q_tiles.data()), "attention inputs");
   const uint32_t Hd = m.heads * up(m.dim, 8), Hv = m.heads * up(m.vdim, 8), ld = greta_cuda_latent_row(m.kv_rank, m.rot_dim);
   greta_linear kv = linear(GRETA_FMT_F16, b.w_kv, Hd + Hv, m.kv_rank, b.kv_ld);
   segment(kv, Hd, GRETA_ACT_NONE, nullptr, w.k_expanded.data(), Hd, 0, GRETA_OUT_F16);
   segment(kv, Hv, GRETA_ACT_NONE, nullptr, w.v_expanded.data(), Hv, 0, GRETA_OUT_F16);
   const uint16_t *latents = static_cast<const uint16_t *>(b.k_cache.data()) + (size_t)rows.slot0 * a.cap * ld;
   GRETA_TRY(greta_cuda_linear_gemm(s, &kv, latents, ld, rows.pos0 + rows.M), "keys and values");
-  GRETA_TRY(greta_cuda_latent_prefill(s, &a, &rows, w.k_expanded.data(), w.v_expanded.data(), cat, cat_fmt, w.cat_ld), "attention");
+  GRETA_TRY(greta_cuda_latent_prefill(s, &a, &rows, w.q_tiles.data(), w.k_expanded.data(), w.v_expanded.data(), cat, cat_fmt, w.cat_ld), "attention");
   return true;
 }
 

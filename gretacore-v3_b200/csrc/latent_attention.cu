@@ -1,6 +1,7 @@
 // Latent attention: every head's keys and values are linear images of one cached latent per token, plus one rotated key part
 // that all heads share.
-//   latent_cache_kernel     norm of the latent, rotation of the shared key part, cache row
+//   latent_prepare_kernel   portions: norm of the latent, rotation of the shared key part, cache row; for the expanded form also the
+//                           rotated and scaled queries in fp16
 //   absorbed form (decode, short portions; 32-bit models always)
 //     latent_query_kernel   q W_uk per head and the rotated q, so that a score is one dot product with a cache row; the new
 //                           tokens' cache rows are written beside it
@@ -9,13 +10,15 @@
 //     latent_rows_kernel    the same in 32-bit on the CUDA cores
 //     latent_value_kernel   merges the splits (with the sink), applies W_uv per head and the output gate
 //   expanded form (prompts)
-//     latent_prefill_kernel keys and values of all heads lie in a workspace (a dense product of the cached latents); tiles of
-//                           query positions x 64 keys on the tensor cores, the rotated key part read from the cache
+//     latent_prefill_kernel keys and values of all heads lie in a workspace (a dense product of the cached latents), the rotated key
+//                           part is read from the cache; 128 query positions of a head per CTA on tcgen05: scores and outputs in
+//                           TMEM, the softmax weights go back to TMEM as the second product's operand
 // Scores, weights, sums and angles are fp32 throughout.
 #include <algorithm>
 
 #include "dense_device.cuh"
 #include "mma_device.cuh"
+#include "tc_device.cuh"
 
 using namespace greta;
 
@@ -69,12 +72,34 @@ __device__ __forceinline__ void write_cache_row(const greta_latent_attn &a, cons
   for (uint32_t c = lane; c < R16; c += 32) row[c] = to_cache<CT>(c < a.rank ? x[c] * inv * __ldg(a.latent_norm + c) : 0.f);
   for (uint32_t c = lane; c < P16; c += 32) row[R16 + c] = to_cache<CT>(c < a.rot_dim ? rotated(a, x + a.rank, at.pos, c) : 0.f);
 }
+__host__ __device__ constexpr uint32_t slabs(uint32_t cols) { return (cols + 63) / 64; }  // column groups of a 128-byte swizzled tile
+// One CTA per row: the last warp writes the cache row, the others the queries (q_out NULL: none) as [head][dim64 | rot64], in powers of
+// two and zero past the head's channels.
 template <typename CT>
-__global__ void __launch_bounds__(256) latent_cache_kernel(const __grid_constant__ LatArgs w) {
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const __grid_constant__ LatArgs w, __half *__restrict__ q_out) {
   pdl_launch_dependents();
   pdl_wait();
-  const uint32_t m = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (m < w.rows.M) write_cache_row<CT>(w.a, w.rows, m, threadIdx.x & 31);
+  const greta_latent_attn &a = w.a;
+  const uint32_t m = blockIdx.x;
+  if (threadIdx.x >= 224) {
+    write_cache_row<CT>(a, w.rows, m, threadIdx.x & 31);
+    return;
+  }
+  if (!q_out) return;
+  const uint32_t d64 = slabs(a.dim) * 64, width = d64 + slabs(a.rot_dim) * 64, pos = where(w.rows, m).pos;
+  const float scale = a.scale * LOG2E;
+  const float *q = a.q + (size_t)m * a.ld_q;
+  for (uint32_t e = threadIdx.x; e < a.heads * width / 2; e += 224) {
+    const uint32_t h = e / (width / 2), c = (e % (width / 2)) * 2;
+    const float *x = q + (size_t)h * (a.dim + a.rot_dim);
+    float v[2];
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
+      const uint32_t col = c + y;
+      v[y] = col < d64 ? (col < a.dim ? x[col] : 0.f) : (col - d64 < a.rot_dim ? rotated(a, x + a.dim, pos, col - d64) : 0.f);
+    }
+    *reinterpret_cast<uint32_t *>(q_out + (size_t)m * a.heads * width + 2 * (size_t)e) = half2_bits(v[0] * scale, v[1] * scale);
+  }
 }
 
 // Eight consecutive weights as floats.
@@ -519,151 +544,269 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant
   }
 }
 
-// Prompts: blockDim / 32 warps x 16 query positions of one head per CTA, 64 keys per step, two steps in flight.
-// DV: value size bucket (64, 128 or 256).
-constexpr uint32_t LP_K = 64;
-template <int DV>
-__global__ void __launch_bounds__(256) latent_prefill_kernel(const __grid_constant__ LatArgs w, const __half *__restrict__ kx, const __half *__restrict__ vx,
-                                                             void *out, int out_fmt, uint32_t ld_out) {
+// ---- prompts: tcgen05
+__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};" ::"r"(taddr),
+      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]),
+      "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]),
+      "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// D[tmem] (+)= A[tmem, fp16 pairs] * B[smem desc], fp32 accumulate.
+__device__ __forceinline__ void umma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint32_t desc_b_lo, uint32_t desc_hi, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t.reg .b64 db;\n\t"
+      "mov.b64 db, {%2, %3};\n\t"
+      "setp.ne.b32 p, %5, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], db, %4, p;\n\t}" ::"r"(tmem_d),
+      "r"(tmem_a), "r"(desc_b_lo), "r"(desc_hi), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+constexpr uint32_t LP_Q = 128, LP_THREADS = 192, LP_TMEM = 512;
+constexpr uint32_t LP_SLAB_Q = LP_Q * 128;          // bytes of 64 columns of the query tile
+constexpr float LP_LAZY = 8.f;                      // a row's maximum may grow by this factor's exponent before its sums are rescaled
+
+// grid (query tiles, heads).  Warp 0: TMA of the queries, keys (per-head part from the workspace, rotated part from the cache) and
+// values; warp 1: MMA issuer; warps 2-5: softmax (one query row per thread) and outputs.  KT: keys per tile.
+// A key tile's column slabs of 64 may reach into the next head's columns: the queries are zero there; surplus output columns are not read.
+// TMEM columns: scores of even and odd tiles at 0 and 128, each overwritten by its weights (fp16 pairs); outputs from 256 on.
+template <int KT>
+__global__ void __launch_bounds__(LP_THREADS, 1)
+latent_prefill_kernel(const __grid_constant__ LatArgs w, const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ CUtensorMap tmap_v,
+                      void *out, int out_fmt, uint32_t ld_out, uint32_t stages) {
   const greta_latent_attn &a = w.a;
-  extern __shared__ __align__(16) uint8_t smb[];
-  const uint32_t D16 = up16(a.dim), P16 = up16(a.rot_dim), KD = D16 + P16, V16 = up16(a.vdim), KB = KD * 2 + 16, VB = V16 * 2 + 16;
-  const uint32_t nq_max = blockDim.x / 2, threads = blockDim.x;
-  uint8_t *qs = smb, *kt = qs + (size_t)nq_max * KB, *vt = kt + 2 * LP_K * KB;
-  const uint32_t smem = nq_max * KB + 2 * LP_K * (KB + VB);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3, mat = lane >> 3, r8 = lane & 7;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t *smem = reinterpret_cast<uint8_t *>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  constexpr uint32_t SLAB = KT * 128;  // bytes of 64 columns of a key tile
+  const uint32_t sd = slabs(a.dim), sr = slabs(a.rot_dim), sv = slabs(a.vdim), d8 = up8(a.dim), v8 = up8(a.vdim);
+  uint8_t *qs = smem, *ks = qs + (sd + sr) * LP_SLAB_Q, *vs = ks + stages * (sd + sr) * SLAB;
+  uint64_t *bars = reinterpret_cast<uint64_t *>(vs + stages * sv * SLAB);
+  uint64_t *kf = bars, *ke = bars + 2, *vf = bars + 4, *ve = bars + 6, *sf = bars + 8, *pf = bars + 10, *od = bars + 12, *qf = bars + 13;
+  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(bars + 14);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t tile = gridDim.x - 1 - blockIdx.x, h = blockIdx.y;  // the longest rows first
-  const uint32_t m0 = tile * nq_max, nq = min(nq_max, w.rows.M - m0), i0 = w.rows.pos0 + m0, total = i0 + nq;
-  const uint32_t R16 = up16(a.rank), LD = R16 + P16, d8 = up8(a.dim), v8 = up8(a.vdim);
-  for (uint32_t e = threadIdx.x; e < smem / 16; e += threads) reinterpret_cast<uint4 *>(smb)[e] = make_uint4(0, 0, 0, 0);
+  const uint32_t m0 = tile * LP_Q, nq = min(LP_Q, w.rows.M - m0), i0 = w.rows.pos0 + m0, total = i0 + nq, ntiles = (total + KT - 1) / KT;
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&kf[i], 1);
+      mbar_init(&ke[i], 1);
+      mbar_init(&vf[i], 1);
+      mbar_init(&ve[i], 1);
+      mbar_init(&sf[i], 1);
+      mbar_init(&pf[i], 4);
+    }
+    mbar_init(od, 1);
+    mbar_init(qf, 1);
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_q) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_k) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_r) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(&tmap_v) : "memory");
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, LP_TMEM);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
   pdl_launch_dependents();
   pdl_wait();
+
+  if (warp == 0) {
+    if (lane == 0) {
+      uint32_t issued = 0;
+      bool ok = true;
+      mbar_arrive_expect_tx(qf, (sd + sr) * LP_SLAB_Q);
+      for (uint32_t c = 0; c < sd + sr; ++c) tma_load_2d(qs + c * LP_SLAB_Q, &tmap_q, (int)((h * (sd + sr) + c) * 64), (int)m0, qf);
+      for (uint32_t t = 0; t < ntiles && ok; ++t) {
+        const uint32_t st = t % stages, ph = ((t / stages) & 1) ^ 1;
+        ok = mbar_wait(&ke[st], ph, abort_flag, 100 + st);
+        if (!ok) break;
+        uint8_t *kd = ks + st * (sd + sr) * SLAB, *vd = vs + st * sv * SLAB;
+        mbar_arrive_expect_tx(&kf[st], (sd + sr) * SLAB);
+        for (uint32_t c = 0; c < sd; ++c) tma_load_2d(kd + c * SLAB, &tmap_k, (int)(h * d8 + c * 64), (int)(t * KT), &kf[st]);
+        for (uint32_t c = 0; c < sr; ++c) tma_load_2d(kd + (sd + c) * SLAB, &tmap_r, (int)(up16(a.rank) + c * 64), (int)(t * KT), &kf[st]);
+        ok = mbar_wait(&ve[st], ph, abort_flag, 110 + st);
+        issued = t + 1;
+        if (!ok) break;
+        mbar_arrive_expect_tx(&vf[st], sv * SLAB);
+        for (uint32_t c = 0; c < sv; ++c) tma_load_2d(vd + c * SLAB, &tmap_v, (int)(h * v8 + c * 64), (int)(t * KT), &vf[st]);
+      }
+      if (*abort_flag) {  // give copies in flight a bounded chance to land before the CTA leaves
+        const long long q0 = clock64();
+        while (!mbar_try_wait(qf, 0) && clock64() - q0 < 20000000ll) {
+        }
+        for (uint32_t t = issued > stages ? issued - stages : 0; t < issued; ++t) {
+          const long long c0 = clock64();
+          while (!mbar_try_wait(&kf[t % stages], (t / stages) & 1) && clock64() - c0 < 20000000ll) {
+          }
+          while (!mbar_try_wait(&vf[t % stages], (t / stages) & 1) && clock64() - c0 < 40000000ll) {
+          }
+        }
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = instr_desc_f16(LP_Q, KT);
+      const uint32_t idesc_o = instr_desc_f16(LP_Q, up16(a.vdim)) | (1u << 16);  // values: keys are the rows of memory (N-major operand)
+      const uint32_t q_lo = smem_desc_lo(smem_u32(qs)), k_lo = smem_desc_lo(smem_u32(ks));
+      const uint32_t v_lo = ((smem_u32(vs) >> 4) & 0x3FFFu) | ((SLAB >> 4) << 16);  // 64-column groups are a slab apart
+      auto scores = [&](uint32_t t) {
+        const uint32_t st = t % stages;
+        if (!mbar_wait_now(&kf[st], (t / stages) & 1, abort_flag, 200 + st)) return false;
+        tc_fence_after();
+        uint32_t acc = 0;
+        auto part = [&](uint32_t slab0, uint32_t cols) {
+          for (uint32_t k16 = 0; k16 < (cols + 15) / 16; ++k16, acc = 1) {
+            const uint32_t s = slab0 + k16 / 4, in = (k16 & 3) * 2;
+            umma_f16(tmem + (t & 1) * 128, q_lo + s * (LP_SLAB_Q >> 4) + in, k_lo + (st * (sd + sr) + s) * (SLAB >> 4) + in, SMEM_DESC_HI_SW128, idesc_s, acc);
+          }
+        };
+        part(0, a.dim);
+        part(sd, a.rot_dim);
+        umma_commit(&ke[st]);
+        umma_commit(&sf[t & 1]);
+        return true;
+      };
+      bool ok = mbar_wait_now(qf, 0, abort_flag, 210);
+      tc_fence_after();
+      ok = ok && scores(0) && (ntiles < 2 || scores(1));
+      for (uint32_t t = 0; t < ntiles && ok; ++t) {
+        const uint32_t st = t % stages;
+        ok = mbar_wait_now(&pf[t & 1], (t >> 1) & 1, abort_flag, 220 + (t & 1)) && mbar_wait_now(&vf[st], (t / stages) & 1, abort_flag, 230 + st);
+        if (!ok) break;
+        tc_fence_after();
+        for (uint32_t k16 = 0; k16 < KT / 16; ++k16)
+          umma_f16_ts(tmem + 256, tmem + (t & 1) * 128 + k16 * 8, v_lo + st * sv * (SLAB >> 4) + k16 * (2048 >> 4), SMEM_DESC_HI_SW128, idesc_o, (t | k16) ? 1u : 0u);
+        umma_commit(&ve[st]);
+        umma_commit(od);
+        if (t + 2 < ntiles) ok = mbar_wait_now(od, t & 1, abort_flag, 240) && scores(t + 2);  // the weights of tile t are read: its columns are free
+      }
+    }
+  } else {
+    const uint32_t quad = warp & 3, row = quad * 32 + lane, i = i0 + row;
+    if (a.gate && row < nq)  // the gates travel to L2 meanwhile
+      for (uint32_t c = 0; c < a.vdim; c += 32)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(a.gate + (size_t)(m0 + row) * a.ld_gate + (size_t)h * a.vdim + c));
+    const uint32_t lanes = tmem + (quad * 32 << 16), o_cols = up16(a.vdim);
+    float mx = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (uint32_t t = 0; t < ntiles && ok; ++t) {
+      const uint32_t sb = lanes + (t & 1) * 128;
+      ok = mbar_wait_now(&sf[t & 1], (t >> 1) & 1, abort_flag, 300 + (t & 1));
+      if (!ok) break;
+      tc_fence_after();
+      __syncwarp();
+      uint32_t v[KT / 32][32];
+#pragma unroll
+      for (int c = 0; c < KT / 32; ++c) tmem_ld32(sb + c * 32, v[c]);
+      tmem_ld_wait();
+      if (t * KT + KT - 1 > i0) {  // the diagonal (or the end) runs through the tile
+#pragma unroll
+        for (int c = 0; c < KT / 32; ++c)
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            if (t * KT + c * 32 + j > i) v[c][j] = 0xFF800000u;
+      }
+      float tm[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int c = 0; c < KT / 32; ++c)
+#pragma unroll
+        for (int j = 0; j < 32; ++j) tm[j & 3] = fmaxf(tm[j & 3], __uint_as_float(v[c][j]));
+      const float nm = fmaxf(mx, fmaxf(fmaxf(tm[0], tm[1]), fmaxf(tm[2], tm[3])));  // finite from the first tile on: key 0
+      if (t == 0) {
+        mx = nm;
+      } else if (__any_sync(0xffffffffu, nm > mx + LP_LAZY)) {
+        const float f = nm > mx + LP_LAZY ? ex2(mx - nm) : 1.f;
+        if (nm > mx + LP_LAZY) mx = nm;
+        l *= f;
+        ok = mbar_wait_now(od, (t - 1) & 1, abort_flag, 310);  // every product so far is in
+        if (!ok) break;
+        tc_fence_after();
+        __syncwarp();
+        for (uint32_t c = 0; c < o_cols; c += 32) {  // the last columns of a group of 32 may be surplus
+          uint32_t o[32];
+          tmem_ld32(lanes + 256 + c, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * f);
+          tmem_st32(lanes + 256 + c, o);
+        }
+      }
+      float sum[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int c = 0; c < KT / 64; ++c) {
+        uint32_t p[32];
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          const float p0 = ex2(__uint_as_float(v[2 * c + j / 16][(2 * j) & 31]) - mx), p1 = ex2(__uint_as_float(v[2 * c + j / 16][(2 * j + 1) & 31]) - mx);
+          sum[(2 * j) & 3] += p0;
+          sum[(2 * j + 1) & 3] += p1;
+          p[j] = half2_bits(p0, p1);
+        }
+        tmem_st32(sb + c * 32, p);
+      }
+      l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&pf[t & 1]);
+    }
+    // the last two products one after the other: a wait may be one phase behind its barrier, not two
+    ok = ok && (ntiles < 2 || mbar_wait_now(od, (ntiles - 2) & 1, abort_flag, 320)) && mbar_wait_now(od, (ntiles - 1) & 1, abort_flag, 321);
+    if (ok) {
+      tc_fence_after();
+      const float sink2 = a.sink ? a.sink[h] * LOG2E : -INFINITY, nm = fmaxf(mx, sink2), f = ex2(mx - nm), inv = f / (l * f + ex2(sink2 - nm));
+      const size_t m = m0 + row, at = m * ld_out + (size_t)h * a.vdim;
+      const float *gate = a.gate ? a.gate + m * a.ld_gate + (size_t)h * a.vdim : nullptr;
+      const bool vec = a.vdim % 8 == 0 && ld_out % 8 == 0 && ((uintptr_t)out & 15) == 0 && (!gate || (a.ld_gate % 4 == 0 && ((uintptr_t)a.gate & 15) == 0));
+      for (uint32_t c = 0; c < a.vdim; c += 32) {
+        uint32_t o[32];
+        __syncwarp();
+        tmem_ld32(lanes + 256 + c, o);
+        tmem_ld_wait();
+        if (row >= nq) continue;
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) {
+          if (c + j >= a.vdim) break;
+          float y[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[e] = __uint_as_float(o[j + e]) * inv;
+          if (vec) {
+            if (gate) {
+              const float4 g0 = *reinterpret_cast<const float4 *>(gate + c + j), g1 = *reinterpret_cast<const float4 *>(gate + c + j + 4);
+              y[0] *= g0.x, y[1] *= g0.y, y[2] *= g0.z, y[3] *= g0.w, y[4] *= g1.x, y[5] *= g1.y, y[6] *= g1.z, y[7] *= g1.w;
+            }
+            if (out_fmt == GRETA_OUT_BF16) {
+              uint4 u;
+              __nv_bfloat162 b0 = __floats2bfloat162_rn(y[0], y[1]), b1 = __floats2bfloat162_rn(y[2], y[3]);
+              __nv_bfloat162 b2 = __floats2bfloat162_rn(y[4], y[5]), b3 = __floats2bfloat162_rn(y[6], y[7]);
+              u.x = *reinterpret_cast<uint32_t *>(&b0), u.y = *reinterpret_cast<uint32_t *>(&b1);
+              u.z = *reinterpret_cast<uint32_t *>(&b2), u.w = *reinterpret_cast<uint32_t *>(&b3);
+              *reinterpret_cast<uint4 *>(static_cast<__nv_bfloat16 *>(out) + at + c + j) = u;
+              continue;
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (c + j + e < a.vdim) store_out(out, out_fmt, at + c + j + e, gate && !vec ? y[e] * gate[c + j + e] : y[e]);
+        }
+      }
+    }
+  }
+  tc_fence_before();
   __syncthreads();
-  const __half *cache = static_cast<const __half *>(a.cache) + (size_t)w.rows.slot0 * a.cap * LD + R16;
-  const __half *kh = kx + (size_t)h * d8, *vh = vx + (size_t)h * v8;
-  const uint32_t ntiles = (total + LP_K - 1) / LP_K, kc = d8 / 8, rc = P16 / 8, per = kc + rc + v8 / 8;
-  auto stage = [&](uint32_t t, int buf) {
-    if (t < ntiles) {
-      for (uint32_t e = threadIdx.x; e < LP_K * per; e += threads) {
-        const uint32_t r = e / per, c = e % per, key = t * LP_K + r;
-        const bool on = key < total;
-        const size_t j = on ? key : 0;
-        uint8_t *krow = kt + (size_t)(buf * LP_K + r) * KB;
-        if (c < kc)
-          cp16z(krow + c * 16, kh + j * a.heads * d8 + c * 8, on);
-        else if (c < kc + rc)
-          cp16z(krow + (D16 / 8 + c - kc) * 16, cache + j * LD + (c - kc) * 8, on);
-        else
-          cp16z(vt + (size_t)(buf * LP_K + r) * VB + (c - kc - rc) * 16, vh + j * a.heads * v8 + (c - kc - rc) * 8, on);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  stage(0, 0);
-  const float scale = a.scale * LOG2E;
-  for (uint32_t e = threadIdx.x; e < nq * KD; e += threads) {
-    const uint32_t r = e / KD, c = e % KD;
-    const float *x = a.q + (size_t)(m0 + r) * a.ld_q + (size_t)h * (a.dim + a.rot_dim);
-    float v = 0.f;
-    if (c < a.dim) v = x[c];
-    else if (c >= D16 && c - D16 < a.rot_dim) v = rotated(a, x + a.dim, i0 + r, c - D16);
-    *reinterpret_cast<__half *>(qs + (size_t)r * KB + c * 2) = __float2half_rn(v * scale);
-  }
-  const uint32_t qi[2] = {i0 + warp * 16 + gq, i0 + warp * 16 + gq + 8};
-  float o[DV / 8][4], mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-#pragma unroll
-  for (int n = 0; n < DV / 8; ++n)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
-  for (uint32_t t = 0; t < ntiles; ++t) {
-    const int buf = t & 1;
-    stage(t + 1, buf ^ 1);
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    if (t * LP_K <= i0 + warp * 16 + 15) {  // some key of the tile is visible to some row of this warp
-      float s[LP_K / 8][4];
-#pragma unroll
-      for (int n = 0; n < (int)LP_K / 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
-#pragma unroll 2
-      for (uint32_t ks = 0; ks < KD / 16; ++ks) {
-        uint32_t qa[4];
-        ldsm_x4(qa, qs + (size_t)(warp * 16 + (mat & 1) * 8 + r8) * KB + ks * 32 + (mat >> 1) * 16);
-#pragma unroll
-        for (int n = 0; n < (int)LP_K / 16; ++n) {
-          uint32_t kb[4];
-          ldsm_x4(kb, kt + (size_t)(buf * LP_K + n * 16 + (mat >> 1) * 8 + r8) * KB + ks * 32 + (mat & 1) * 16);
-          mma16816(s[2 * n], qa, kb[0], kb[1]);
-          mma16816(s[2 * n + 1], qa, kb[2], kb[3]);
-        }
-      }
-      if (t * LP_K + LP_K - 1 > i0 + warp * 16) {  // the diagonal runs through the tile
-#pragma unroll
-        for (int n = 0; n < (int)LP_K / 8; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; ++e)
-            if (t * LP_K + n * 8 + 2 * tq + (e & 1) > qi[e >> 1]) s[n][e] = -INFINITY;
-      }
-      float f[2], base[2];
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        float tm = -INFINITY;
-#pragma unroll
-        for (int n = 0; n < (int)LP_K / 8; ++n) tm = fmaxf(tm, fmaxf(s[n][2 * r], s[n][2 * r + 1]));
-        tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, 1));
-        tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, 2));
-        const float nm = fmaxf(mx[r], tm);
-        base[r] = nm == -INFINITY ? 0.f : nm;
-        f[r] = ex2(mx[r] - base[r]);
-        mx[r] = nm;
-        l[r] *= f[r];
-      }
-#pragma unroll
-      for (int n = 0; n < (int)LP_K / 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          s[n][e] = ex2(s[n][e] - base[e >> 1]);
-          l[e >> 1] += s[n][e];
-        }
-#pragma unroll
-      for (int n = 0; n < DV / 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) o[n][e] *= f[e >> 1];
-#pragma unroll
-      for (int ks = 0; ks < (int)LP_K / 16; ++ks) {
-        const uint32_t pa[4] = {half2_bits(s[2 * ks][0], s[2 * ks][1]), half2_bits(s[2 * ks][2], s[2 * ks][3]),
-                                half2_bits(s[2 * ks + 1][0], s[2 * ks + 1][1]), half2_bits(s[2 * ks + 1][2], s[2 * ks + 1][3])};
-#pragma unroll
-        for (int n = 0; n < DV / 16; ++n) {
-          if (n * 16 >= (int)V16) break;
-          uint32_t vb[4];
-          ldsm_x4_trans(vb, vt + (size_t)(buf * LP_K + ks * 16 + (mat & 1) * 8 + r8) * VB + n * 32 + (mat >> 1) * 16);
-          mma16816(o[2 * n], pa, vb[0], vb[1]);
-          mma16816(o[2 * n + 1], pa, vb[2], vb[3]);
-        }
-      }
-    }
-    __syncthreads();  // the tile may be overwritten
-  }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  const float sink2 = a.sink ? a.sink[h] * LOG2E : -INFINITY;
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
-    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
-    const float nm = fmaxf(mx[r], sink2), f = ex2(mx[r] - nm), inv = f / (l[r] * f + ex2(sink2 - nm));
-    const uint32_t row = warp * 16 + gq + 8 * r, m = m0 + row;
-    if (row >= nq) continue;
-#pragma unroll
-    for (int n = 0; n < DV / 8; ++n)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const uint32_t c = n * 8 + 2 * tq + e, col = h * a.vdim + c;
-        if (c >= a.vdim) continue;
-        const float y = o[n][2 * r + e] * inv;
-        store_out(out, out_fmt, (size_t)m * ld_out + col, a.gate ? y * a.gate[(size_t)m * a.ld_gate + col] : y);
-      }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, LP_TMEM);
   }
 }
 
@@ -742,22 +885,46 @@ int launch_value(cudaStream_t s, const LatArgs &w, const Parts &parts, uint32_t 
                             parts, splits, out, out_fmt, ld_out));
   return launched("latent_value_kernel");
 }
-template <int DV>
-int launch_prefill(cudaStream_t s, const LatArgs &w, const __half *k, const __half *v, void *out, int out_fmt, uint32_t ld_out) {
-  constexpr size_t LIMIT = 227 * 1024;
-  const uint32_t KB = (up16(w.a.dim) + up16(w.a.rot_dim)) * 2 + 16, VB = up16(w.a.vdim) * 2 + 16;
-  auto bytes = [&](uint32_t warps) { return (size_t)warps * 16 * KB + 2 * LP_K * (KB + VB); };
-  const uint32_t warps = w.rows.M > 64 && bytes(8) <= LIMIT ? 8 : 4;
-  GRETA_REQUIRE(bytes(warps) <= LIMIT, "latent_prefill: head sizes %u + %u / %u need %zu bytes of shared memory", w.a.dim, w.a.rot_dim, w.a.vdim, bytes(warps));
+// 64-column boxes of a row-major fp16 matrix, 128-byte swizzle; columns and rows outside read as zero.
+int make_map(CUtensorMap *map, const void *base, uint32_t cols, uint32_t rows, uint32_t box_rows) {
+  EncodeTiledFn enc = encode_tiled();
+  if (!enc) {
+    set_error("latent_prefill: cuTensorMapEncodeTiled is not available from this driver");
+    return GRETA_ERR_NOT_IMPLEMENTED;
+  }
+  const cuuint64_t dims[2] = {cols, rows}, strides[1] = {(cuuint64_t)cols * 2};
+  const cuuint32_t box[2] = {64, box_rows}, estr[2] = {1, 1};
+  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) {
+    set_error("latent_prefill: cuTensorMapEncodeTiled failed with code %d", (int)r);
+    return GRETA_ERR_INVALID_ARGS;
+  }
+  return GRETA_OK;
+}
+constexpr size_t LP_SMEM_LIMIT = 227 * 1024;
+size_t prefill_smem(const greta_latent_attn &a, uint32_t kt, uint32_t stages) {
+  const uint32_t q = slabs(a.dim) + slabs(a.rot_dim);
+  return (size_t)q * LP_SLAB_Q + (size_t)stages * (q + slabs(a.vdim)) * kt * 128 + 1024 + 256;
+}
+template <int KT>
+int launch_prefill(cudaStream_t s, const LatArgs &w, const void *q, const void *k, const void *v, void *out, int out_fmt, uint32_t ld_out, uint32_t stages) {
+  const greta_latent_attn &a = w.a;
+  const uint32_t total = w.rows.pos0 + w.rows.M, LD = up16(a.rank) + up16(a.rot_dim);
+  CUtensorMap mq, mk, mr, mv;
+  if (int rc = make_map(&mq, q, a.heads * (slabs(a.dim) + slabs(a.rot_dim)) * 64, w.rows.M, LP_Q)) return rc;
+  if (int rc = make_map(&mk, k, a.heads * up8(a.dim), total, KT)) return rc;
+  if (int rc = make_map(&mr, static_cast<const __half *>(a.cache) + (size_t)w.rows.slot0 * a.cap * LD, LD, total, KT)) return rc;
+  if (int rc = make_map(&mv, v, a.heads * up8(a.vdim), total, KT)) return rc;
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-    GRETA_CUDA_TRY(cudaFuncSetAttribute(latent_prefill_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LIMIT));
+    GRETA_CUDA_TRY(cudaFuncSetAttribute(latent_prefill_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LP_SMEM_LIMIT));
     attr_set[dev] = true;
   }
-  GRETA_CUDA_TRY(launch_pdl(latent_prefill_kernel<DV>, dim3((w.rows.M + warps * 16 - 1) / (warps * 16), w.a.heads), dim3(warps * 32), bytes(warps), s, w, k, v,
-                            out, out_fmt, ld_out));
+  GRETA_CUDA_TRY(launch_pdl(latent_prefill_kernel<KT>, dim3((w.rows.M + LP_Q - 1) / LP_Q, a.heads), dim3(LP_THREADS), prefill_smem(a, KT, stages), s, w, mq, mk, mr, mv,
+                            out, out_fmt, ld_out, stages));
   return launched("latent_prefill_kernel");
 }
 size_t q_bytes(const greta_latent_attn &a, uint32_t M) {
@@ -766,19 +933,26 @@ size_t q_bytes(const greta_latent_attn &a, uint32_t M) {
 
 }  // namespace
 
+namespace greta {
+cudaError_t latent_wait_status(int *code) { return cudaMemcpyFromSymbol(code, g_gemm_error, sizeof(int)); }
+}  // namespace greta
+
 extern "C" {
 
 uint32_t greta_cuda_latent_row(uint32_t rank, uint32_t rot_dim) { return up16(rank) + up16(rot_dim); }
 
-int greta_cuda_latent_cache(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows) {
-  if (int rc = check_latent("latent_cache", a, rows)) return rc;
+uint32_t greta_cuda_latent_query_row(uint32_t heads, uint32_t dim, uint32_t rot_dim) { return heads * (slabs(dim) + slabs(rot_dim)) * 64; }
+
+int greta_cuda_latent_prepare(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, void *q_out) {
+  if (int rc = check_latent("latent_prepare", a, rows)) return rc;
+  GRETA_REQUIRE(!q_out || (a->q && aligned16(q_out)), "latent_prepare: no queries, or a misaligned output");
   const LatArgs w{*a, *rows};
-  const dim3 grid((rows->M + 7) / 8);
+  __half *q = static_cast<__half *>(q_out);
   if (a->fmt == GRETA_FMT_F16)
-    GRETA_CUDA_TRY(launch_pdl(latent_cache_kernel<__half>, grid, dim3(256), 0, (cudaStream_t)stream, w));
+    GRETA_CUDA_TRY(launch_pdl(latent_prepare_kernel<__half>, dim3(rows->M), dim3(256), 0, (cudaStream_t)stream, w, q));
   else
-    GRETA_CUDA_TRY(launch_pdl(latent_cache_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, w));
-  return launched("latent_cache_kernel");
+    GRETA_CUDA_TRY(launch_pdl(latent_prepare_kernel<float>, dim3(rows->M), dim3(256), 0, (cudaStream_t)stream, w, q));
+  return launched("latent_prepare_kernel");
 }
 
 size_t greta_cuda_latent_scratch_bytes(const greta_latent_attn *a, uint32_t M, uint32_t max_len) {
@@ -811,17 +985,19 @@ int greta_cuda_latent_absorbed(greta_stream_t stream, const greta_latent_attn *a
   return M == 1 ? launch_value<float, 1>(s, w, parts, S, out, out_fmt, ld_out) : launch_value<float, 4>(s, w, parts, S, out, out_fmt, ld_out);
 }
 
-int greta_cuda_latent_prefill(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, const void *k, const void *v, void *out,
-                              int out_fmt, uint32_t ld_out) {
+int greta_cuda_latent_prefill(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, const void *q, const void *k, const void *v,
+                              void *out, int out_fmt, uint32_t ld_out) {
   if (int rc = check_latent("latent_prefill", a, rows)) return rc;
-  GRETA_REQUIRE(!rows->d_pos && k && v && aligned16(k) && aligned16(v) && out && a->q && a->heads <= 65535, "latent_prefill: null pointer, or rows of a batch");
+  GRETA_REQUIRE(!rows->d_pos && q && k && v && aligned16(q) && aligned16(k) && aligned16(v) && out && a->heads <= 65535, "latent_prefill: null pointer, or rows of a batch");
   GRETA_REQUIRE(a->fmt == GRETA_FMT_F16, "latent_prefill: the cache must be F16");
   const LatArgs w{*a, *rows};
   cudaStream_t s = (cudaStream_t)stream;
-  const __half *kh = static_cast<const __half *>(k), *vh = static_cast<const __half *>(v);
-  if (a->vdim <= 64) return launch_prefill<64>(s, w, kh, vh, out, out_fmt, ld_out);
-  if (a->vdim <= 128) return launch_prefill<128>(s, w, kh, vh, out, out_fmt, ld_out);
-  return launch_prefill<256>(s, w, kh, vh, out, out_fmt, ld_out);
+  for (uint32_t stages = 2; stages >= 1; --stages) {  // wide heads: shorter key tiles, then a single stage
+    if (prefill_smem(*a, 128, stages) <= LP_SMEM_LIMIT) return launch_prefill<128>(s, w, q, k, v, out, out_fmt, ld_out, stages);
+    if (prefill_smem(*a, 64, stages) <= LP_SMEM_LIMIT) return launch_prefill<64>(s, w, q, k, v, out, out_fmt, ld_out, stages);
+  }
+  set_error("latent_prefill: head sizes %u + %u / %u do not fit shared memory", a->dim, a->rot_dim, a->vdim);
+  return GRETA_ERR_INVALID_ARGS;
 }
 
 }  // extern "C"

@@ -48,17 +48,28 @@ __device__ __forceinline__ bool mbar_try_wait(uint64_t *bar, uint32_t parity) {
 // Bounded wait.  Returns false when the kernel is aborting (this wait timed out, or another role's did).
 // The common case, a barrier that has already completed, is one try_wait; the polling loop with its
 // clock reads is kept out of line so the issuing threads' instruction streams stay short.
+template <bool NAP>
 __device__ __noinline__ bool mbar_wait_slow(uint32_t bar, uint32_t parity, volatile int *abort_flag, int code) {
   const long long t0 = clock64();
   for (;;) {
     uint32_t ok;
-    asm volatile(  // with a time hint the thread sleeps in hardware until the phase completes instead of spinning through issue slots
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2, %3;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(ok)
-        : "r"(bar), "r"(parity), "r"(1000u)
-        : "memory");
+    if (NAP) {
+      asm volatile(  // with a time hint the thread sleeps in hardware instead of spinning through issue slots, at the price of a late waking
+          "{\n\t.reg .pred p;\n\t"
+          "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2, %3;\n\t"
+          "selp.u32 %0, 1, 0, p;\n\t}"
+          : "=r"(ok)
+          : "r"(bar), "r"(parity), "r"(1000u)
+          : "memory");
+    } else {
+      asm volatile(
+          "{\n\t.reg .pred p;\n\t"
+          "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+          "selp.u32 %0, 1, 0, p;\n\t}"
+          : "=r"(ok)
+          : "r"(bar), "r"(parity)
+          : "memory");
+    }
     if (ok) return true;
     if (*abort_flag) return false;
     if (clock64() - t0 > WAIT_LIMIT_CYCLES) {
@@ -70,7 +81,11 @@ __device__ __noinline__ bool mbar_wait_slow(uint32_t bar, uint32_t parity, volat
 }
 __device__ __forceinline__ bool mbar_wait(uint64_t *bar, uint32_t parity, volatile int *abort_flag, int code) {
   if (mbar_try_wait(bar, parity)) return true;
-  return mbar_wait_slow(smem_u32(bar), parity, abort_flag, code);
+  return mbar_wait_slow<true>(smem_u32(bar), parity, abort_flag, code);
+}
+// The same for waits on a kernel's critical path: polls without sleeping.
+__device__ __forceinline__ bool mbar_wait_now(uint64_t *bar, uint32_t parity, volatile int *abort_flag, int code) {
+  return mbar_wait_slow<false>(smem_u32(bar), parity, abort_flag, code);
 }
 __device__ __forceinline__ void tma_load_2d(void *smem_dst, const CUtensorMap *map, int x, int y, uint64_t *bar) {
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(

@@ -687,7 +687,7 @@ private:
   struct HybridActivations {
     gcore::rt::cuda::Buffer h, proj, cat, cat16, q, low, low16, decay, o, x_rows, logits_rows;
     uint32_t h_ld = 0, proj_ld = 0, cat_ld = 0, low_ld = 0, low16_ld = 0, decay_ld = 0;
-    gcore::rt::cuda::Buffer q_latent, latent_scratch, k_expanded, v_expanded, u, gate;  // latent attention; gated delta
+    gcore::rt::cuda::Buffer q_latent, latent_scratch, q_tiles, k_expanded, v_expanded, u, gate;  // latent attention; gated delta
     uint32_t q_latent_ld = 0, u_ld = 0, gate_ld = 0;
   } hact_;
   std::vector<RotarySpec> rotations_;                    // distinct rotations of the model and their tables

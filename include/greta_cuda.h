@@ -465,7 +465,7 @@ GRETA_API int greta_cuda_linear_gemv(greta_stream_t stream, const greta_linear *
 /* Many rows.  BF16 / F16: tensor cores (tcgen05), x is of the weights' type, [M][ldx], ldx a multiple of 8; columns past K are
  * not read.  F32: true 32-bit products on the CUDA cores, x is fp32 [M][ldx], ldx >= ldw, zero-padded. */
 GRETA_API int greta_cuda_linear_gemm(greta_stream_t stream, const greta_linear *lin, const void *x, uint32_t ldx, uint32_t M);
-/* greta_cuda_gemm_status for the kernels of greta_cuda_linear_gemm. */
+/* greta_cuda_gemm_status for the kernels of greta_cuda_linear_gemm and greta_cuda_latent_prefill. */
 GRETA_API int greta_cuda_linear_gemm_status(int *code);
 /* y = (x - mean) / sqrt(var + eps) * w + b per row of D values; out fp32, fp16 or bf16 (GRETA_OUT_*), row stride ld_out. */
 GRETA_API int greta_cuda_layer_norm(greta_stream_t stream, const float *x, const float *w, const float *b, float eps, void *out, int out_fmt,
@@ -552,18 +552,20 @@ typedef struct greta_latent_attn {
   void *cache;
 } greta_latent_attn;
 GRETA_API uint32_t greta_cuda_latent_row(uint32_t rank, uint32_t rot_dim); /* elements of a cache row */
-/* Norm, rotation and cache write of a portion's rows. */
-GRETA_API int greta_cuda_latent_cache(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows);
+/* A portion's rows: norm, rotation and cache write; and, unless q_out is NULL, the queries as the expanded form takes them, fp16
+ * [M][greta_cuda_latent_query_row]: rotated, scaled, each head's two parts padded to multiples of 64. */
+GRETA_API uint32_t greta_cuda_latent_query_row(uint32_t heads, uint32_t dim, uint32_t rot_dim);
+GRETA_API int greta_cuda_latent_prepare(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, void *q_out);
 /* Absorbed form (decode and short portions): q_h W_uk,h meets the cached latents themselves, W_uv,h is applied to the weighted sum of
  * latents.  Writes the rows' cache entries as well.  scratch: greta_cuda_latent_scratch_bytes for at least these rows;
  * max_len bounds the position of any row plus one. */
 GRETA_API size_t greta_cuda_latent_scratch_bytes(const greta_latent_attn *a, uint32_t M, uint32_t max_len);
 GRETA_API int greta_cuda_latent_absorbed(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, void *scratch, void *out,
                                          int out_fmt, uint32_t ld_out, uint32_t max_len);
-/* Expanded form (prompts; F16): k [pos0 + M][heads * dim8] and v [pos0 + M][heads * vdim8] in fp16 are the products of the cached
- * latents with w_kv (greta_cuda_linear_gemm).  The rows' cache entries must be there. */
-GRETA_API int greta_cuda_latent_prefill(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, const void *k, const void *v,
-                                        void *out, int out_fmt, uint32_t ld_out);
+/* Expanded form (prompts; F16): q from greta_cuda_latent_prepare; k [pos0 + M][heads * dim8] and v [pos0 + M][heads * vdim8] in fp16
+ * are the products of the cached latents with w_kv (greta_cuda_linear_gemm), the rows' own included. */
+GRETA_API int greta_cuda_latent_prefill(greta_stream_t stream, const greta_latent_attn *a, const greta_rows *rows, const void *q, const void *k,
+                                        const void *v, void *out, int out_fmt, uint32_t ld_out);
 
 /* ------------------------------------------------------------------ generalised delta rule
  * Per head, key dimension = value dimension = dim, state S [dim x dim] in fp32, zero in front of position 0:

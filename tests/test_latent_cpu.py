@@ -81,23 +81,23 @@ def test_argument_checks_of_the_operators(pkg):
     p = (C.addressof(buf) + 15) // 16 * 16
     rows = f.Rows(4, 0, 0, None)
     a = f.LatentAttn(4, 16, 8, 16, 32, 8, 0, 10, 10, 0.3, 1e-6, p, None, p, p, 96, p, 40, None, 0, f.FMT_F16, p, 64, p)
-    assert lib.greta_cuda_latent_cache(None, C.byref(a), C.byref(f.Rows(4, 0, 7, None))) == 4                  # positions past the cache
+    assert lib.greta_cuda_latent_prepare(None, C.byref(a), C.byref(f.Rows(4, 0, 7, None)), p) == 4                  # positions past the cache
     for change in (dict(dim=257), dict(vdim=0), dict(rank=1025), dict(rot_dim=129), dict(rot_dims=7), dict(rot_dims=10), dict(rotation=None),
                    dict(fmt=f.FMT_BF16), dict(cache=None), dict(cache=p + 4), dict(down=None), dict(latent_norm=None)):
         a2 = f.LatentAttn.from_buffer_copy(a)
         for k, v in change.items():
             setattr(a2, k, v)
-        assert lib.greta_cuda_latent_cache(None, C.byref(a2), C.byref(rows)) == 4, change
+        assert lib.greta_cuda_latent_prepare(None, C.byref(a2), C.byref(rows), p) == 4, change
         assert lib.greta_cuda_latent_absorbed(None, C.byref(a2), C.byref(rows), p, p, 0, 64, 10) == 4, change
-        assert lib.greta_cuda_latent_prefill(None, C.byref(a2), C.byref(rows), p, p, p, 0, 64) == 4, change
+        assert lib.greta_cuda_latent_prefill(None, C.byref(a2), C.byref(rows), p, p, p, p, 0, 64) == 4, change
     for change in (dict(ld_w=63), dict(ld_w=0), dict(w_kv=None), dict(q=None)):
         a2 = f.LatentAttn.from_buffer_copy(a)
         for k, v in change.items():
             setattr(a2, k, v)
         assert lib.greta_cuda_latent_absorbed(None, C.byref(a2), C.byref(rows), p, p, 0, 64, 10) == 4, change
     a.fmt = f.FMT_F32
-    assert lib.greta_cuda_latent_prefill(None, C.byref(a), C.byref(rows), p, p, p, 0, 64) == 4
-    assert lib.greta_cuda_latent_row(33, 8) == 48 + 16
+    assert lib.greta_cuda_latent_prefill(None, C.byref(a), C.byref(rows), p, p, p, p, 0, 64) == 4
+    assert lib.greta_cuda_latent_row(33, 8) == 48 + 16 and lib.greta_cuda_latent_query_row(3, 65, 8) == 3 * (128 + 64)
     d = f.GatedDelta(4, 2, 16, 24, 3, 8, 8, 1e-6, p, 200, p, p, p, 4, p, p)
     for change in (dict(kv_heads=3), dict(dim=300), dict(vdim=257), dict(taps=0), dict(history=None), dict(state=None), dict(state=p + 4)):
         d2 = f.GatedDelta.from_buffer_copy(d)

@@ -169,12 +169,13 @@ class Latent:
         k, v = g.DeviceBuffer(n * self.Hd * 2), g.DeviceBuffer(n * self.Hv * 2)
         ld = p["H"] * p["vdim"] + 5
         o = g.DeviceBuffer(M * ld * 4, zero=True)
-        g.check(self.lib.greta_cuda_latent_cache(None, C.byref(self.a), C.byref(rows)), "cache")
+        q = g.DeviceBuffer(M * self.lib.greta_cuda_latent_query_row(p["H"], p["dim"], p["rot"]) * 2)
+        g.check(self.lib.greta_cuda_latent_prepare(None, C.byref(self.a), C.byref(rows), q.ptr), "prepare")
         lin = g.Linear(g.FMT_F16, self.w.ptr, self.kv_rows, p["rank"], self.a.ld_w, 2)
         lin.seg[0] = g.OutSegment(0, self.Hd, 0, g.OUT_F16, 0, None, k.ptr, self.Hd, 0, 0)
         lin.seg[1] = g.OutSegment(self.Hd, self.Hv, 0, g.OUT_F16, 0, None, v.ptr, self.Hv, 0, 0)
         g.check(self.lib.greta_cuda_linear_gemm(None, C.byref(lin), self.bufs[3].ptr + slot * self.cap * self.row * 2, self.row, n), "keys and values")
-        g.check(self.lib.greta_cuda_latent_prefill(None, C.byref(self.a), C.byref(rows), k.ptr, v.ptr, o.ptr, g.OUT_F32, ld), "prefill")
+        g.check(self.lib.greta_cuda_latent_prefill(None, C.byref(self.a), C.byref(rows), q.ptr, k.ptr, v.ptr, o.ptr, g.OUT_F32, ld), "prefill")
         sync(g)
         del d
         return o.download(np.float32, M * ld).reshape(M, ld)[:, :ld - 5]
