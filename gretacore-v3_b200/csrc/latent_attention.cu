@@ -27,7 +27,7 @@ namespace {
 __host__ __device__ constexpr uint32_t up8(uint32_t d) { return (d + 7u) & ~7u; }
 __host__ __device__ constexpr uint32_t up16(uint32_t d) { return (d + 15u) & ~15u; }
 constexpr float LOG2E = 1.4426950408889634f;
-constexpr uint32_t MAX_RANK = 1024, MAX_ROT = 128, MAX_DIM = 256, MAX_SPLITS = 32;
+constexpr uint32_t MAX_RANK = 1024, MAX_ROT = 128, MAX_DIM = 256, MAX_SPLITS = 64;
 
 struct LatArgs {
   greta_latent_attn a;
@@ -486,8 +486,9 @@ constexpr uint32_t LV_ROWS = 32;
 template <typename CT, int MT>
 __global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant__ LatArgs w, Parts parts, uint32_t S, void *out, int out_fmt, uint32_t ld_out) {
   const greta_latent_attn &a = w.a;
-  __shared__ float lat[MT][MAX_RANK];
+  __shared__ __align__(16) float lat[MT][MAX_RANK];
   __shared__ float ws[MT][MAX_SPLITS];
+  __shared__ uint32_t active[MT];
   const uint32_t h = blockIdx.y, m0 = blockIdx.z * MT, R16 = up16(a.rank), j0 = blockIdx.x * LV_ROWS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const CT *wv = static_cast<const CT *>(a.w_kv) + ((size_t)a.heads * up8(a.dim) + (size_t)h * up8(a.vdim)) * a.ld_w;
@@ -496,45 +497,62 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const __grid_constant
       asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(wv + (size_t)j * a.ld_w) + b));
   pdl_launch_dependents();
   pdl_wait();
-  if (warp < MT && m0 + warp < w.rows.M) {  // weight of every split: exp(max - common max) / denominator
-    const float *ml = parts.ml + ((size_t)(m0 + warp) * a.heads + h) * S * 2;
-    const float mine = lane < (int)S ? ml[lane * 2] : -INFINITY, sum = lane < (int)S ? ml[lane * 2 + 1] : 0.f;
-    const bool p2 = sizeof(CT) == 2;
-    const float sink = a.sink ? a.sink[h] * (p2 ? LOG2E : 1.f) : -INFINITY;
-    const float mx = fmaxf(warp_max(mine), sink), f = p2 ? exp2f(mine - mx) : expf(mine - mx);
-    const float den = warp_sum(sum * f) + (a.sink ? (p2 ? exp2f(sink - mx) : expf(sink - mx)) : 0.f);
-    if (lane < (int)S) ws[warp][lane] = f / den;
-  }
-  __syncthreads();
-  for (uint32_t e = threadIdx.x; e < MT * R16; e += 256) {
-    const uint32_t t = e / R16, r = e % R16, m = m0 + t;
-    float x = 0.f;
-    if (m < w.rows.M) {
-      const float *o = parts.o + ((size_t)m * a.heads + h) * S * R16 + r;
-      for (uint32_t s = 0; s < S; ++s)
-        if (ws[t][s] != 0.f) x = fmaf(ws[t][s], o[(size_t)s * R16], x);  // a split without keys has left nothing
+  if (warp < MT) {  // weight of every split: exp(max - common max) / denominator; splits with keys come first
+    uint32_t n = 0;
+    if (m0 + warp < w.rows.M) {
+      const float2 *ml = reinterpret_cast<const float2 *>(parts.ml) + ((size_t)(m0 + warp) * a.heads + h) * S;
+      const float2 none = make_float2(-INFINITY, 0.f), x = lane < (int)S ? ml[lane] : none, y = lane + 32 < (int)S ? ml[lane + 32] : none;
+      const bool p2 = sizeof(CT) == 2;
+      const float sink = a.sink ? a.sink[h] * (p2 ? LOG2E : 1.f) : -INFINITY, mx = fmaxf(warp_max(fmaxf(x.x, y.x)), sink);
+      const float fx = p2 ? exp2f(x.x - mx) : expf(x.x - mx), fy = p2 ? exp2f(y.x - mx) : expf(y.x - mx);
+      const float den = warp_sum(fmaf(x.y, fx, y.y * fy)) + (a.sink ? (p2 ? exp2f(sink - mx) : expf(sink - mx)) : 0.f);
+      ws[warp][lane] = fx / den;
+      ws[warp][lane + 32] = fy / den;
+      n = __popc(__ballot_sync(0xffffffffu, x.y > 0.f)) + __popc(__ballot_sync(0xffffffffu, y.y > 0.f));
     }
-    lat[t][r] = x;
+    if (lane == 0) active[warp] = n;
   }
   __syncthreads();
+  for (uint32_t e = threadIdx.x * 4; e < MT * R16; e += 256 * 4) {
+    const uint32_t t = e / R16, r = e % R16, m = m0 + t, n = active[t];
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float *o = parts.o + ((size_t)m * a.heads + h) * S * R16 + r;
+#pragma unroll 8
+    for (uint32_t s = 0; s < n; ++s) {
+      const float4 v = *reinterpret_cast<const float4 *>(o + (size_t)s * R16);
+      const float f = ws[t][s];
+      x.x = fmaf(f, v.x, x.x), x.y = fmaf(f, v.y, x.y), x.z = fmaf(f, v.z, x.z), x.w = fmaf(f, v.w, x.w);
+    }
+    *reinterpret_cast<float4 *>(&lat[t][r]) = x;
+  }
+  __syncthreads();
+  float acc[4][MT];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int t = 0; t < MT; ++t) acc[i][t] = 0.f;
+  for (uint32_t r = lane * 8; r < R16; r += 256) {
+    float f[4][8];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) weights8(wv + (size_t)min(j0 + warp * 4 + i, a.vdim - 1) * a.ld_w + r, f[i]);
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+      const float4 u = *reinterpret_cast<const float4 *>(&lat[t][r]), v = *reinterpret_cast<const float4 *>(&lat[t][r + 4]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        float y = acc[i][t];
+        y = fmaf(f[i][0], u.x, fmaf(f[i][1], u.y, fmaf(f[i][2], u.z, fmaf(f[i][3], u.w, y))));
+        acc[i][t] = fmaf(f[i][4], v.x, fmaf(f[i][5], v.y, fmaf(f[i][6], v.z, fmaf(f[i][7], v.w, y))));
+      }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const uint32_t j = j0 + warp * 4 + i;
     if (j >= a.vdim) break;
-    float acc[MT];
-#pragma unroll
-    for (int t = 0; t < MT; ++t) acc[t] = 0.f;
-    for (uint32_t r = lane * 8; r < R16; r += 256) {
-      float f[8];
-      weights8(wv + (size_t)j * a.ld_w + r, f);
-#pragma unroll
-      for (int t = 0; t < MT; ++t)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[t] = fmaf(f[e], lat[t][r + e], acc[t]);
-    }
 #pragma unroll
     for (int t = 0; t < MT; ++t) {
-      const float y = warp_sum(acc[t]);
+      const float y = warp_sum(acc[i][t]);
       const uint32_t m = m0 + t;
       if (lane == 0 && m < w.rows.M) {
         const uint32_t c = h * a.vdim + j;
@@ -839,7 +857,9 @@ int launch_mma(cudaStream_t s, const LatArgs &w, const __half *q, const Parts &p
   constexpr size_t LIMIT = 227 * 1024;
   const uint32_t row = (up16(w.a.rank) + up16(w.a.rot_dim)) * 2 + 16;
   auto bytes = [&](int buffers) { return (size_t)16 * HT * (row + LM_K * 2 + 16) + (size_t)buffers * LM_K * row + 8 * 16 * HT * 4; };
-  const int buffers = bytes(2) <= LIMIT ? 2 : 1;
+  // Two tiles in flight, unless two CTAs with one each fit an SM and there are enough of them.
+  const uint64_t ctas = (uint64_t)splits * ((w.a.heads + 16 * HT - 1) / (16 * HT)) * w.rows.M;
+  const int buffers = bytes(2) <= LIMIT && !(ctas > (uint32_t)sm_count() && bytes(1) <= LIMIT / 2) ? 2 : 1;
   static bool attr_set[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
