@@ -141,11 +141,11 @@ struct ScanArgs {
   float *state;
 };
 
-// The recurrence over a portion: grid (heads, column groups).  A CTA keeps 32 columns of one head in the registers of its
+// The recurrence over a portion: grid (heads, column groups).  A CTA keeps COLS columns of one head in the registers of its
 // first warps, NC columns per group of eight lanes, and walks the tokens in chunks of TC = a block per producer warp.
-template <int RB, int NC, bool GATED>
+template <int RB, int NC, int COLS_, bool GATED>
 struct ScanCfg {
-  static constexpr int DP = RB * 32, COLS = 32;
+  static constexpr int DP = RB * 32, COLS = COLS_;
   static constexpr int TC = RB <= 2 ? 32 : RB <= 4 ? 16 : 8, NB = TC / 4;
   static constexpr int NV = GATED ? 3 : 4;                                      // staged vectors of a token: w, k, (a,) r
   static constexpr int RAW_ROW = NV * DP + COLS + (GATED ? 4 : 0), RAW = TC * RAW_ROW;  // then v (and the write strength)
@@ -179,9 +179,9 @@ __device__ __forceinline__ float sum32_of(float (&v)[N], int lane) {
   return v[0];
 }
 
-template <int RB, int NC, bool GATED>
-__global__ void __launch_bounds__(ScanCfg<RB, NC, GATED>::THREADS) delta_scan_kernel(const __grid_constant__ ScanArgs a, float *__restrict__ o_buf, int vec) {
-  using C = ScanCfg<RB, NC, GATED>;
+template <int RB, int NC, int COLS_, bool GATED>
+__global__ void __launch_bounds__(ScanCfg<RB, NC, COLS_, GATED>::THREADS) delta_scan_kernel(const __grid_constant__ ScanArgs a, float *__restrict__ o_buf, int vec) {
+  using C = ScanCfg<RB, NC, COLS_, GATED>;
   constexpr int DP = C::DP, TC = C::TC, COLS = C::COLS, NV = C::NV;
   extern __shared__ __align__(16) float sm[];
   float *derived = sm + 2 * C::RAW, *so = derived + 2 * C::DER;  // so: [2][TC][COLS]
@@ -305,7 +305,7 @@ __global__ void __launch_bounds__(ScanCfg<RB, NC, GATED>::THREADS) delta_scan_ke
     const int x = lane < FIRST ? 0 : (lane - FIRST) % 10, ri = x < 1 ? 0 : x < 3 ? 1 : x < 6 ? 2 : 3;
     if (lane < PAIRS) der[C::SCAL + (lane < FIRST ? lane : (lane < FIRST + 10 ? 16 : 32) + ri * 4 + x - ri * (ri + 1) / 2)] = total;
     const float *v = raw + NV * DP + lane;
-    *reinterpret_cast<float4 *>(der + C::VT + lane * 4) = make_float4(v[0], v[C::RAW_ROW], v[2 * C::RAW_ROW], v[3 * C::RAW_ROW]);
+    if (lane < COLS) *reinterpret_cast<float4 *>(der + C::VT + lane * 4) = make_float4(v[0], v[C::RAW_ROW], v[2 * C::RAW_ROW], v[3 * C::RAW_ROW]);
   };
   auto write_back = [&](uint32_t c) {
     const uint32_t n = min((uint32_t)TC, T - c * TC);
@@ -735,9 +735,9 @@ int check_delta(const char *what, const greta_delta_rule *d, const greta_rows *r
   return GRETA_OK;
 }
 
-template <int RB, int NC, bool GATED>
+template <int RB, int NC, int COLS, bool GATED>
 int launch_scan(cudaStream_t s, const ScanArgs &a, float *o_buf, int vec) {
-  using C = ScanCfg<RB, NC, GATED>;
+  using C = ScanCfg<RB, NC, COLS, GATED>;
   // A grid that fits the SMs asks for more than half of an SM's shared memory: CTAs that become resident while the previous
   // kernel drains would otherwise pair up on the SMs that fall idle first, and the pairs would set the pace.
   constexpr size_t ALONE = 118 * 1024;
@@ -745,27 +745,29 @@ int launch_scan(cudaStream_t s, const ScanArgs &a, float *o_buf, int vec) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-    GRETA_CUDA_TRY(cudaFuncSetAttribute(delta_scan_kernel<RB, NC, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(C::SMEM, ALONE)));
+    GRETA_CUDA_TRY(cudaFuncSetAttribute(delta_scan_kernel<RB, NC, COLS, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(C::SMEM, ALONE)));
     attr_set[dev] = true;
   }
   const dim3 grid(a.heads, (a.vdim + C::COLS - 1) / C::COLS);
   const size_t smem = grid.x * grid.y <= (uint32_t)sm_count() ? std::max(C::SMEM, ALONE) : C::SMEM;
-  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC, GATED>, grid, dim3(C::THREADS), smem, s, a, o_buf, vec));
+  GRETA_CUDA_TRY(launch_pdl(delta_scan_kernel<RB, NC, COLS, GATED>, grid, dim3(C::THREADS), smem, s, a, o_buf, vec));
   return launched("delta_scan_kernel");
 }
 template <bool GATED>
 int pick_scan(cudaStream_t s, const ScanArgs &a, float *o_buf) {
   const int vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld_w % 4 == 0 && a.ld_k % 4 == 0 && a.ld_r % 4 == 0 && a.ld_v % 4 == 0 && aligned16(a.w) &&
                   aligned16(a.k) && aligned16(a.r) && aligned16(a.v) && (GATED || (a.ld_a % 4 == 0 && aligned16(a.a)));
+  // Few heads: half the columns per CTA where the doubled grid still has an SM for every CTA (the usual head sizes).
+  const bool narrow = a.heads * ((a.vdim + 15) / 16) <= (uint32_t)sm_count();
   switch (dim32(a.dim) / 32) {
-    case 1: return launch_scan<1, 2, GATED>(s, a, o_buf, vec);
-    case 2: return launch_scan<2, 2, GATED>(s, a, o_buf, vec);
-    case 3: return launch_scan<3, 2, GATED>(s, a, o_buf, vec);
-    case 4: return launch_scan<4, 2, GATED>(s, a, o_buf, vec);
-    case 5: return launch_scan<5, 1, GATED>(s, a, o_buf, vec);
-    case 6: return launch_scan<6, 1, GATED>(s, a, o_buf, vec);
-    case 7: return launch_scan<7, 1, GATED>(s, a, o_buf, vec);
-    default: return launch_scan<8, 1, GATED>(s, a, o_buf, vec);
+    case 1: return launch_scan<1, 2, 32, GATED>(s, a, o_buf, vec);
+    case 2: return narrow ? launch_scan<2, 1, 16, GATED>(s, a, o_buf, vec) : launch_scan<2, 2, 32, GATED>(s, a, o_buf, vec);
+    case 3: return launch_scan<3, 2, 32, GATED>(s, a, o_buf, vec);
+    case 4: return narrow ? launch_scan<4, 1, 16, GATED>(s, a, o_buf, vec) : launch_scan<4, 2, 32, GATED>(s, a, o_buf, vec);
+    case 5: return launch_scan<5, 1, 32, GATED>(s, a, o_buf, vec);
+    case 6: return launch_scan<6, 1, 32, GATED>(s, a, o_buf, vec);
+    case 7: return launch_scan<7, 1, 32, GATED>(s, a, o_buf, vec);
+    default: return launch_scan<8, 1, 32, GATED>(s, a, o_buf, vec);
   }
 }
 int launch_output(cudaStream_t s, const OutArgs &a, const float *o_buf, void *out, int out_fmt, uint32_t ld_out) {
