@@ -41,15 +41,19 @@ __device__ __forceinline__ void store_out(void *out, int fmt, size_t idx, float 
     if (fmt == GRETA_OUT_BF16_PAIR) static_cast<__nv_bfloat16 *>(out)[idx + pair_offset] = __float2bfloat16_rn(v - __bfloat162float(hi));
   }
 }
-__device__ __forceinline__ void store_segment(const greta_out_segment &g, uint32_t row, uint32_t m, float z) {
+// old: what is there already, for segments that accumulate.
+__device__ __forceinline__ void store_segment(const greta_out_segment &g, uint32_t row, uint32_t m, float z, float old) {
   const uint32_t r = row - g.row0;
   if (g.bias) z += __ldg(g.bias + r);
   z = apply_act(g.act, z, g.rate ? __ldg(g.rate + r) : 0.f);
   const size_t idx = (size_t)m * g.ld + g.col0 + r;
   if (g.accumulate)
-    static_cast<float *>(g.out)[idx] += z;
+    static_cast<float *>(g.out)[idx] = old + z;
   else
     store_out(g.out, g.out_fmt, idx, z, g.pair_offset);
+}
+__device__ __forceinline__ void store_segment(const greta_out_segment &g, uint32_t row, uint32_t m, float z) {
+  store_segment(g, row, m, z, g.accumulate ? static_cast<float *>(g.out)[(size_t)m * g.ld + g.col0 + row - g.row0] : 0.f);
 }
 
 __device__ __forceinline__ float block_sum_all(float v, float *sm) {  // every thread receives the total; sm: 32 floats

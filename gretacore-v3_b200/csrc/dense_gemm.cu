@@ -39,11 +39,36 @@ struct DCfg {
   static_assert(COLS <= 512 && SMEM <= 232448, "tile configuration");
 };
 
-// 32 consecutive tokens (from m on, cnt of them present) of one weight row: bias, activation, store.
+// 32 consecutive tokens (from m on, cnt of them present) of one weight row per lane: bias, activation, store.  All lanes call; those
+// past the last row are off.  PAIRED (16-bit outputs): neighbouring lanes hold neighbouring columns of one segment and exchange every
+// other token, so that each stores two columns at a time.
 template <int ACT>
-__device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
+__device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32], bool on,
+                                               bool paired) {
   const size_t base = (size_t)m * g.ld + g.col0 + r;
-  const float rate = ACT == GRETA_ACT_SOFTPLUS_DECAY ? __ldg(g.rate + r) : 0.f;
+  const float rate = ACT == GRETA_ACT_SOFTPLUS_DECAY && on ? __ldg(g.rate + r) : 0.f;
+  if (paired) {
+    const uint32_t odd = threadIdx.x & 1;
+    uint32_t *o = reinterpret_cast<uint32_t *>(static_cast<uint16_t *>(g.out) + base + (size_t)odd * g.ld - odd);
+    const bool half = g.out_fmt == GRETA_OUT_F16;
+#pragma unroll
+    for (int j = 0; j < 32; j += 2) {
+      const float x = apply_act(ACT, __uint_as_float(v[j]) + bias, rate), y = apply_act(ACT, __uint_as_float(v[j + 1]) + bias, rate);
+      const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
+      const float lo = odd ? other : x, hi = odd ? y : other;
+      uint32_t bits;
+      if (half) {
+        const __half2 h = __floats2half2_rn(lo, hi);
+        bits = *reinterpret_cast<const uint32_t *>(&h);
+      } else {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+        bits = *reinterpret_cast<const uint32_t *>(&h);
+      }
+      if (j + odd < cnt) o[(size_t)(j / 2) * g.ld] = bits;
+    }
+    return;
+  }
+  if (!on) return;
   if (g.accumulate) {
     float *o = static_cast<float *>(g.out) + base;
     float old[32];
@@ -63,16 +88,24 @@ __device__ __forceinline__ void finish_row_act(const greta_out_segment &g, uint3
       if (j < cnt) store_out(g.out, g.out_fmt, base + (size_t)j * g.ld, apply_act(ACT, __uint_as_float(v[j]) + bias, rate), g.pair_offset);
   }
 }
-__device__ __forceinline__ void finish_row(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32]) {
+__device__ __forceinline__ void finish_row(const greta_out_segment &g, uint32_t r, float bias, uint32_t m, uint32_t cnt, const uint32_t (&v)[32], bool on,
+                                           bool paired) {
   switch (g.act) {
-    case GRETA_ACT_GELU_ERF: finish_row_act<GRETA_ACT_GELU_ERF>(g, r, bias, m, cnt, v); break;
-    case GRETA_ACT_SIGMOID: finish_row_act<GRETA_ACT_SIGMOID>(g, r, bias, m, cnt, v); break;
-    case GRETA_ACT_TANH: finish_row_act<GRETA_ACT_TANH>(g, r, bias, m, cnt, v); break;
-    case GRETA_ACT_DELTA_DECAY: finish_row_act<GRETA_ACT_DELTA_DECAY>(g, r, bias, m, cnt, v); break;
-    case GRETA_ACT_RELU2: finish_row_act<GRETA_ACT_RELU2>(g, r, bias, m, cnt, v); break;
-    case GRETA_ACT_SOFTPLUS_DECAY: finish_row_act<GRETA_ACT_SOFTPLUS_DECAY>(g, r, bias, m, cnt, v); break;
-    default: finish_row_act<GRETA_ACT_NONE>(g, r, bias, m, cnt, v); break;
+    case GRETA_ACT_GELU_ERF: finish_row_act<GRETA_ACT_GELU_ERF>(g, r, bias, m, cnt, v, on, paired); break;
+    case GRETA_ACT_SIGMOID: finish_row_act<GRETA_ACT_SIGMOID>(g, r, bias, m, cnt, v, on, paired); break;
+    case GRETA_ACT_TANH: finish_row_act<GRETA_ACT_TANH>(g, r, bias, m, cnt, v, on, paired); break;
+    case GRETA_ACT_DELTA_DECAY: finish_row_act<GRETA_ACT_DELTA_DECAY>(g, r, bias, m, cnt, v, on, paired); break;
+    case GRETA_ACT_RELU2: finish_row_act<GRETA_ACT_RELU2>(g, r, bias, m, cnt, v, on, paired); break;
+    case GRETA_ACT_SOFTPLUS_DECAY: finish_row_act<GRETA_ACT_SOFTPLUS_DECAY>(g, r, bias, m, cnt, v, on, paired); break;
+    default: finish_row_act<GRETA_ACT_NONE>(g, r, bias, m, cnt, v, on, paired); break;
   }
+}
+// The whole warp's 32 rows can be stored in pairs: one segment with 16-bit outputs, even columns on even lanes.
+__device__ __forceinline__ bool rows_paired(const greta_out_segment &g, uint32_t r, int segment, bool on) {
+  const bool same = __shfl_sync(0xffffffffu, segment, 0) == segment;
+  const bool fits = on && (g.out_fmt == GRETA_OUT_F16 || g.out_fmt == GRETA_OUT_BF16) && g.ld % 2 == 0 && ((g.col0 + r + threadIdx.x) & 1) == 0 &&
+                    (reinterpret_cast<uintptr_t>(g.out) & 3) == 0;
+  return __all_sync(0xffffffffu, same && fits);
 }
 
 // A copy still in flight must not outlive the CTA: after an abort the producer gives the last ones a bounded chance to land.
@@ -182,11 +215,14 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
       greta_out_segment g{};
       uint32_t r = 0;
       float bias = 0.f;
+      int which = -1;
       if (row < N) {
-        g = sg.s[segment_of(sg, row)];
+        which = segment_of(sg, row);
+        g = sg.s[which];
         r = row - g.row0;
         if (g.bias) bias = __ldg(g.bias + r);
       }
+      const bool paired = rows_paired(g, r, which, row < N);
       if (!mbar_wait(&acc_full[b], (it >> 1) & 1, abort_flag, 400 + b)) break;
       tc_fence_after();
 #pragma unroll 1
@@ -202,7 +238,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_consta
           __syncwarp();
           if (lane == 0) mbar_arrive(&acc_empty[b]);
         }
-        if (row < N && m0 + c < M) finish_row(g, r, bias, m0 + c, min(32u, M - m0 - c), v);
+        if (m0 + c < M) finish_row(g, r, bias, m0 + c, min(32u, M - m0 - c), v, row < N, paired);
       }
     }
   }
@@ -322,12 +358,24 @@ linear_tc_split_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_
     const uint32_t row_l = wq * 32 + lane, row = n0 + row_l;
     if (row < N) {
       const greta_out_segment g = sg.s[segment_of(sg, row)];
-      for (uint32_t j = half; j < per; j += halves) {
+      constexpr int U = 8;  // tokens whose partial sums (and old values) are in flight together
+      for (uint32_t j = half; j < per; j += halves * U) {
         const uint32_t c = rank * per + j, m = m0 + c;
-        if (m >= M) break;
-        float z = 0.f;
-        for (uint32_t r = 0; r < S; ++r) z += *cl.map_shared_rank(part + (size_t)c * TILE_N + row_l, r);
-        store_segment(g, row, m, z);
+        float z[U], old[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          z[u] = old[u] = 0.f;
+          if (g.accumulate && j + u * halves < per && m + u * halves < M) old[u] = static_cast<float *>(g.out)[(size_t)(m + u * halves) * g.ld + g.col0 + row - g.row0];
+        }
+        for (uint32_t q = 0; q < S; ++q) {
+          const float *from = cl.map_shared_rank(part + (size_t)c * TILE_N + row_l, q);
+#pragma unroll
+          for (int u = 0; u < U; ++u)
+            if (j + u * halves < per) z[u] += from[(size_t)u * halves * TILE_N];
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+          if (j + u * halves < per && m + u * halves < M) store_segment(g, row, m + u * halves, z[u], old[u]);
       }
     }
   }
@@ -418,22 +466,23 @@ int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, cons
   return launched("linear_tc_kernel");
 }
 
-// Token tile and K split for a product: the widest tile whose tiles (times the CTAs that share one) fill most SMs.
+// Token tile and K split for a product: the pair with the smallest estimate of its time.  Of one SM, in ns: a stage's bytes from L2 (all
+// SMs share about 13.5 TB/s, one takes up to 170 GB/s) or its products, whichever takes longer; the last tile's epilogue; and, for a split,
+// the exchange of the partial tiles.
 void plan_dense(uint32_t M, uint32_t N, uint32_t K, uint32_t *tn, uint32_t *split) {
   const uint32_t row_tiles = (N + TILE_N - 1) / TILE_N, KT = (K + BK - 1) / BK, sms = (uint32_t)sm_count();
-  uint32_t best = 0;
+  float best = 0.f;
   for (uint32_t t : {256u, 128u, 64u, 32u}) {
     if (t > 32 && M <= t / 2) continue;  // mostly padding
     const uint32_t tiles = row_tiles * ((M + t - 1) / t);
-    uint32_t s = 1;
-    while (s < 8 && tiles * s * 2 <= sms && KT >= s * 2 * 4) s *= 2;
-    const uint32_t fill = std::min(sms, tiles * s);
-    if (fill * 10 > best * 12 || best == 0) {  // a narrower tile has to fill clearly more SMs
-      best = fill;
-      *tn = t;
-      *split = s;
+    for (uint32_t s = 1; s <= 8; s *= 2) {
+      if (s > 1 && (tiles * s > sms || KT < s * 3)) break;
+      const uint32_t ctas = std::min(tiles * s, sms), rounds = (tiles * s + sms - 1) / sms;
+      const float bytes = TILE_N * BK * 2 + (float)t * BK * 2, rate = std::min(170.f, 13500.f / ctas);
+      const float stage = std::max(bytes / rate, t * 1.5f);
+      const float ns = rounds * (float)((KT + s - 1) / s) * stage + (s == 1 ? t * (t >= 64 ? 11.f : 20.f) : 1500.f + t * 20.f / s);
+      if (best == 0.f || ns < best) best = ns, *tn = t, *split = s;
     }
-    if (best * 10 >= sms * 8) break;
   }
 }
 
