@@ -466,6 +466,35 @@ int launch_dense(cudaStream_t s, const greta_linear *l, const Segments &sg, cons
   return launched("linear_tc_kernel");
 }
 
+// Clusters of `split` CTAs (one per SM) that the device runs at the same time: a GPC's SMs may not divide by the cluster size.
+uint32_t resident_clusters(uint32_t split) {
+  static uint32_t known[64][4] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  uint32_t *n = &known[dev & 63][split == 2 ? 1 : split == 4 ? 2 : 3];
+  if (*n == 0) {
+    using C = DCfg<32>;
+    cudaFuncSetAttribute(linear_tc_split_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((uint32_t)sm_count() / split * split);
+    cfg.blockDim = dim3(C::THREADS);
+    cfg.dynamicSmemBytes = C::SMEM;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = split;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    int got = 0;
+    if (cudaOccupancyMaxActiveClusters(&got, linear_tc_split_kernel<32>, &cfg) != cudaSuccess || got < 1) {
+      cudaGetLastError();
+      got = sm_count() / (int)split;
+    }
+    *n = (uint32_t)got;
+  }
+  return *n;
+}
+
 // Token tile and K split for a product: the pair with the smallest estimate of its time.  Of one SM, in ns: a stage's bytes from L2 (all
 // SMs share about 13.5 TB/s, one takes up to 170 GB/s) or its products, whichever takes longer; the last tile's epilogue; and, for a split,
 // the exchange of the partial tiles.
@@ -477,7 +506,7 @@ void plan_dense(uint32_t M, uint32_t N, uint32_t K, uint32_t *tn, uint32_t *spli
     const uint32_t tiles = row_tiles * ((M + t - 1) / t);
     for (uint32_t s = 1; s <= 8; s *= 2) {
       if (s > 1 && (tiles * s > sms || KT < s * 3)) break;
-      const uint32_t ctas = std::min(tiles * s, sms), rounds = (tiles * s + sms - 1) / sms;
+      const uint32_t at_once = s == 1 ? sms : resident_clusters(s), ctas = std::min(tiles, at_once) * s, rounds = (tiles + at_once - 1) / at_once;
       const float bytes = TILE_N * BK * 2 + (float)t * BK * 2, rate = std::min(170.f, 13500.f / ctas);
       const float stage = std::max(bytes / rate, t * 1.5f);
       const float ns = rounds * (float)((KT + s - 1) / s) * stage + (s == 1 ? t * (t >= 64 ? 11.f : 20.f) : 1500.f + t * 20.f / s);
