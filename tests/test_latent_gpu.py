@@ -10,7 +10,7 @@ import pytest
 
 from _latent import CONFIGS, L, bf16_bits, bf16_round, logits_error, make_weights, write_model
 from _support import ROOT, load_package, max_abs_rel
-from test_hybrid_gpu import dev, pad_cols, run_linear, sync
+from test_hybrid_gpu import dev, pad_cols, sync
 
 pytestmark = pytest.mark.gpu
 
